@@ -1,4 +1,5 @@
-"""ctypes binding of ``libleankv_b200.so`` (the C ABI declared in ``include/leankv_b200.h``).
+"""ctypes bindings of ``libleankv_b200.so`` and ``libleankv_mixers.so`` (the C ABI declared in
+``include/leankv_b200.h`` and ``include/leankv_mixers.h``).
 
 There is no CPU or PyTorch fallback behind these calls: if the library is missing or a
 kernel reports an error, a ``RuntimeError`` is raised.
@@ -13,6 +14,7 @@ from ctypes import (POINTER, Structure, c_char_p, c_float, c_int, c_int32, c_lon
 
 _PKG_DIR = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_PKG_DIR, "libleankv_b200.so")
+MIXERS_PATH = os.path.join(_PKG_DIR, "libleankv_mixers.so")
 
 MAX_SEGMENTS = 4
 TQ_PAGE_TOKENS = 16
@@ -122,31 +124,121 @@ SIGNATURES = {
                                         c_void_p]),
 }
 
+
+# ── libleankv_mixers.so ──────────────────────────────────────────────────────────────────────
+
+DT_BF16, DT_F32 = 1, 2
+MAX_MIX = 8
+STATE_PARITY = 6         # state word that selects the half of a double-buffered previous-token vector
+
+
+class DenseGemv(Structure):
+    """Mirror of ``leankv_dense_gemv_t``."""
+
+    _fields_ = [("w", c_void_p), ("x", c_void_p), ("y", c_void_p),
+                ("dtype", c_int), ("rows", c_int), ("cols", c_int), ("gated", c_int),
+                ("gain", c_void_p), ("eps", c_float),
+                ("n_mix", c_int), ("mix_end", c_int * MAX_MIX), ("mu", c_void_p * MAX_MIX),
+                ("prev", c_void_p), ("state", c_void_p),
+                ("bias", c_void_p), ("bias_rows", c_int),
+                ("scale", c_void_p), ("residual", c_void_p)]
+
+
+class StreamNorm(Structure):
+    """Mirror of ``leankv_stream_norm_t``."""
+
+    _fields_ = [("x_in", c_void_p), ("x_out", c_void_p), ("delta", c_void_p), ("scale", c_void_p),
+                ("gain", c_void_p), ("h", c_void_p), ("mixed", c_void_p), ("mu", c_void_p * MAX_MIX),
+                ("prev_in", c_void_p), ("prev_out", c_void_p),
+                ("dtype", c_int), ("delta_dtype", c_int), ("rows", c_int), ("width", c_int), ("n_mix", c_int),
+                ("eps", c_float)]
+
+
+class WindowPool(Structure):
+    """Mirror of ``leankv_window_pool_t``."""
+
+    _fields_ = [("dtype", c_int), ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("vdim", c_int),
+                ("dim_pad", c_int), ("vdim_pad", c_int),
+                ("size", c_int), ("pool", c_int), ("ring", c_int), ("max_blocks", c_int),
+                ("scale", c_float),
+                ("k_ring", c_void_p), ("v_ring", c_void_p), ("k_pool", c_void_p), ("v_pool", c_void_p),
+                ("q_norm", c_void_p), ("k_norm", c_void_p), ("eps", c_float), ("talk", c_void_p)]
+
+
+class TimeMix(Structure):
+    """Mirror of ``leankv_time_mix_t``."""
+
+    _fields_ = [("dtype", c_int), ("heads", c_int), ("dim", c_int),
+                ("S", c_void_p), ("u", c_void_p), ("w0", c_void_p), ("norm", c_void_p), ("eps", c_float)]
+
+
+class MixerStep(Structure):
+    """Mirror of ``leankv_mixer_step_t``."""
+
+    _fields_ = [("y", c_void_p), ("qkv_off", c_int), ("rkvg_off", c_int), ("w1_off", c_int), ("rank", c_int),
+                ("w2", c_void_p), ("out", c_void_p), ("right_off", c_int),
+                ("left_scale", c_float), ("right_scale", c_float), ("state", c_void_p), ("max_pos", c_int),
+                ("ws", c_void_p), ("ws_bytes", c_size_t)]
+
+
+MIXER_SIGNATURES = {
+    "leankv_dense_gemv": (c_int, [POINTER(DenseGemv), c_void_p]),
+    "leankv_embed_begin": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]),
+    "leankv_greedy_end": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
+    "leankv_stream_norm": (c_int, [POINTER(StreamNorm), c_void_p]),
+    "leankv_silu_mul": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "leankv_tanh_split": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "leankv_window_pool_append": (c_int, [POINTER(WindowPool), c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                          c_void_p]),
+    "leankv_window_pool_workspace_bytes": (c_size_t, [POINTER(WindowPool), c_int, c_int]),
+    "leankv_window_pool_attend": (c_int, [POINTER(WindowPool), c_void_p, c_void_p, c_int, c_float, c_int, c_int,
+                                          c_void_p, c_size_t, c_void_p]),
+    "leankv_time_mix_workspace_bytes": (c_size_t, [POINTER(TimeMix), c_int]),
+    "leankv_time_mix_rows": (c_int, [POINTER(TimeMix), c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                     c_int, c_float, c_int, c_void_p, c_size_t, c_void_p]),
+    "leankv_mixer_step_workspace_bytes": (c_size_t, [POINTER(WindowPool), c_int]),
+    "leankv_mixer_step": (c_int, [POINTER(WindowPool), POINTER(TimeMix), POINTER(MixerStep), c_void_p]),
+}
+_COMMON = ("leankv_strerror", "leankv_last_cuda_error", "leankv_abi_version")     # capi.cu, in both libraries
+
 _lib = None
+_mixers = None
+
+
+def _load(path: str, signatures: dict) -> ctypes.CDLL:
+    if not os.path.exists(path):
+        raise RuntimeError(
+            f"{path} is missing: build it with `python -m leankv_b200.build` "
+            "(leankv_b200 has no CPU or PyTorch fallback)")
+    handle = ctypes.CDLL(path)
+    for name, (restype, argtypes) in signatures.items():
+        fn = getattr(handle, name)   # AttributeError if the build is stale
+        fn.restype = restype
+        fn.argtypes = argtypes
+    return handle
 
 
 def lib() -> ctypes.CDLL:
     """Load the shared library once; raise if it has not been built."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise RuntimeError(
-                f"{LIB_PATH} is missing: build it with `python -m leankv_b200.build` "
-                "(leankv_b200 has no CPU or PyTorch fallback)")
-        handle = ctypes.CDLL(LIB_PATH)
-        for name, (restype, argtypes) in SIGNATURES.items():
-            fn = getattr(handle, name)   # AttributeError if the build is stale
-            fn.restype = restype
-            fn.argtypes = argtypes
-        _lib = handle
+        _lib = _load(LIB_PATH, SIGNATURES)
     return _lib
 
 
-def check(code: int, what: str) -> None:
-    """Raise ``RuntimeError`` for a negative status code."""
+def mixers() -> ctypes.CDLL:
+    """The token-mixer library, loaded once."""
+    global _mixers
+    if _mixers is None:
+        _mixers = _load(MIXERS_PATH, {**MIXER_SIGNATURES, **{n: SIGNATURES[n] for n in _COMMON}})
+    return _mixers
+
+
+def check(code: int, what: str, handle=None) -> None:
+    """Raise ``RuntimeError`` for a negative status code (``handle``: the library that returned it)."""
     if code == 0:
         return
-    handle = lib()
+    handle = handle or lib()
     msg = handle.leankv_strerror(code).decode()
     if code == -4:
         msg += ": " + handle.leankv_last_cuda_error().decode()

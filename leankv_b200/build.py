@@ -1,12 +1,14 @@
-"""Builds ``libleankv_b200.so`` (the C-ABI library) in-tree with nvcc for sm_100a.
+"""Builds the C-ABI libraries in-tree with nvcc for sm_100a.
 
-Usage: ``python -m leankv_b200.build [--force] [--verbose]``. The library is placed next
-to this file so that it travels with a snapshot of the source tree. nvcc cross-compiles
-without a GPU present.
+Usage: ``python -m leankv_b200.build [--force] [--verbose]``. ``libleankv_b200.so`` holds the TEAL and
+TurboQuant kernels, ``libleankv_mixers.so`` the token mixers and dense layers; a model loads (and on
+first use builds) the one it needs. The libraries are placed next to this file so that they travel
+with a snapshot of the source tree. nvcc cross-compiles without a GPU present.
 """
 
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -17,9 +19,16 @@ PKG_DIR = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(PKG_DIR)
 CSRC = os.path.join(PKG_DIR, "csrc")
 BUILD_DIR = os.path.join(PKG_DIR, "build")
-LIB_PATH = os.path.join(PKG_DIR, "libleankv_b200.so")
 
-SOURCES = ["capi.cu", "teal_gemv.cu", "tq_quantize.cu", "tq_attn.cu", "decoder_ops.cu", "decode_fused.cu"]
+# library -> sources; capi.cu (status codes, device queries) is linked into each
+LIBRARIES = {
+    "libleankv_b200.so": ["capi.cu", "teal_gemv.cu", "tq_quantize.cu", "tq_attn.cu", "decoder_ops.cu",
+                          "decode_fused.cu"],
+    "libleankv_mixers.so": ["capi.cu", "dense_gemv.cu", "stream_ops.cu", "window_pool.cu", "time_mix.cu",
+                            "mixer_step.cu"],
+}
+LIB_PATH = os.path.join(PKG_DIR, "libleankv_b200.so")
+MIXERS_PATH = os.path.join(PKG_DIR, "libleankv_mixers.so")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -44,13 +53,15 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    """Compile every kernel source and link the shared library. Returns its path."""
+def build_library(name: str, force: bool = False, verbose: bool = False) -> str:
+    """Compile the sources of one library and link it. Returns its path. Safe to call from several
+    processes at once (one builds, the others wait)."""
     os.makedirs(BUILD_DIR, exist_ok=True)
     nvcc = _nvcc()
     headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    headers.append(os.path.join(ROOT, "include", "leankv_b200.h"))
-    sources = [s for s in SOURCES if os.path.exists(os.path.join(CSRC, s))]
+    headers += [os.path.join(ROOT, "include", f) for f in os.listdir(os.path.join(ROOT, "include"))]
+    sources = LIBRARIES[name]
+    target = os.path.join(PKG_DIR, name)
 
     def compile_one(src: str) -> str:
         path = os.path.join(CSRC, src)
@@ -67,15 +78,23 @@ def build(force: bool = False, verbose: bool = False) -> str:
                 raise RuntimeError(f"nvcc failed on {src}")
         return obj
 
-    with ThreadPoolExecutor(max_workers=min(8, len(sources))) as pool:
-        objs = list(pool.map(compile_one, sources))
+    with open(os.path.join(BUILD_DIR, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        with ThreadPoolExecutor(max_workers=min(8, len(sources))) as pool:
+            objs = list(pool.map(compile_one, sources))
+        if force or _stale(target, objs):
+            cmd = [nvcc, "-shared", "-o", target, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+            res = subprocess.run(cmd, capture_output=True, text=True)
+            if res.returncode != 0:
+                sys.stderr.write(res.stdout + res.stderr)
+                raise RuntimeError(f"link of {name} failed")
+    return target
 
-    if force or _stale(LIB_PATH, objs):
-        cmd = [nvcc, "-shared", "-o", LIB_PATH, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            sys.stderr.write(res.stdout + res.stderr)
-            raise RuntimeError("link of libleankv_b200.so failed")
+
+def build(force: bool = False, verbose: bool = False) -> str:
+    """Build every library. Returns the path of ``libleankv_b200.so``."""
+    for name in LIBRARIES:
+        build_library(name, force, verbose)
     return LIB_PATH
 
 

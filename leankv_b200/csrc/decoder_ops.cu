@@ -7,27 +7,10 @@
 
 #include <algorithm>
 
-#include "common.cuh"
+#include "decode_frame.cuh"
 
 namespace leankv {
 namespace {
-
-// Decode state words (int32[8], device), as the header describes them beside leankv_decode_begin: position,
-// step count, and the one-sequence page table (kv_indptr[0..1], kv_last_page_len, start position).
-enum { kPos = 0, kStep = 1, kIndptr0 = 2, kIndptr1 = 3, kLastLen = 4, kStartPos = 5 };
-
-__device__ __forceinline__ float block_sum(float v, float* s_tmp) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    if (lane == 0) s_tmp[warp] = v;
-    __syncthreads();
-    const int nw = (blockDim.x + 31) >> 5;
-    float t = 0.f;
-    for (int w = 0; w < nw; ++w) t += s_tmp[w];   // fixed order: bit-reproducible
-    __syncthreads();
-    return t;
-}
 
 // Optional residual update h += delta (fp16 add, as the decoder block does), then
 // y = w * fp16( h * rsqrt(mean(h^2) + eps) ), statistics in fp32.
@@ -68,7 +51,7 @@ __global__ void __launch_bounds__(kNormThreads) rmsnorm_kernel(__half* x, const 
             }
         }
     }
-    const float tot = block_sum(ss, s_tmp);
+    const float tot = cta_sum(ss, s_tmp);
     const float r = rsqrtf(tot / (float)n + eps);
 #pragma unroll
     for (int it = 0; it < kNormVecs; ++it) {
@@ -86,25 +69,6 @@ __global__ void __launch_bounds__(kNormThreads) rmsnorm_kernel(__half* x, const 
             }
             reinterpret_cast<uint4*>(y)[i] = o;
         }
-    }
-}
-
-// Fetch the embedding row of the current token and derive this step's page-table words.
-__global__ void __launch_bounds__(256) decode_begin_kernel(const __half* table, const long long* token,
-                                                           __half* h, int hidden, int vocab,
-                                                           int* state) {
-    pdl_begin();
-    long long tok = *token;
-    if (tok < 0 || tok >= vocab) tok = 0;
-    const uint4* src = reinterpret_cast<const uint4*>(table + (size_t)tok * hidden);
-    uint4* dst = reinterpret_cast<uint4*>(h);
-    for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) dst[i] = __ldg(src + i);
-    if (threadIdx.x == 0) {
-        const int pos = state[kPos];
-        state[kStartPos] = pos;
-        state[kIndptr0] = 0;
-        state[kIndptr1] = pos / 16 + 1;
-        state[kLastLen] = pos % 16 + 1;
     }
 }
 
@@ -126,57 +90,7 @@ __global__ void __launch_bounds__(64) rope_kernel(const __half* qkv, const float
     dst[i + 64] = __hadd(__hmul(b, c), __hmul(a, s));
 }
 
-// Greedy next token (lowest index wins ties), appended to the history; advances the position.
-// One CTA per sequence: pos / step are that sequence's words.
-__global__ void __launch_bounds__(1024) decode_end_kernel(const __half* logits, int vocab,
-                                                          long long* token, long long* history,
-                                                          int history_cap, int* pos, int* step_ptr) {
-    __shared__ float s_v[32];
-    __shared__ int s_i[32];
-    pdl_begin();
-    logits += (size_t)blockIdx.x * vocab;
-    token += blockIdx.x;
-    history += (size_t)blockIdx.x * history_cap;
-    pos += blockIdx.x;
-    step_ptr += blockIdx.x;
-    float best = -INFINITY;
-    int best_i = 0x7fffffff;
-    const int nvec = vocab >> 3;     // 16-byte loads; indices ascend within a thread, so '>' keeps the lowest
-    for (int vi = threadIdx.x; vi < nvec; vi += blockDim.x) {
-        const uint4 a = __ldg(reinterpret_cast<const uint4*>(logits) + vi);
-        const __half* hp = reinterpret_cast<const __half*>(&a);
-#pragma unroll
-        for (int q = 0; q < 8; ++q) {
-            const float v = __half2float(hp[q]);
-            if (v > best) { best = v; best_i = vi * 8 + q; }
-        }
-    }
-    for (int i = nvec * 8 + threadIdx.x; i < vocab; i += blockDim.x) {
-        const float v = __half2float(logits[i]);
-        if (v > best || (v == best && i < best_i)) { best = v; best_i = i; }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, best_i, o);
-        if (ov > best || (ov == best && oi < best_i)) { best = ov; best_i = oi; }
-    }
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    if (lane == 0) { s_v[warp] = best; s_i[warp] = best_i; }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        for (int w = 1; w < (int)(blockDim.x >> 5); ++w)
-            if (s_v[w] > best || (s_v[w] == best && s_i[w] < best_i)) { best = s_v[w]; best_i = s_i[w]; }
-        if (best_i == 0x7fffffff) best_i = 0;   // all-NaN row
-        *token = best_i;
-        const int step = *step_ptr;
-        if (step < history_cap) history[step] = best_i;
-        *step_ptr = step + 1;
-        *pos = *pos + 1;
-    }
-}
-
-// The same for an output head that is split over the vocabulary among tensor-parallel ranks: every
+// Greedy next token (as decode_end_kernel) for an output head that is split over the vocabulary among tensor-parallel ranks: every
 // rank finds the best of its own slice, sends {value, index} (two 64-bit words, each tagged with the
 // step's epoch like the partial sums of the row-parallel GEMV) to every rank's receive area, waits
 // (bounded) for all ranks' words, and takes the largest value, lowest index on ties: every rank
@@ -349,7 +263,7 @@ extern "C" int leankv_decode_begin(const void* embed_table, const long long* tok
                                    int hidden, int vocab, int32_t* state, void* stream) {
     if (!embed_table || !token || !h || !state || hidden <= 0 || vocab <= 0) return LEANKV_EINVAL;
     if (hidden % 8 != 0 || !aligned16(embed_table) || !aligned16(h)) return LEANKV_EALIGN;
-    LEANKV_CUDA_TRY(launch_kernel(decode_begin_kernel, dim3(1), dim3(256), 0, static_cast<cudaStream_t>(stream),
+    LEANKV_CUDA_TRY(launch_kernel(decode_begin_kernel<__half, __half>, dim3(1), dim3(256), 0, static_cast<cudaStream_t>(stream),
                                   static_cast<const __half*>(embed_table), token, static_cast<__half*>(h),
                                   hidden, vocab, state));
     return LEANKV_OK;
@@ -372,9 +286,9 @@ extern "C" int leankv_decode_end(const void* logits, int vocab, long long* token
                                  int history_cap, int32_t* state, void* stream) {
     if (!logits || !token || !history || !state || vocab <= 0 || history_cap < 0) return LEANKV_EINVAL;
     if (!aligned16(logits)) return LEANKV_EALIGN;
-    LEANKV_CUDA_TRY(launch_kernel(decode_end_kernel, dim3(1), dim3(1024), 0, static_cast<cudaStream_t>(stream),
+    LEANKV_CUDA_TRY(launch_kernel(decode_end_kernel<__half>, dim3(1), dim3(1024), 0, static_cast<cudaStream_t>(stream),
                                   static_cast<const __half*>(logits), vocab, token, history, history_cap,
-                                  state + kPos, state + kStep));
+                                  state + kPos, state + kStep, static_cast<int*>(nullptr)));
     return LEANKV_OK;
 }
 
@@ -456,9 +370,9 @@ extern "C" int leankv_batch_decode_end(const void* logits, int vocab, int B, lon
     if (!logits || !tokens || !history || !pos || !steps || vocab <= 0 || B <= 0 || history_cap < 0)
         return LEANKV_EINVAL;
     if (!aligned16(logits) || vocab % 8 != 0) return LEANKV_EALIGN;
-    LEANKV_CUDA_TRY(launch_kernel(decode_end_kernel, dim3(B), dim3(1024), 0, static_cast<cudaStream_t>(stream),
+    LEANKV_CUDA_TRY(launch_kernel(decode_end_kernel<__half>, dim3(B), dim3(1024), 0, static_cast<cudaStream_t>(stream),
                                   static_cast<const __half*>(logits), vocab, tokens, history, history_cap, pos,
-                                  steps));
+                                  steps, static_cast<int*>(nullptr)));
     return LEANKV_OK;
 }
 

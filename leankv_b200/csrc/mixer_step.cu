@@ -1,0 +1,204 @@
+// One decode step of a layer's token mixers, in one launch. The first thread-block cluster runs the window +
+// pooled-block attention (its CTAs split the visible keys and merge through distributed shared memory), every
+// further CTA one head of the matrix-state time mixing: the two mixers read the same projections and are
+// independent, so they run side by side.
+
+#include <algorithm>
+
+#include "decode_frame.cuh"
+#include "window_pool.cuh"
+
+namespace leankv {
+namespace {
+
+constexpr int kStepThreads = 512;
+constexpr int kStepCluster = 8;
+constexpr int kStepSmemFloats = 200 * 1024 / 4;
+
+struct StepParams {
+    leankv_window_pool_t left;
+    leankv_time_mix_t right;
+    leankv_mixer_step_t s;
+    int has_left, has_right, n_max;
+};
+
+template <typename T>
+__device__ void left_step(const StepParams& p, float* sm, float* s_tmp, int rank) {
+    const leankv_window_pool_t& a = p.left;
+    const AttendPlan pl(a, kStepThreads, (p.n_max + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
+    const int tid = threadIdx.x, i = p.s.state[kPos], G = a.kv_heads;
+    const int nq = a.heads * a.dim, nk = G * a.dim;
+    const float* y = p.s.y + p.s.qkv_off;       // biases are already in
+    const float fq = row_factor(y, nullptr, nq, a.q_norm != nullptr, a.eps, s_tmp);
+    const float fk = row_factor(y + nq, nullptr, nk, a.k_norm != nullptr, a.eps, s_tmp);
+    for (int e = tid; e < a.heads * a.dim_pad; e += kStepThreads) {
+        const int h = e / a.dim_pad, d = e - h * a.dim_pad, x = h * a.dim + d;
+        sm[pl.q + e] = d < a.dim ? y[x] * fq * (a.q_norm ? __ldg(a.q_norm + x) : 1.f) * a.scale : 0.f;
+    }
+    const int slot = i % a.ring;
+    T* k_ring = static_cast<T*>(a.k_ring);
+    T* v_ring = static_cast<T*>(a.v_ring);
+    for (int e = tid; e < G * a.dim_pad; e += kStepThreads) {
+        const int g = e / a.dim_pad, d = e - g * a.dim_pad, x = g * a.dim + d;
+        const T v = from_f32<T>(d < a.dim ? y[nq + x] * fk * (a.k_norm ? __ldg(a.k_norm + x) : 1.f) : 0.f);
+        sm[pl.knew + e] = to_f32(v);
+        if (rank == 0) k_ring[(size_t)slot * G * a.dim_pad + e] = v;
+    }
+    for (int e = tid; e < G * a.vdim_pad; e += kStepThreads) {
+        const int g = e / a.vdim_pad, d = e - g * a.vdim_pad;
+        const T v = from_f32<T>(d < a.vdim ? y[nq + nk + g * a.vdim + d] : 0.f);
+        sm[pl.vnew + e] = to_f32(v);
+        if (rank == 0) v_ring[(size_t)slot * G * a.vdim_pad + e] = v;
+    }
+    __syncthreads();
+    float* p_gmem = static_cast<float*>(p.s.ws) + (size_t)rank * 2 * a.heads * pl.ldp;
+    attend_query<T, float>(a, pl, sm, p_gmem, i, true, rank, kStepCluster, p.s.out, p.s.left_scale);
+
+    // the block this token completes (not visible to it: it ends at i > i - size)
+    if ((i + 1) % a.pool == 0 && (i + 1) / a.pool <= a.max_blocks) {
+        const int b = i / a.pool, p0 = b * a.pool;
+        auto mean = [&](const T* ring, const float* fresh, T* dst, int n) {
+            for (int e = rank * kStepThreads + tid; e < n; e += kStepCluster * kStepThreads) {
+                float t = 0.f;
+                for (int x = 0; x < a.pool - 1; ++x) t += to_f32(ring[(size_t)((p0 + x) % a.ring) * n + e]);
+                dst[(size_t)b * n + e] = from_f32<T>((t + fresh[e]) / (float)a.pool);
+            }
+        };
+        mean(k_ring, sm + pl.knew, static_cast<T*>(a.k_pool), G * a.dim_pad);
+        mean(v_ring, sm + pl.vnew, static_cast<T*>(a.v_pool), G * a.vdim_pad);
+    }
+}
+
+template <typename T>
+__device__ void right_step(const StepParams& p, float* sm, float* s_tmp, int head) {
+    const leankv_time_mix_t& a = p.right;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.dim, N = a.heads * d, c0 = head * d;
+    float* s_r = sm;
+    float* s_k = s_r + d;
+    float* s_w = s_k + d;
+    float* s_v = s_w + d;
+    float* s_o = s_v + d;                      // [slices][d]
+    const float* y = p.s.y + p.s.rkvg_off + c0;
+    const float* y1 = p.s.y + p.s.w1_off;
+    const T* w2 = static_cast<const T*>(p.s.w2);
+    float bonus = 0.f;
+    for (int c = tid; c < d; c += kStepThreads) {
+        const float r = y[c], k = y[N + c];
+        s_r[c] = r;
+        s_k[c] = k;
+        s_v[c] = y[2 * N + c];
+        bonus = fmaf(r * __ldg(a.u + c0 + c), k, bonus);
+    }
+    for (int c = warp; c < d; c += kStepThreads / 32) {
+        float z = 0.f;
+        for (int x = lane; x < p.s.rank; x += 32) z = fmaf(to_f32(w2[(size_t)(c0 + c) * p.s.rank + x]), tanhf(y1[x]), z);
+        z = warp_sum(z);
+        if (lane == 0) s_w[c] = expf(-expf(z + __ldg(a.w0 + c0 + c)));
+    }
+    bonus = cta_sum(bonus, s_tmp);             // synchronises
+    const int slices = max(1, kStepThreads / d), sl = tid / d, col = tid - sl * d;
+    float* S = a.S + (size_t)head * d * d;
+    if (sl < slices) {
+        const int k0 = d * sl / slices, k1 = d * (sl + 1) / slices;
+        const float v = s_v[col];
+        float o = 0.f;
+#pragma unroll 8
+        for (int k = k0; k < k1; ++k) {
+            const float s = S[(size_t)k * d + col];
+            o = fmaf(s_r[k], s, o);
+            S[(size_t)k * d + col] = fmaf(s_w[k], s, s_k[k] * v);
+        }
+        s_o[sl * d + col] = o;
+    }
+    __syncthreads();
+    float o = 0.f;
+    if (tid < d) {
+        for (int x = 0; x < slices; ++x) o += s_o[x * d + tid];
+        o = fmaf(bonus, s_v[tid], o);
+    }
+    const float f = p.s.right_scale / sqrtf(cta_sum(o * o, s_tmp) / (float)d + a.eps);
+    if (tid < d) {
+        const float g = y[3 * N + tid];
+        p.s.out[p.s.right_off + c0 + tid] = o * f * __ldg(a.norm + c0 + tid) * g * sigmoid_f32(g);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kStepThreads) mixer_step_kernel(const __grid_constant__ StepParams p) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float s_tmp[32];
+    pdl_begin();
+    const int first = p.has_left ? kStepCluster : 0;
+    if ((int)blockIdx.x < first) left_step<T>(p, sm, s_tmp, blockIdx.x);
+    else if ((int)blockIdx.x - first < p.right.heads) right_step<T>(p, sm, s_tmp, blockIdx.x - first);
+}
+
+int keys_bound(const leankv_window_pool_t& a, int max_pos) {
+    return VisibleKeys(std::max(max_pos - 1, 0), a.size, a.pool).n;
+}
+
+template <typename T>
+int launch_step(const StepParams& p, cudaStream_t st) {
+    size_t smem = 0;
+    int grid = 0;
+    if (p.has_left) {
+        const AttendPlan pl(p.left, kStepThreads, (p.n_max + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
+        smem = (size_t)pl.total * 4;
+        grid = kStepCluster;
+    }
+    if (p.has_right) {
+        smem = std::max(smem, (size_t)(4 * p.right.dim + kStepThreads + p.right.dim) * 4);
+        grid += (p.right.heads + kStepCluster - 1) / kStepCluster * kStepCluster;
+    }
+    if (smem > 226 * 1024) return LEANKV_ELIMIT;
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(mixer_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LEANKV_CUDA_TRY(launch_cluster_kernel_ex(false, dim3(kStepCluster), mixer_step_kernel<T>, dim3(grid),
+                                             dim3(kStepThreads), smem, st, p));
+    return LEANKV_OK;
+}
+
+}  // namespace
+}  // namespace leankv
+
+using namespace leankv;
+
+extern "C" size_t leankv_mixer_step_workspace_bytes(const leankv_window_pool_t* left, int max_pos) {
+    if (!left || max_pos <= 0) return 0;
+    const int n = keys_bound(*left, max_pos);
+    const AttendPlan pl(*left, kStepThreads, (n + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
+    return pl.p_in_smem ? 0 : (size_t)kStepCluster * 2 * left->heads * pl.ldp * 4;
+}
+
+extern "C" int leankv_mixer_step(const leankv_window_pool_t* left, const leankv_time_mix_t* right,
+                                 const leankv_mixer_step_t* s, void* stream) {
+    if (!s || (!left && !right) || !s->y || !s->out || !s->state || s->max_pos <= 0) return LEANKV_EINVAL;
+    StepParams p{};
+    p.s = *s;
+    int dtype = 0;
+    if (left) {
+        if (left->heads <= 0 || left->kv_heads <= 0 || left->heads % left->kv_heads || left->dim <= 0 ||
+            left->vdim <= 0 || left->size <= 0 || left->pool <= 0 || !left->k_ring || !left->v_ring)
+            return LEANKV_EINVAL;
+        if (left->ring < std::max(left->size, left->pool) ||
+            VisibleKeys(s->max_pos - 1, left->size, left->pool).n_blk > left->max_blocks)
+            return LEANKV_ELIMIT;
+        if (left->dim_pad % 16 || left->vdim_pad % 16 || left->dim_pad < left->dim || left->vdim_pad < left->vdim)
+            return LEANKV_EALIGN;
+        if (leankv_mixer_step_workspace_bytes(left, s->max_pos) > (s->ws ? s->ws_bytes : 0)) return LEANKV_EWORKSPACE;
+        p.left = *left;
+        p.has_left = 1;
+        p.n_max = keys_bound(*left, s->max_pos);
+        dtype = left->dtype;
+    }
+    if (right) {
+        if (right->heads <= 0 || right->dim <= 0 || right->dim > kStepThreads || !right->S || !right->u || !right->w0 ||
+            !right->norm || !s->w2 || s->rank <= 0 || (left && left->dtype != right->dtype))
+            return LEANKV_EINVAL;
+        p.right = *right;
+        p.has_right = 1;
+        dtype = right->dtype;
+    }
+    if (dtype != LEANKV_DT_BF16 && dtype != LEANKV_DT_F32) return LEANKV_EUNSUPPORTED;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    return dtype == LEANKV_DT_BF16 ? launch_step<bf16>(p, st) : launch_step<float>(p, st);
+}

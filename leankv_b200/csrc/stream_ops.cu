@@ -1,0 +1,190 @@
+// Row-wise kernels around the projections of a prompt portion (residual sum, norm, token shift, gating) and
+// the two frame kernels of a decode step whose residual stream is fp32.
+
+#include <algorithm>
+
+#include "decode_frame.cuh"
+#include "leankv_mixers.h"
+
+namespace leankv {
+namespace {
+
+constexpr int kRowThreads = 256;
+
+// One CTA per row. With token shift the row above is normed a second time here (two rows of L2 reads)
+// rather than handed over through memory, so rows stay independent and one launch does the whole chain.
+template <typename T, typename D>
+__global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const leankv_stream_norm_t a) {
+    __shared__ float s_tmp[32];
+    pdl_begin();
+    const int t = blockIdx.x, W = a.width;
+    const D* delta = static_cast<const D*>(a.delta);
+    auto value = [&](int row, int i) {
+        float x = a.x_in[(size_t)row * W + i];
+        if (delta != nullptr) x = fmaf(to_f32(delta[(size_t)row * W + i]), __ldg(a.scale + i), x);
+        return x;
+    };
+    const bool shift = a.n_mix > 0;
+    float ss = 0.f, ss_above = 0.f;
+    for (int i = threadIdx.x; i < W; i += kRowThreads) {
+        const float x = value(t, i);
+        ss = fmaf(x, x, ss);
+        if (delta != nullptr) a.x_out[(size_t)t * W + i] = x;
+        if (shift && t > 0) {
+            const float y = value(t - 1, i);
+            ss_above = fmaf(y, y, ss_above);
+        }
+    }
+    const float gain = __ldg(a.gain);
+    const float rs = gain / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+    float rs_above = 0.f;
+    if (shift && t > 0) rs_above = gain / sqrtf(cta_sum(ss_above, s_tmp) / (float)W + a.eps);
+    T* h = static_cast<T*>(a.h);
+    T* mixed = static_cast<T*>(a.mixed);
+    for (int i = threadIdx.x; i < W; i += kRowThreads) {
+        const float hv = value(t, i) * rs;
+        if (h != nullptr) h[(size_t)t * W + i] = from_f32<T>(hv);
+        if (shift) {
+            const float d = (t > 0 ? value(t - 1, i) * rs_above : a.prev_in[i]) - hv;
+            for (int m = 0; m < a.n_mix; ++m)
+                mixed[((size_t)m * a.rows + t) * W + i] = from_f32<T>(fmaf(d, __ldg(a.mu[m] + i), hv));
+        }
+        if (a.prev_out != nullptr && t == a.rows - 1) a.prev_out[i] = hv;
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) silu_mul_rows_kernel(const T* gate_up, T* out, int inter, long long total) {
+    pdl_begin();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
+         i += (long long)gridDim.x * blockDim.x) {
+        const long long r = i / inter, c = i - r * inter;
+        const float g = to_f32(gate_up[r * 2 * inter + c]), u = to_f32(gate_up[r * 2 * inter + inter + c]);
+        out[i] = from_f32<T>(g * sigmoid_f32(g) * u);
+    }
+}
+
+// Eight elements per thread (inter % 8 == 0, aligned).
+template <typename T>
+__global__ void __launch_bounds__(256) silu_mul_vec_kernel(const T* gate_up, T* out, int inter, long long total8) {
+    pdl_begin();
+    const int n8 = inter >> 3;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total8;
+         i += (long long)gridDim.x * blockDim.x) {
+        const long long r = i / n8;
+        const int c = (int)(i - r * n8) * 8;
+        Raw8<T> rg, ru;
+        load8(gate_up + r * 2 * inter + c, rg);
+        load8(gate_up + r * 2 * inter + inter + c, ru);
+        float g[8], u[8];
+        unpack8(rg, g);
+        unpack8(ru, u);
+        T o[8];
+#pragma unroll
+        for (int q = 0; q < 8; ++q) o[q] = from_f32<T>(g[q] * sigmoid_f32(g[q]) * u[q]);
+        memcpy(&rg, o, sizeof(rg));
+        *reinterpret_cast<Raw8<T>*>(out + r * inter + c) = rg;
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_split_kernel(const float* in, T* out, int n, long long total) {
+    pdl_begin();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
+         i += (long long)gridDim.x * blockDim.x) {
+        const float v = tanhf(in[i]);
+        if constexpr (sizeof(T) == 4) {
+            out[i] = v;
+        } else {
+            const long long r = i / n, c = i - r * n;
+            const T hi = from_f32<T>(v);
+            out[r * 2 * n + c] = hi;
+            out[r * 2 * n + n + c] = from_f32<T>(v - to_f32(hi));
+        }
+    }
+}
+
+template <typename T, typename D>
+int launch_stream_norm(const leankv_stream_norm_t* a, cudaStream_t st) {
+    LEANKV_CUDA_TRY(launch_kernel(stream_norm_kernel<T, D>, dim3(a->rows), dim3(kRowThreads), 0, st, *a));
+    return LEANKV_OK;
+}
+
+bool known(int dtype) { return dtype == LEANKV_DT_BF16 || dtype == LEANKV_DT_F32; }
+
+}  // namespace
+}  // namespace leankv
+
+using namespace leankv;
+
+extern "C" int leankv_embed_begin(const void* table, int dtype, const long long* token, float* x, int width,
+                                  int vocab, int32_t* state, void* stream) {
+    if (!table || !token || !x || !state || width <= 0 || vocab <= 0) return LEANKV_EINVAL;
+    if (!known(dtype)) return LEANKV_EUNSUPPORTED;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (dtype == LEANKV_DT_BF16)
+        LEANKV_CUDA_TRY(launch_kernel(decode_begin_kernel<bf16, float>, dim3(1), dim3(256), 0, st,
+                                      static_cast<const bf16*>(table), token, x, width, vocab, state));
+    else
+        LEANKV_CUDA_TRY(launch_kernel(decode_begin_kernel<float, float>, dim3(1), dim3(256), 0, st,
+                                      static_cast<const float*>(table), token, x, width, vocab, state));
+    return LEANKV_OK;
+}
+
+extern "C" int leankv_greedy_end(const float* logits, int vocab, long long* token, long long* history,
+                                 int history_cap, int32_t* state, void* stream) {
+    if (!logits || !token || !history || !state || vocab <= 0 || history_cap < 0) return LEANKV_EINVAL;
+    if (!aligned16(logits)) return LEANKV_EALIGN;
+    LEANKV_CUDA_TRY(launch_kernel(decode_end_kernel<float>, dim3(1), dim3(1024), 0, static_cast<cudaStream_t>(stream),
+                                  logits, vocab, token, history, history_cap, state + kPos, state + kStep,
+                                  state + kParity));
+    return LEANKV_OK;
+}
+
+extern "C" int leankv_stream_norm(const leankv_stream_norm_t* a, void* stream) {
+    if (!a || !a->x_in || !a->gain || a->rows <= 0 || a->width <= 0 || a->n_mix < 0 || a->n_mix > LEANKV_MAX_MIX)
+        return LEANKV_EINVAL;
+    if (a->delta && (!a->x_out || !a->scale || a->x_out == a->x_in)) return LEANKV_EINVAL;
+    if (a->n_mix > 0) {
+        if (!a->mixed || !a->prev_in || !a->prev_out || a->prev_in == a->prev_out) return LEANKV_EINVAL;
+        for (int i = 0; i < a->n_mix; ++i)
+            if (!a->mu[i]) return LEANKV_EINVAL;
+    }
+    if (!known(a->dtype) || (a->delta && !known(a->delta_dtype))) return LEANKV_EUNSUPPORTED;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const bool d16 = a->delta && a->delta_dtype == LEANKV_DT_BF16;
+    if (a->dtype == LEANKV_DT_BF16)
+        return d16 ? launch_stream_norm<bf16, bf16>(a, st) : launch_stream_norm<bf16, float>(a, st);
+    return d16 ? launch_stream_norm<float, bf16>(a, st) : launch_stream_norm<float, float>(a, st);
+}
+
+extern "C" int leankv_silu_mul(const void* gate_up, void* out, int dtype, int rows, int inter, void* stream) {
+    if (!gate_up || !out || rows <= 0 || inter <= 0) return LEANKV_EINVAL;
+    if (!known(dtype)) return LEANKV_EUNSUPPORTED;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const bool vec = inter % 8 == 0 && aligned16(gate_up) && aligned16(out);
+    const long long total = (long long)rows * inter / (vec ? 8 : 1);
+    const int grid = (int)std::min<long long>((total + 255) / 256, (long long)sm_count() * 16);
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        LEANKV_CUDA_TRY(launch_kernel(vec ? silu_mul_vec_kernel<T> : silu_mul_rows_kernel<T>, dim3(grid), dim3(256), 0,
+                                      st, static_cast<const T*>(gate_up), static_cast<T*>(out), inter, total));
+        return LEANKV_OK;
+    };
+    return dtype == LEANKV_DT_BF16 ? go(bf16{}) : go(float{});
+}
+
+extern "C" int leankv_tanh_split(const float* in, void* out, int dtype, int rows, int n, void* stream) {
+    if (!in || !out || rows <= 0 || n <= 0) return LEANKV_EINVAL;
+    if (!known(dtype)) return LEANKV_EUNSUPPORTED;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const long long total = (long long)rows * n;
+    const int grid = (int)std::min<long long>((total + 255) / 256, (long long)sm_count() * 8);
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        LEANKV_CUDA_TRY(launch_kernel(tanh_split_kernel<T>, dim3(grid), dim3(256), 0, st, in, static_cast<T*>(out), n,
+                                      total));
+        return LEANKV_OK;
+    };
+    return dtype == LEANKV_DT_BF16 ? go(bf16{}) : go(float{});
+}

@@ -1,0 +1,156 @@
+// Window + pooled-block attention of a prompt portion: append (q / k norm, ring write), pooling of the blocks
+// that become complete, and attention.
+
+#include <algorithm>
+
+#include "window_pool.cuh"
+
+namespace leankv {
+namespace {
+
+constexpr int kAppendThreads = 256;
+constexpr int kAttendThreads = 256;
+constexpr int kAttendSmemFloats = 200 * 1024 / 4;
+
+// One CTA per token: bias and norm over the whole q / k projections, q to the chunk buffer, k / v into the ring.
+template <typename T>
+__global__ void __launch_bounds__(kAppendThreads) window_pool_append_kernel(const leankv_window_pool_t a,
+                                                                            const float* qkv, int ld, const float* bias,
+                                                                            T* q_out, int start) {
+    __shared__ float s_tmp[32];
+    pdl_begin();
+    const int t = blockIdx.x, G = a.kv_heads, nq = a.heads * a.dim, nk = G * a.dim;
+    const float* row = qkv + (size_t)t * ld;
+    const int slot = (start + t) % a.ring;
+    const float fq = row_factor(row, bias, nq, a.q_norm != nullptr, a.eps, s_tmp);
+    const float fk = row_factor(row + nq, bias ? bias + nq : nullptr, nk, a.k_norm != nullptr, a.eps, s_tmp);
+    auto at = [&](int i) { return row[i] + (bias != nullptr ? __ldg(bias + i) : 0.f); };
+    T* q = q_out + (size_t)t * a.heads * a.dim_pad;
+    for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAppendThreads) {
+        const int h = e / a.dim_pad, d = e - h * a.dim_pad, i = h * a.dim + d;
+        q[e] = from_f32<T>(d < a.dim ? at(i) * fq * (a.q_norm ? __ldg(a.q_norm + i) : 1.f) : 0.f);
+    }
+    T* k = static_cast<T*>(a.k_ring) + (size_t)slot * G * a.dim_pad;
+    for (int e = threadIdx.x; e < G * a.dim_pad; e += kAppendThreads) {
+        const int g = e / a.dim_pad, d = e - g * a.dim_pad, i = g * a.dim + d;
+        k[e] = from_f32<T>(d < a.dim ? at(nq + i) * fk * (a.k_norm ? __ldg(a.k_norm + i) : 1.f) : 0.f);
+    }
+    T* v = static_cast<T*>(a.v_ring) + (size_t)slot * G * a.vdim_pad;
+    for (int e = threadIdx.x; e < G * a.vdim_pad; e += kAppendThreads) {
+        const int g = e / a.vdim_pad, d = e - g * a.vdim_pad;
+        v[e] = from_f32<T>(d < a.vdim ? at(nq + nk + g * a.vdim + d) : 0.f);
+    }
+}
+
+// Blocks first .. : mean of the block's keys / values as the ring holds them. One CTA per block.
+template <typename T>
+__global__ void __launch_bounds__(256) window_pool_blocks_kernel(const leankv_window_pool_t a, int first) {
+    pdl_begin();
+    const int b = first + blockIdx.x, p0 = b * a.pool;
+    const float inv = (float)a.pool;
+    auto mean = [&](const void* ring, void* dst, int n) {
+        const T* src = static_cast<const T*>(ring);
+        for (int e = threadIdx.x; e < n; e += blockDim.x) {
+            float t = 0.f;
+            for (int i = 0; i < a.pool; ++i) t += to_f32(src[(size_t)((p0 + i) % a.ring) * n + e]);
+            static_cast<T*>(dst)[(size_t)b * n + e] = from_f32<T>(t / inv);
+        }
+    };
+    mean(a.k_ring, a.k_pool, a.kv_heads * a.dim_pad);
+    mean(a.v_ring, a.v_pool, a.kv_heads * a.vdim_pad);
+}
+
+// One CTA per query row (the fp32 route, and shapes the tile kernel does not take).
+template <typename T>
+__global__ void __launch_bounds__(kAttendThreads) window_pool_rows_kernel(const leankv_window_pool_t a, const T* q,
+                                                                          T* out, int out_ld, float out_scale,
+                                                                          int start, int n_max, float* ws) {
+    extern __shared__ __align__(16) float sm[];
+    pdl_begin();
+    const int t = blockIdx.x;
+    const AttendPlan pl(a, kAttendThreads, n_max, kAttendSmemFloats);
+    const T* row = q + (size_t)t * a.heads * a.dim_pad;
+    for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAttendThreads) sm[pl.q + e] = to_f32(row[e]) * a.scale;
+    __syncthreads();
+    attend_query<T, T>(a, pl, sm, ws + (size_t)t * 2 * a.heads * pl.ldp, start + t, false, 0, 1,
+                       out + (size_t)t * out_ld, out_scale);
+}
+
+int check_args(const leankv_window_pool_t* a) {
+    if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 ||
+        a->dim_pad < a->dim || a->vdim_pad < a->vdim || a->size <= 0 || a->pool <= 0 || a->ring <= 0 ||
+        a->max_blocks < 0 || !a->k_ring || !a->v_ring || (a->max_blocks > 0 && (!a->k_pool || !a->v_pool)))
+        return LEANKV_EINVAL;
+    if (a->dim_pad % 16 || a->vdim_pad % 16 || !aligned16(a->k_ring) || !aligned16(a->v_ring) ||
+        !aligned16(a->k_pool) || !aligned16(a->v_pool))
+        return LEANKV_EALIGN;
+    if (a->dtype != LEANKV_DT_BF16 && a->dtype != LEANKV_DT_F32) return LEANKV_EUNSUPPORTED;
+    return LEANKV_OK;
+}
+
+template <typename T>
+int append(const leankv_window_pool_t& a, const float* qkv, int ld, const float* bias, void* q, int rows, int start,
+           cudaStream_t st) {
+    LEANKV_CUDA_TRY(launch_kernel(window_pool_append_kernel<T>, dim3(rows), dim3(kAppendThreads), 0, st, a, qkv, ld,
+                                  bias, static_cast<T*>(q), start));
+    const int b0 = start / a.pool, b1 = std::min((start + rows) / a.pool, a.max_blocks);
+    if (b1 > b0)
+        LEANKV_CUDA_TRY(launch_kernel(window_pool_blocks_kernel<T>, dim3(b1 - b0), dim3(256), 0, st, a, b0));
+    return LEANKV_OK;
+}
+
+// The most keys any position below max_pos sees (the count never falls from one position to the next).
+int max_keys(const leankv_window_pool_t& a, int max_pos) {
+    return VisibleKeys(std::max(max_pos - 1, 0), a.size, a.pool).n;
+}
+
+template <typename T>
+int attend(const leankv_window_pool_t& a, const void* q, void* out, int out_ld, float out_scale, int rows, int start,
+           float* ws, cudaStream_t st) {
+    const int n_max = max_keys(a, start + rows);
+    const AttendPlan pl(a, kAttendThreads, n_max, kAttendSmemFloats);
+    const size_t smem = (size_t)pl.total * 4;
+    if (smem > 227 * 1024) return LEANKV_ELIMIT;
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(window_pool_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem));
+    LEANKV_CUDA_TRY(launch_kernel(window_pool_rows_kernel<T>, dim3(rows), dim3(kAttendThreads), smem, st, a,
+                                  static_cast<const T*>(q), static_cast<T*>(out), out_ld, out_scale, start, n_max, ws));
+    return LEANKV_OK;
+}
+
+}  // namespace
+}  // namespace leankv
+
+using namespace leankv;
+
+extern "C" int leankv_window_pool_append(const leankv_window_pool_t* a, const float* qkv, int ld, const float* bias,
+                                         void* q, int rows, int start, void* stream) {
+    const int rc = check_args(a);
+    if (rc) return rc;
+    if (!qkv || !q || rows <= 0 || start < 0 || ld < (a->heads + a->kv_heads) * a->dim + a->kv_heads * a->vdim)
+        return LEANKV_EINVAL;
+    if (rows + std::max(a->size, a->pool) - 1 > a->ring) return LEANKV_ELIMIT;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    return a->dtype == LEANKV_DT_BF16 ? append<bf16>(*a, qkv, ld, bias, q, rows, start, st)
+                                      : append<float>(*a, qkv, ld, bias, q, rows, start, st);
+}
+
+extern "C" size_t leankv_window_pool_workspace_bytes(const leankv_window_pool_t* a, int rows, int max_pos) {
+    if (check_args(a) || rows <= 0 || max_pos <= 0) return 0;
+    const AttendPlan pl(*a, kAttendThreads, max_keys(*a, max_pos), kAttendSmemFloats);
+    return pl.p_in_smem ? 0 : (size_t)rows * 2 * a->heads * pl.ldp * 4;
+}
+
+extern "C" int leankv_window_pool_attend(const leankv_window_pool_t* a, const void* q, void* out, int out_ld,
+                                         float out_scale, int rows, int start, void* ws, size_t ws_bytes,
+                                         void* stream) {
+    const int rc = check_args(a);
+    if (rc) return rc;
+    if (!q || !out || rows <= 0 || start < 0 || out_ld < a->heads * a->vdim) return LEANKV_EINVAL;
+    if (VisibleKeys(start + rows - 1, a->size, a->pool).n_blk > a->max_blocks) return LEANKV_ELIMIT;
+    if (leankv_window_pool_workspace_bytes(a, rows, start + rows) > (ws ? ws_bytes : 0)) return LEANKV_EWORKSPACE;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    float* w = static_cast<float*>(ws);
+    return a->dtype == LEANKV_DT_BF16 ? attend<bf16>(*a, q, out, out_ld, out_scale, rows, start, w, st)
+                                      : attend<float>(*a, q, out, out_ld, out_scale, rows, start, w, st);
+}

@@ -33,6 +33,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _native
+from .decode_loop import DecodeLoop
 from .teal.sparse_fns import compute_threshold_for_sparsity
 from .turboquant.codebook import get_codebook_tensors
 from .turboquant.rotation import generate_rotation_matrix
@@ -86,7 +87,7 @@ def _rope(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor
     return x * cos + rot * sin
 
 
-class DecodeEngine:
+class DecodeEngine(DecodeLoop):
     """Owns the (sharded) weights in kernel layout, the paged 3-bit KV pool and the step graph."""
 
     def __init__(self, cfg: DecoderConfig, weights: dict, device, max_seq_len: int = 1024,
@@ -104,7 +105,7 @@ class DecodeEngine:
         self.nkv = cfg.num_kv_heads // tp_size
         self.inter = cfg.intermediate_size // tp_size
         self.n_qkv = (self.nq + 2 * self.nkv) * 128
-        self.max_seq_len = max_seq_len
+        self._init_loop(max_seq_len)
         self.max_pages = (max_seq_len + PAGE - 1) // PAGE
         L, dev = cfg.num_layers, self.dev
 
@@ -135,10 +136,6 @@ class DecodeEngine:
         self.fused_norm = True   # False: RMSNorm + residual add as launches of their own
         self.mlp_h, self.down = half(self.inter), half(cfg.hidden_size)
         self.logits = half(cfg.vocab_size)
-        self.token = torch.zeros(1, dtype=torch.int64, device=dev)
-        self.history_cap = max_seq_len + 8
-        self.history = torch.zeros(self.history_cap, dtype=torch.int64, device=dev)
-        self.state = torch.zeros(8, dtype=torch.int32, device=dev)
         self.active_elems = torch.zeros(1, dtype=torch.int64, device=dev)
         self.inv_freq = (1.0 / (cfg.rope_theta ** (torch.arange(0, 128, 2, dtype=torch.int64).float() / 128))
                          ).to(dev).contiguous()
@@ -168,10 +165,6 @@ class DecodeEngine:
             self.vocab_local, self.vocab_offset = vl, tp_rank * vl
             self.lm_head_local = self.w["lm_head_t"][:, self.vocab_offset:self.vocab_offset + vl].contiguous()
         self.set_thresholds(thresholds)
-        self.graph = None
-        self.launches_per_step = 0
-        self._pinned_token = torch.zeros(1, dtype=torch.int64).pin_memory() if torch.cuda.is_available() else None
-        self._pinned_status = torch.zeros(2, dtype=torch.int32).pin_memory() if torch.cuda.is_available() else None
 
     # ── construction helpers ─────────────────────────────────────────────
 
@@ -288,9 +281,6 @@ class DecodeEngine:
         return segs
 
     # ── kernel launches (all on the current stream) ──────────────────────
-
-    def _st(self) -> int:
-        return torch.cuda.current_stream().cuda_stream
 
     def _gemv(self, wt, x, y, t, segs=None, residual=None, norm_w=None):
         """y = [residual +] Wt^T . mask_t(x); with ``norm_w`` the kernel first applies RMSNorm(x; norm_w)."""
@@ -467,30 +457,14 @@ class DecodeEngine:
                                             self.history.data_ptr(), self.history_cap, sp, st()), "decode_end")
         self.launches_per_step += 1
 
-    def capture(self) -> None:
-        """Capture one decode step into a CUDA graph (a throw-away eager step warms everything up first)."""
-        with torch.cuda.device(self.dev):
-            snap = (self.state.clone(), self.token.clone(), self.history.clone(),
-                    [p.clone() for p in self.pools], self.active_elems.clone())
-            side = torch.cuda.Stream()
-            side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):
-                self._step_launches()
-            torch.cuda.current_stream().wait_stream(side)
+    def _step_state(self) -> list:
+        return [self.state, self.token, self.history, *self.pools, self.active_elems]
+
+    def _capture_barrier(self) -> None:
+        if self.tp_size > 1:
+            # the in-kernel exchange waits a bounded time for its peers: start the replays together
             torch.cuda.synchronize()
-            self.state.copy_(snap[0]); self.token.copy_(snap[1]); self.history.copy_(snap[2])
-            for p, s in zip(self.pools, snap[3]):
-                p.copy_(s)
-            self.active_elems.copy_(snap[4])
-            self.graph = torch.cuda.CUDAGraph()
-            # thread_local: the NCCL watchdog thread (tensor parallel runs) may touch CUDA while we capture
-            with torch.cuda.graph(self.graph, capture_error_mode="thread_local"):
-                self._step_launches()
-            # capture does not execute; state is unchanged
-            if self.tp_size > 1:
-                # the in-kernel exchange waits a bounded time for its peers: start the replays together
-                torch.cuda.synchronize()
-                torch.distributed.barrier(group=self.group)
+            torch.distributed.barrier(group=self.group)
 
     def full_logits(self) -> torch.Tensor:
         """Logits of the last decode step over the whole vocabulary (fp16 [vocab]). With the output head
@@ -521,14 +495,10 @@ class DecodeEngine:
                                f"(1 = a peer's partial sum never arrived), attention status {at} "
                                f"(1 = page copy wait gave up, 2 = page id out of range)")
 
-    def step(self, use_graph: bool = True) -> None:
-        if use_graph:
-            if self.graph is None:
-                self.capture()
-            self.graph.replay()
-        else:
-            with torch.cuda.device(self.dev):
-                self._step_launches()
+    def _queue_status(self) -> None:
+        self._pinned_status[0:1].copy_(self.ws_attn[:4].view(torch.int32), non_blocking=True)
+        if self.xchg is not None:
+            self._pinned_status[1:2].copy_(self.xchg.status, non_blocking=True)
 
     # ── prefill ──────────────────────────────────────────────────────────
 
@@ -749,33 +719,6 @@ class DecodeEngine:
             self.state[0], self.state[1] = T, 1
             self.prefill_logits = logits
         return int(tok.item())
-
-    @torch.no_grad()
-    def generate(self, prompt_ids, max_new_tokens: int, stream_to_host: bool = True) -> list[int]:
-        """Greedy generation. With ``stream_to_host`` every token is copied to pinned host memory and
-        waited for before the next step is launched (what an interactive caller sees); without it the
-        steps are enqueued back to back and the tokens are read once at the end."""
-        first = self.prefill(prompt_ids)
-        n_steps = min(max_new_tokens - 1, self.max_seq_len - len(prompt_ids) - 1)
-        out = [first]
-        with torch.cuda.device(self.dev):
-            if self.graph is None:
-                self.capture()
-            for _ in range(max(n_steps, 0)):
-                self.graph.replay()
-                if stream_to_host:
-                    self._pinned_token.copy_(self.token, non_blocking=True)
-                    self._pinned_status[0:1].copy_(self.ws_attn[:4].view(torch.int32), non_blocking=True)
-                    if self.xchg is not None:
-                        self._pinned_status[1:2].copy_(self.xchg.status, non_blocking=True)
-                    torch.cuda.current_stream().synchronize()
-                    if int(self._pinned_status[0]) or int(self._pinned_status[1]):
-                        self.check_status()
-                    out.append(int(self._pinned_token[0]))
-            if not stream_to_host:
-                out = self.history[:1 + max(n_steps, 0)].tolist()
-            self.check_status()
-        return out
 
     def bytes_streamed(self) -> int:
         """Weight bytes the sparse GEMVs have streamed since the counter was last zeroed."""
