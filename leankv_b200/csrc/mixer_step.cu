@@ -12,60 +12,61 @@ namespace leankv {
 namespace {
 
 constexpr int kStepThreads = 512;
-constexpr int kStepCluster = 8;
+constexpr int kMaxCluster = 16;     // non-portable; 8 where the device does not place 16
 constexpr int kStepSmemFloats = 200 * 1024 / 4;
 
 struct StepParams {
     leankv_window_pool_t left;
     leankv_time_mix_t right;
     leankv_mixer_step_t s;
-    int has_left, has_right, n_max;
+    int has_left, has_right, n_max, cluster;
 };
 
 template <typename T>
 __device__ void left_step(const StepParams& p, float* sm, float* s_tmp, int rank) {
     const leankv_window_pool_t& a = p.left;
-    const AttendPlan pl(a, kStepThreads, (p.n_max + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
+    const AttendPlan pl(a, kStepThreads, (p.n_max + p.cluster - 1) / p.cluster, kStepSmemFloats);
     const int tid = threadIdx.x, i = p.s.state[kPos], G = a.kv_heads;
     const int nq = a.heads * a.dim, nk = G * a.dim;
     const float* y = p.s.y + p.s.qkv_off;       // biases are already in
-    const float fq = row_factor(y, nullptr, nq, a.q_norm != nullptr, a.eps, s_tmp);
-    const float fk = row_factor(y + nq, nullptr, nk, a.k_norm != nullptr, a.eps, s_tmp);
+    const RowFactors f = row_factors(y, nullptr, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
     for (int e = tid; e < a.heads * a.dim_pad; e += kStepThreads) {
         const int h = e / a.dim_pad, d = e - h * a.dim_pad, x = h * a.dim + d;
-        sm[pl.q + e] = d < a.dim ? y[x] * fq * (a.q_norm ? __ldg(a.q_norm + x) : 1.f) * a.scale : 0.f;
+        put_query<T>(pl, sm, a.heads, h, d, d < a.dim ? y[x] * f.q * (a.q_norm ? __ldg(a.q_norm + x) : 1.f) * a.scale : 0.f);
     }
     const int slot = i % a.ring;
     T* k_ring = static_cast<T*>(a.k_ring);
     T* v_ring = static_cast<T*>(a.v_ring);
+    T* k_new = reinterpret_cast<T*>(sm + pl.knew);
+    T* v_new = reinterpret_cast<T*>(sm + pl.vnew);
     for (int e = tid; e < G * a.dim_pad; e += kStepThreads) {
         const int g = e / a.dim_pad, d = e - g * a.dim_pad, x = g * a.dim + d;
-        const T v = from_f32<T>(d < a.dim ? y[nq + x] * fk * (a.k_norm ? __ldg(a.k_norm + x) : 1.f) : 0.f);
-        sm[pl.knew + e] = to_f32(v);
+        const T v = from_f32<T>(d < a.dim ? y[nq + x] * f.k * (a.k_norm ? __ldg(a.k_norm + x) : 1.f) : 0.f);
+        k_new[e] = v;
         if (rank == 0) k_ring[(size_t)slot * G * a.dim_pad + e] = v;
     }
     for (int e = tid; e < G * a.vdim_pad; e += kStepThreads) {
         const int g = e / a.vdim_pad, d = e - g * a.vdim_pad;
         const T v = from_f32<T>(d < a.vdim ? y[nq + nk + g * a.vdim + d] : 0.f);
-        sm[pl.vnew + e] = to_f32(v);
+        v_new[e] = v;
         if (rank == 0) v_ring[(size_t)slot * G * a.vdim_pad + e] = v;
     }
     __syncthreads();
     float* p_gmem = static_cast<float*>(p.s.ws) + (size_t)rank * 2 * a.heads * pl.ldp;
-    attend_query<T, float>(a, pl, sm, p_gmem, i, true, rank, kStepCluster, p.s.out, p.s.left_scale);
+    attend_query<T, float>(a, pl, sm, p_gmem, i, true, rank, p.cluster, p.s.out, p.s.left_scale);
 
     // the block this token completes (not visible to it: it ends at i > i - size)
     if ((i + 1) % a.pool == 0 && (i + 1) / a.pool <= a.max_blocks) {
         const int b = i / a.pool, p0 = b * a.pool;
-        auto mean = [&](const T* ring, const float* fresh, T* dst, int n) {
-            for (int e = rank * kStepThreads + tid; e < n; e += kStepCluster * kStepThreads) {
+        auto mean = [&](const T* ring, const T* fresh, T* dst, int n) {
+            for (int e = rank * kStepThreads + tid; e < n; e += p.cluster * kStepThreads) {
                 float t = 0.f;
                 for (int x = 0; x < a.pool - 1; ++x) t += to_f32(ring[(size_t)((p0 + x) % a.ring) * n + e]);
-                dst[(size_t)b * n + e] = from_f32<T>((t + fresh[e]) / (float)a.pool);
+                dst[(size_t)b * n + e] = from_f32<T>((t + to_f32(fresh[e])) / (float)a.pool);
             }
         };
-        mean(k_ring, sm + pl.knew, static_cast<T*>(a.k_pool), G * a.dim_pad);
-        mean(v_ring, sm + pl.vnew, static_cast<T*>(a.v_pool), G * a.vdim_pad);
+        mean(k_ring, k_new, static_cast<T*>(a.k_pool), G * a.dim_pad);
+        mean(v_ring, v_new, static_cast<T*>(a.v_pool), G * a.vdim_pad);
     }
 }
 
@@ -128,7 +129,7 @@ __global__ void __launch_bounds__(kStepThreads) mixer_step_kernel(const __grid_c
     extern __shared__ __align__(16) float sm[];
     __shared__ float s_tmp[32];
     pdl_begin();
-    const int first = p.has_left ? kStepCluster : 0;
+    const int first = p.has_left ? p.cluster : 0;
     if ((int)blockIdx.x < first) left_step<T>(p, sm, s_tmp, blockIdx.x);
     else if ((int)blockIdx.x - first < p.right.heads) right_step<T>(p, sm, s_tmp, blockIdx.x - first);
 }
@@ -138,23 +139,44 @@ int keys_bound(const leankv_window_pool_t& a, int max_pos) {
 }
 
 template <typename T>
-int launch_step(const StepParams& p, cudaStream_t st) {
+size_t step_smem(const StepParams& p) {
     size_t smem = 0;
-    int grid = 0;
-    if (p.has_left) {
-        const AttendPlan pl(p.left, kStepThreads, (p.n_max + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
-        smem = (size_t)pl.total * 4;
-        grid = kStepCluster;
+    if (p.has_left)
+        smem = 4 * (size_t)AttendPlan(p.left, kStepThreads, (p.n_max + p.cluster - 1) / p.cluster, kStepSmemFloats).total;
+    if (p.has_right) smem = std::max(smem, (size_t)(4 * p.right.dim + kStepThreads + p.right.dim) * 4);
+    return smem;
+}
+
+template <typename T>
+int launch_step(StepParams& p, cudaStream_t st) {
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(mixer_step_kernel<T>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+    for (p.cluster = kMaxCluster;; p.cluster = 8) {
+        const size_t smem = step_smem<T>(p);
+        if (smem > 226 * 1024) return LEANKV_ELIMIT;
+        LEANKV_CUDA_TRY(cudaFuncSetAttribute(mixer_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        const int heads = p.has_right ? p.right.heads : 0;
+        const int grid = (p.has_left ? p.cluster : 0) + (heads + p.cluster - 1) / p.cluster * p.cluster;
+        if (p.cluster > 8) {      // does a cluster of this size fit this device?
+            cudaLaunchConfig_t cfg = {};
+            cfg.gridDim = dim3(grid);
+            cfg.blockDim = dim3(kStepThreads);
+            cfg.dynamicSmemBytes = smem;
+            cudaLaunchAttribute attr[1];
+            attr[0].id = cudaLaunchAttributeClusterDimension;
+            attr[0].val.clusterDim.x = p.cluster;
+            attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+            cfg.attrs = attr;
+            cfg.numAttrs = 1;
+            int fits = 0;
+            if (cudaOccupancyMaxActiveClusters(&fits, mixer_step_kernel<T>, &cfg) != cudaSuccess || fits < 1) {
+                (void)cudaGetLastError();
+                continue;
+            }
+        }
+        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(false, dim3(p.cluster), mixer_step_kernel<T>, dim3(grid),
+                                                 dim3(kStepThreads), smem, st, p));
+        return LEANKV_OK;
     }
-    if (p.has_right) {
-        smem = std::max(smem, (size_t)(4 * p.right.dim + kStepThreads + p.right.dim) * 4);
-        grid += (p.right.heads + kStepCluster - 1) / kStepCluster * kStepCluster;
-    }
-    if (smem > 226 * 1024) return LEANKV_ELIMIT;
-    LEANKV_CUDA_TRY(cudaFuncSetAttribute(mixer_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    LEANKV_CUDA_TRY(launch_cluster_kernel_ex(false, dim3(kStepCluster), mixer_step_kernel<T>, dim3(grid),
-                                             dim3(kStepThreads), smem, st, p));
-    return LEANKV_OK;
 }
 
 }  // namespace
@@ -165,8 +187,12 @@ using namespace leankv;
 extern "C" size_t leankv_mixer_step_workspace_bytes(const leankv_window_pool_t* left, int max_pos) {
     if (!left || max_pos <= 0) return 0;
     const int n = keys_bound(*left, max_pos);
-    const AttendPlan pl(*left, kStepThreads, (n + kStepCluster - 1) / kStepCluster, kStepSmemFloats);
-    return pl.p_in_smem ? 0 : (size_t)kStepCluster * 2 * left->heads * pl.ldp * 4;
+    size_t need = 0;
+    for (int c = 8; c <= kMaxCluster; c *= 2) {
+        const AttendPlan pl(*left, kStepThreads, (n + c - 1) / c, kStepSmemFloats);
+        if (!pl.p_in_smem) need = std::max(need, (size_t)c * 2 * left->heads * pl.ldp * 4);
+    }
+    return need;
 }
 
 extern "C" int leankv_mixer_step(const leankv_window_pool_t* left, const leankv_time_mix_t* right,

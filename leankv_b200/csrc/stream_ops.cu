@@ -53,6 +53,97 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const leankv_s
     }
 }
 
+// The same with 4-element accesses and rows in registers (width % 4 == 0, width <= kRowThreads * 4 * NV). A CTA
+// walks `per_cta` consecutive rows and keeps the row above, so only its first row is normed twice.
+template <typename T>
+__device__ __forceinline__ void store4(T* p, const float (&v)[4]) {
+    if constexpr (sizeof(T) == 4)
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else
+        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+}
+__device__ __forceinline__ void fetch4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void fetch4(const bf16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(a.x << 16); v[1] = __uint_as_float(a.x & 0xffff0000u);
+    v[2] = __uint_as_float(a.y << 16); v[3] = __uint_as_float(a.y & 0xffff0000u);
+}
+
+template <typename T, typename D, int NV>
+__global__ void __launch_bounds__(kRowThreads) stream_norm_vec_kernel(const leankv_stream_norm_t a, int per_cta) {
+    __shared__ float s_tmp[32];
+    pdl_begin();
+    const int W = a.width, r0 = blockIdx.x * per_cta, r1 = min(a.rows, r0 + per_cta), tid = threadIdx.x;
+    const D* delta = static_cast<const D*>(a.delta);
+    T* h = static_cast<T*>(a.h);
+    T* mixed = static_cast<T*>(a.mixed);
+    const bool shift = a.n_mix > 0;
+    const float gain = __ldg(a.gain);
+    float cur[NV][4], above[NV][4];
+    auto load = [&](int row, bool store) -> float {       // the updated stream of `row` into cur; its norm factor
+        float ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (tid + n * kRowThreads) * 4;
+            if (i < W) {
+                fetch4(a.x_in + (size_t)row * W + i, cur[n]);
+                if (delta != nullptr) {
+                    float dv[4], sv[4];
+                    fetch4(delta + (size_t)row * W + i, dv);
+                    fetch4(a.scale + i, sv);
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) cur[n][q] = fmaf(dv[q], sv[q], cur[n][q]);
+                    if (store) store4(a.x_out + (size_t)row * W + i, cur[n]);
+                }
+#pragma unroll
+                for (int q = 0; q < 4; ++q) ss = fmaf(cur[n][q], cur[n][q], ss);
+            }
+        }
+        return gain / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+    };
+    if (shift) {
+        if (r0 > 0) {
+            const float rs = load(r0 - 1, false);
+#pragma unroll
+            for (int n = 0; n < NV; ++n)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) above[n][q] = cur[n][q] * rs;
+        } else {
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int i = (tid + n * kRowThreads) * 4;
+                if (i < W) fetch4(a.prev_in + i, above[n]);
+            }
+        }
+    }
+    for (int row = r0; row < r1; ++row) {
+        const float rs = load(row, true);
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (tid + n * kRowThreads) * 4;
+            if (i >= W) continue;
+#pragma unroll
+            for (int q = 0; q < 4; ++q) cur[n][q] *= rs;
+            if (h != nullptr) store4(h + (size_t)row * W + i, cur[n]);
+            if (shift) {
+                for (int m = 0; m < a.n_mix; ++m) {
+                    float mv[4];
+                    fetch4(a.mu[m] + i, mv);
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) mv[q] = fmaf(above[n][q] - cur[n][q], mv[q], cur[n][q]);
+                    store4(mixed + ((size_t)m * a.rows + row) * W + i, mv);
+                }
+#pragma unroll
+                for (int q = 0; q < 4; ++q) above[n][q] = cur[n][q];
+                if (row == a.rows - 1) store4(a.prev_out + i, cur[n]);
+            }
+        }
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) silu_mul_rows_kernel(const T* gate_up, T* out, int inter, long long total) {
     pdl_begin();
@@ -106,7 +197,21 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float* in, T* out
 
 template <typename T, typename D>
 int launch_stream_norm(const leankv_stream_norm_t* a, cudaStream_t st) {
-    LEANKV_CUDA_TRY(launch_kernel(stream_norm_kernel<T, D>, dim3(a->rows), dim3(kRowThreads), 0, st, *a));
+    bool vec = a->width % 4 == 0 && a->width <= kRowThreads * 4 * 8 && aligned16(a->x_in) && aligned16(a->x_out) &&
+               aligned16(a->delta) && aligned16(a->scale) && aligned16(a->h) && aligned16(a->mixed) &&
+               aligned16(a->prev_in) && aligned16(a->prev_out);
+    for (int i = 0; i < a->n_mix; ++i) vec = vec && aligned16(a->mu[i]);
+    if (!vec) {
+        LEANKV_CUDA_TRY(launch_kernel(stream_norm_kernel<T, D>, dim3(a->rows), dim3(kRowThreads), 0, st, *a));
+        return LEANKV_OK;
+    }
+    const int per = a->n_mix > 0 && a->rows >= sm_count() * 8 ? 4 : 1;
+    const dim3 grid((a->rows + per - 1) / per), block(kRowThreads);
+    const int nv = (a->width + kRowThreads * 4 - 1) / (kRowThreads * 4);
+    if (nv <= 1) LEANKV_CUDA_TRY(launch_kernel(stream_norm_vec_kernel<T, D, 1>, grid, block, 0, st, *a, per));
+    else if (nv <= 2) LEANKV_CUDA_TRY(launch_kernel(stream_norm_vec_kernel<T, D, 2>, grid, block, 0, st, *a, per));
+    else if (nv <= 4) LEANKV_CUDA_TRY(launch_kernel(stream_norm_vec_kernel<T, D, 4>, grid, block, 0, st, *a, per));
+    else LEANKV_CUDA_TRY(launch_kernel(stream_norm_vec_kernel<T, D, 8>, grid, block, 0, st, *a, per));
     return LEANKV_OK;
 }
 

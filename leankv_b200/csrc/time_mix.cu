@@ -11,9 +11,18 @@
 namespace leankv {
 namespace {
 
-constexpr int kCols = 32;        // value columns per CTA
-constexpr int kSlices = 4;       // lanes that share a column, each with a quarter of the key channels
+constexpr int kSlices = 8;       // lanes that share a column group, each with an eighth of the key channels
+constexpr int kColGroup = 4;     // value columns per thread: one read of r / k / w serves four columns
 constexpr int kMinPiece = 64;
+
+// L: key channels per slice (a power of two from 4), kSlices * L >= dim.
+template <int L>
+struct ScanShape {
+    static constexpr int kCols = L == 4 ? 32 : 64;                   // value columns per CTA
+    static constexpr int kThreads = kCols / kColGroup * kSlices;
+    static constexpr int kTok = kThreads / L;                        // tokens staged at a time: 8 channels per thread
+    static constexpr int kRow = kSlices * (L + 4);                   // staged row; slices start in different banks
+};
 
 template <typename T>
 struct ScanParams {
@@ -30,123 +39,162 @@ struct ScanParams {
     int heads, dim, rows, piece, n_pieces;
 };
 
-// L: key channels per slice, a multiple of 4, kSlices * L >= dim.
+// Eight consecutive channels of one token, zero beyond `n`.
+template <typename T>
+__device__ __forceinline__ void fetch8(const T* p, int n, bool vec, float (&v)[8]) {
+    if (vec && n >= 8) {
+        Raw8<T> r;
+        load8(p, r);
+        unpack8(r, v);
+    } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = i < n ? to_f32(p[i]) : 0.f;
+    }
+}
+
 template <typename T, int L, bool OUT>
-__global__ void __launch_bounds__(kCols * kSlices) time_mix_scan_kernel(const ScanParams<T> p) {
-    constexpr int kStride = kSlices * (L + 4);       // slices start in different banks
-    constexpr int kTok = L > 32 ? 8 : 16;            // tokens staged in shared memory at a time
-    __shared__ __align__(16) float s_r[kTok][OUT ? kStride : 4], s_k[kTok][kStride], s_w[kTok][kStride];
-    __shared__ float s_v[kTok][kCols], s_bonus[kTok];
+__global__ void __launch_bounds__(ScanShape<L>::kThreads) time_mix_scan_kernel(const ScanParams<T> p, bool vec) {
+    using Sh = ScanShape<L>;
+    constexpr int kTok = Sh::kTok, kCols = Sh::kCols, kRow = Sh::kRow;
+    __shared__ __align__(16) float s_r[OUT ? kTok : 1][kRow], s_k[kTok][kRow], s_w[kTok][kRow];
+    __shared__ __align__(16) float s_v[kTok][kCols], s_bonus[kTok];
     pdl_begin();
-    const int tid = threadIdx.x, slice = tid & (kSlices - 1), col = tid >> 2;
+    const int tid = threadIdx.x, slice = tid & (kSlices - 1), cg = tid / kSlices;
     const int head = blockIdx.x, c0 = blockIdx.y * kCols, piece = blockIdx.z, d = p.dim;
     const int t0 = piece * p.piece, t1 = min(p.rows, t0 + p.piece);
-    const int N = p.heads * d;
-    const bool live = c0 + col < d;
+    const int N = p.heads * d, col0 = c0 + cg * kColGroup;
     const size_t state = (size_t)d * d;
-    float S[L];
-#pragma unroll
-    for (int i = 0; i < L; ++i) S[i] = 0.f;
-    if (OUT && live) {
-        const float* src = p.S_in + ((size_t)piece * p.heads + head) * state + c0 + col;
-#pragma unroll
-        for (int i = 0; i < L; ++i) {
-            const int k = slice * L + i;
-            if (k < d) S[i] = src[(size_t)k * d];
-        }
-    }
-    float prod[(kSlices * L + kCols * kSlices - 1) / (kCols * kSlices)];
-#pragma unroll
-    for (auto& x : prod) x = 1.f;
 
+    float S[L][kColGroup];
+#pragma unroll
+    for (int i = 0; i < L; ++i)
+#pragma unroll
+        for (int c = 0; c < kColGroup; ++c) {
+            const int k = slice * L + i;
+            S[i][c] = OUT && k < d && col0 + c < d
+                          ? p.S_in[((size_t)piece * p.heads + head) * state + (size_t)k * d + col0 + c] : 0.f;
+        }
+
+    // this thread's share of the staging: channels k8 .. k8 + 7 (and columns, for v) of token st_t
+    const int st_t = tid / L, k8 = tid % L * 8, nk = d - k8;
+    const int v_t = tid / (kCols / 8), v8 = tid % (kCols / 8) * 8;
+    float w0[8], u[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        w0[i] = i < nk ? __ldg(p.w0 + head * d + k8 + i) : 0.f;
+        u[i] = OUT && i < nk ? __ldg(p.u + head * d + k8 + i) : 0.f;
+    }
+    float rr[8], kk[8], zz[8], vv[8], esum[8] = {};
+    auto fetch = [&](int tb) {
+        const bool on = tb + st_t < t1;
+        const size_t g = (size_t)(tb + st_t) * N + head * d + k8;
+        fetch8(p.k + g, on ? nk : 0, vec, kk);
+        fetch8(p.z + g, on ? nk : 0, vec, zz);
+        if (OUT) fetch8(p.r + g, on ? nk : 0, vec, rr);
+        if (v_t < kTok)
+            fetch8(p.v + (size_t)(tb + v_t) * N + head * d + c0 + v8, tb + v_t < t1 ? d - c0 - v8 : 0, vec, vv);
+    };
+    fetch(t0);
     for (int tb = t0; tb < t1; tb += kTok) {
         const int nt = min(kTok, t1 - tb);
         __syncthreads();
-        for (int e = tid; e < kTok * kSlices * L; e += kCols * kSlices) {
-            const int t = e / (kSlices * L), k = e - t * (kSlices * L);
-            const int at = k / L * (L + 4) + k % L;
-            float rv = 0.f, kv = 0.f, wv = 1.f;
-            if (t < nt && k < d) {
-                const size_t g = (size_t)(tb + t) * N + head * d + k;
-                kv = to_f32(p.k[g]);
-                wv = expf(-expf(p.z[g] + __ldg(p.w0 + head * d + k)));
-                if (OUT) rv = to_f32(p.r[g]);
+        float bonus = 0.f;
+#pragma unroll
+        for (int h = 0; h < 8; h += 4) {
+            const int k = k8 + h, at = k / L * (L + 4) + k % L;
+            float w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const bool on = st_t < nt && h + i < nk;
+                const float e = on ? expf(zz[h + i] + w0[h + i]) : 0.f;      // -log of the decay
+                w[i] = expf(-e);
+                if (!OUT) esum[h + i] += e;
+                else bonus = fmaf(rr[h + i] * u[h + i], kk[h + i], bonus);
             }
-            s_k[t][at] = kv;
-            s_w[t][at] = wv;
-            if (OUT) s_r[t][at] = rv;
+            if (k < kSlices * L) {
+                *reinterpret_cast<float4*>(&s_k[st_t][at]) = make_float4(kk[h], kk[h + 1], kk[h + 2], kk[h + 3]);
+                *reinterpret_cast<float4*>(&s_w[st_t][at]) = make_float4(w[0], w[1], w[2], w[3]);
+                if (OUT) *reinterpret_cast<float4*>(&s_r[st_t][at]) = make_float4(rr[h], rr[h + 1], rr[h + 2], rr[h + 3]);
+            }
         }
-        for (int e = tid; e < kTok * kCols; e += kCols * kSlices) {
-            const int t = e / kCols, c = e - t * kCols;
-            s_v[t][c] = t < nt && c0 + c < d ? to_f32(p.v[(size_t)(tb + t) * N + head * d + c0 + c]) : 0.f;
+        if (v_t < kTok) {
+            *reinterpret_cast<float4*>(&s_v[v_t][v8]) = make_float4(vv[0], vv[1], vv[2], vv[3]);
+            *reinterpret_cast<float4*>(&s_v[v_t][v8 + 4]) = make_float4(vv[4], vv[5], vv[6], vv[7]);
+        }
+        if (OUT) {      // bonus_t = sum over k of r u k: the L threads of a token are neighbours
+#pragma unroll
+            for (int o = L / 2; o > 0; o >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, o);
+            if (tid % L == 0) s_bonus[st_t] = bonus;
         }
         __syncthreads();
-        if (OUT) {      // bonus_t = sum over k of r u k: 8 threads per token
-            const int t = tid >> 3, part = tid & 7;
-            float b = 0.f;
-            for (int k = part; k < d && t < kTok; k += 8) {
-                const int at = k / L * (L + 4) + k % L;
-                b = fmaf(s_r[t][at] * __ldg(p.u + head * d + k), s_k[t][at], b);
-            }
+        if (tb + kTok < t1) fetch(tb + kTok);       // the next tokens travel while these are consumed
+#pragma unroll 1
+        for (int tq = 0; tq < nt; tq += 2) {        // a token beyond nt has k = 0 and w = 1: no effect
+            float acc[2 * kColGroup];
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1) b += __shfl_xor_sync(0xffffffffu, b, o);
-            if (part == 0 && t < kTok) s_bonus[t] = b;
-            __syncthreads();
-        } else if (blockIdx.y == 0) {
-            int x = 0;
-            for (int k = tid; k < kSlices * L; k += kCols * kSlices, ++x) {
-                const int at = k / L * (L + 4) + k % L;
-                float q = 1.f;
-                for (int t = 0; t < nt; ++t) q *= s_w[t][at];
-                prod[x] *= q;
-            }
-        }
-        for (int tq = 0; tq < nt; tq += 4) {
-            float acc[4];
-#pragma unroll
-            for (int tt = 0; tt < 4; ++tt) {           // tokens beyond nt: k = 0, w = 1, no effect
+            for (int tt = 0; tt < 2; ++tt) {
                 const int t = tq + tt;
-                const float vv = s_v[t][col];
-                float a = 0.f;
+                const float4 v4 = *reinterpret_cast<const float4*>(&s_v[t][cg * kColGroup]);
+                const float v[kColGroup] = {v4.x, v4.y, v4.z, v4.w};
+                float a[kColGroup] = {};
 #pragma unroll
                 for (int i = 0; i < L; i += 4) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[t][slice * (L + 4) + i]);
-                    const float4 w4 = *reinterpret_cast<const float4*>(&s_w[t][slice * (L + 4) + i]);
+                    const int at = slice * (L + 4) + i;
+                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[t][at]);
+                    const float4 w4 = *reinterpret_cast<const float4*>(&s_w[t][at]);
+                    const float ka[4] = {k4.x, k4.y, k4.z, k4.w}, wa[4] = {w4.x, w4.y, w4.z, w4.w};
+                    float ra[4] = {};
                     if (OUT) {
-                        const float4 r4 = *reinterpret_cast<const float4*>(&s_r[t][slice * (L + 4) + i]);
-                        a = fmaf(r4.x, S[i], a); a = fmaf(r4.y, S[i + 1], a);
-                        a = fmaf(r4.z, S[i + 2], a); a = fmaf(r4.w, S[i + 3], a);
+                        const float4 r4 = *reinterpret_cast<const float4*>(&s_r[t][at]);
+                        ra[0] = r4.x; ra[1] = r4.y; ra[2] = r4.z; ra[3] = r4.w;
                     }
-                    S[i] = fmaf(w4.x, S[i], k4.x * vv);
-                    S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * vv);
-                    S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * vv);
-                    S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * vv);
-                }
-                acc[tt] = a;
-            }
-            if (OUT) {      // sum over the four slices; lane `slice` keeps token tq + slice
-                const bool hi2 = slice & 2, hi1 = slice & 1;
-                const float a0 = (hi2 ? acc[2] : acc[0]) + __shfl_xor_sync(0xffffffffu, hi2 ? acc[0] : acc[2], 2);
-                const float a1 = (hi2 ? acc[3] : acc[1]) + __shfl_xor_sync(0xffffffffu, hi2 ? acc[1] : acc[3], 2);
-                const float r = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 1);
-                const int t = tq + slice;
-                if (live && t < nt)
-                    p.o[(size_t)(tb + t) * N + head * d + c0 + col] = fmaf(s_bonus[t], s_v[t][col], r);
-            }
-        }
-    }
-    if (live && (!OUT || piece == p.n_pieces - 1)) {
-        float* dst = p.S_out + ((size_t)(OUT ? 0 : piece) * p.heads + head) * state + c0 + col;
 #pragma unroll
-        for (int i = 0; i < L; ++i) {
-            const int k = slice * L + i;
-            if (k < d) dst[(size_t)k * d] = S[i];
+                    for (int x = 0; x < 4; ++x)
+#pragma unroll
+                        for (int c = 0; c < kColGroup; ++c) {
+                            if (OUT) a[c] = fmaf(ra[x], S[i + x][c], a[c]);
+                            S[i + x][c] = fmaf(wa[x], S[i + x][c], ka[x] * v[c]);
+                        }
+                }
+#pragma unroll
+                for (int c = 0; c < kColGroup; ++c) acc[tt * kColGroup + c] = a[c];
+            }
+            if (OUT) {      // sum over the eight slices; lane `slice` ends with (token, column) number `slice`
+#pragma unroll
+                for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+                    for (int i = 0; i < o; ++i) {
+                        const bool up = (slice & o) != 0;
+                        const float send = up ? acc[i] : acc[i + o], keep = up ? acc[i + o] : acc[i];
+                        acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                    }
+                const int t = tq + slice / kColGroup, c = slice % kColGroup;
+                if (t < nt && col0 + c < d)
+                    p.o[(size_t)(tb + t) * N + head * d + col0 + c] = fmaf(s_bonus[t], s_v[t][cg * kColGroup + c], acc[0]);
+            }
         }
     }
-    if (!OUT && blockIdx.y == 0) {
-        int x = 0;
-        for (int k = tid; k < kSlices * L; k += kCols * kSlices, ++x)
-            if (k < d) p.decay[((size_t)piece * p.heads + head) * d + k] = prod[x];
+    if (!OUT || piece == p.n_pieces - 1) {
+        float* dst = p.S_out + ((size_t)(OUT ? 0 : piece) * p.heads + head) * state;
+#pragma unroll
+        for (int i = 0; i < L; ++i)
+#pragma unroll
+            for (int c = 0; c < kColGroup; ++c) {
+                const int k = slice * L + i;
+                if (k < d && col0 + c < d) dst[(size_t)k * d + col0 + c] = S[i][c];
+            }
+    }
+    if (!OUT && blockIdx.y == 0) {      // decay of the whole piece: exp(-sum over its tokens)
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (k8 + i < kRow) s_k[st_t][k8 + i] = esum[i];
+        __syncthreads();
+        for (int k = tid; k < d; k += Sh::kThreads) {
+            float e = 0.f;
+            for (int t = 0; t < kTok; ++t) e += s_k[t][k];
+            p.decay[((size_t)piece * p.heads + head) * d + k] = expf(-e);
+        }
     }
 }
 
@@ -188,8 +236,8 @@ __global__ void __launch_bounds__(256) time_mix_out_kernel(const float* o, const
 }
 
 int pieces_for(int heads, int dim, int rows) {
-    const int base = heads * ((dim + kCols - 1) / kCols);
-    const int want = std::max(1, sm_count() * 8 / base);
+    const int base = heads * ((dim + 63) / 64);
+    const int want = std::max(1, sm_count() * 4 / base);
     const int n = std::min(want, rows / kMinPiece);
     return n < 3 ? 1 : n;
 }
@@ -215,14 +263,16 @@ int scan(const leankv_time_mix_t& a, const void* r, const void* k, const void* v
     p.o = ws;
     float* pieces = ws + (size_t)rows * a.heads * a.dim;
     float* decay = pieces + (size_t)n * state_floats(a.heads, a.dim);
-    const dim3 block(kCols * kSlices);
-    const int cb = (a.dim + kCols - 1) / kCols;
+    using Sh = ScanShape<L>;
+    const dim3 block(Sh::kThreads);
+    const int cb = (a.dim + Sh::kCols - 1) / Sh::kCols;
+    const bool vec = a.dim % 8 == 0 && aligned16(r) && aligned16(k) && aligned16(v) && aligned16(z);
     p.S_in = a.S;
     if (p.n_pieces > 1) {
         p.S_out = pieces;
         p.decay = decay;
         LEANKV_CUDA_TRY(launch_kernel(time_mix_scan_kernel<T, L, false>, dim3(a.heads, cb, p.n_pieces - 1), block, 0, st,
-                                      p));
+                                      p, vec));
         const long long total = (long long)state_floats(a.heads, a.dim);
         LEANKV_CUDA_TRY(launch_kernel(time_mix_carry_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, st,
                                       static_cast<const float*>(a.S), pieces, static_cast<const float*>(decay), a.heads,
@@ -230,7 +280,7 @@ int scan(const leankv_time_mix_t& a, const void* r, const void* k, const void* v
         p.S_in = pieces;
     }
     p.S_out = a.S;
-    LEANKV_CUDA_TRY(launch_kernel(time_mix_scan_kernel<T, L, true>, dim3(a.heads, cb, p.n_pieces), block, 0, st, p));
+    LEANKV_CUDA_TRY(launch_kernel(time_mix_scan_kernel<T, L, true>, dim3(a.heads, cb, p.n_pieces), block, 0, st, p, vec));
     return LEANKV_OK;
 }
 
@@ -238,10 +288,10 @@ template <typename T>
 int rows_all(const leankv_time_mix_t& a, const void* r, const void* k, const void* v, const void* g, const float* z,
              void* out, int out_ld, float out_scale, int rows, float* ws, cudaStream_t st) {
     int rc = LEANKV_ELIMIT;
-    if (a.dim <= 4 * 8) rc = scan<T, 8>(a, r, k, v, z, ws, rows, st);
-    else if (a.dim <= 4 * 16) rc = scan<T, 16>(a, r, k, v, z, ws, rows, st);
-    else if (a.dim <= 4 * 32) rc = scan<T, 32>(a, r, k, v, z, ws, rows, st);
-    else if (a.dim <= 4 * 64) rc = scan<T, 64>(a, r, k, v, z, ws, rows, st);
+    if (a.dim <= 8 * 4) rc = scan<T, 4>(a, r, k, v, z, ws, rows, st);
+    else if (a.dim <= 8 * 8) rc = scan<T, 8>(a, r, k, v, z, ws, rows, st);
+    else if (a.dim <= 8 * 16) rc = scan<T, 16>(a, r, k, v, z, ws, rows, st);
+    else if (a.dim <= 8 * 32) rc = scan<T, 32>(a, r, k, v, z, ws, rows, st);
     if (rc) return rc;
     const long long warps = (long long)rows * a.heads;
     LEANKV_CUDA_TRY(launch_kernel(time_mix_out_kernel<T>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, st,

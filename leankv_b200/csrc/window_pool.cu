@@ -22,24 +22,88 @@ __global__ void __launch_bounds__(kAppendThreads) window_pool_append_kernel(cons
     const int t = blockIdx.x, G = a.kv_heads, nq = a.heads * a.dim, nk = G * a.dim;
     const float* row = qkv + (size_t)t * ld;
     const int slot = (start + t) % a.ring;
-    const float fq = row_factor(row, bias, nq, a.q_norm != nullptr, a.eps, s_tmp);
-    const float fk = row_factor(row + nq, bias ? bias + nq : nullptr, nk, a.k_norm != nullptr, a.eps, s_tmp);
+    const RowFactors f = row_factors(row, bias, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
     auto at = [&](int i) { return row[i] + (bias != nullptr ? __ldg(bias + i) : 0.f); };
     T* q = q_out + (size_t)t * a.heads * a.dim_pad;
     for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAppendThreads) {
         const int h = e / a.dim_pad, d = e - h * a.dim_pad, i = h * a.dim + d;
-        q[e] = from_f32<T>(d < a.dim ? at(i) * fq * (a.q_norm ? __ldg(a.q_norm + i) : 1.f) : 0.f);
+        q[e] = from_f32<T>(d < a.dim ? at(i) * f.q * (a.q_norm ? __ldg(a.q_norm + i) : 1.f) : 0.f);
     }
     T* k = static_cast<T*>(a.k_ring) + (size_t)slot * G * a.dim_pad;
     for (int e = threadIdx.x; e < G * a.dim_pad; e += kAppendThreads) {
         const int g = e / a.dim_pad, d = e - g * a.dim_pad, i = g * a.dim + d;
-        k[e] = from_f32<T>(d < a.dim ? at(nq + i) * fk * (a.k_norm ? __ldg(a.k_norm + i) : 1.f) : 0.f);
+        k[e] = from_f32<T>(d < a.dim ? at(nq + i) * f.k * (a.k_norm ? __ldg(a.k_norm + i) : 1.f) : 0.f);
     }
     T* v = static_cast<T*>(a.v_ring) + (size_t)slot * G * a.vdim_pad;
     for (int e = threadIdx.x; e < G * a.vdim_pad; e += kAppendThreads) {
         const int g = e / a.vdim_pad, d = e - g * a.vdim_pad;
         v[e] = from_f32<T>(d < a.vdim ? at(nq + nk + g * a.vdim + d) : 0.f);
     }
+}
+
+// The same with 4-element accesses, the row in registers (dim, vdim and ld multiples of 4, at most
+// kAppendThreads * 4 * NV columns).
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v) {
+    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = v;
+    else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+template <typename T, int NV>
+__global__ void __launch_bounds__(kAppendThreads) window_pool_append_vec_kernel(const leankv_window_pool_t a,
+                                                                                const float* qkv, int ld,
+                                                                                const float* bias, T* q_out, int start) {
+    __shared__ float s_tmp[32];
+    pdl_begin();
+    const int t = blockIdx.x, tid = threadIdx.x, G = a.kv_heads, nq = a.heads * a.dim, nk = G * a.dim, nv = G * a.vdim;
+    const float* row = qkv + (size_t)t * ld;
+    const int slot = (start + t) % a.ring;
+    float4 x[NV];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int i = (tid + n * kAppendThreads) * 4;
+        if (i >= nq + nk + nv) continue;
+        x[n] = *reinterpret_cast<const float4*>(row + i);
+        if (bias != nullptr) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + i);
+            x[n].x += b.x; x[n].y += b.y; x[n].z += b.z; x[n].w += b.w;
+        }
+        const float ss = x[n].x * x[n].x + x[n].y * x[n].y + x[n].z * x[n].z + x[n].w * x[n].w;
+        if (i < nq) sq += ss;
+        else if (i < nq + nk) sk += ss;
+    }
+    const RowFactors f = norm_factors(sq, sk, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
+    T* q = q_out + (size_t)t * a.heads * a.dim_pad;
+    T* k = static_cast<T*>(a.k_ring) + (size_t)slot * G * a.dim_pad;
+    T* v = static_cast<T*>(a.v_ring) + (size_t)slot * G * a.vdim_pad;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        int i = (tid + n * kAppendThreads) * 4;
+        if (i >= nq + nk + nv) continue;
+        const bool is_q = i < nq, is_k = !is_q && i < nq + nk;
+        T* dst;
+        if (is_q || is_k) {
+            const float* w = is_q ? a.q_norm : a.k_norm;
+            const float fac = is_q ? f.q : f.k;
+            if (is_k) i -= nq;
+            if (w != nullptr) {
+                const float4 g = *reinterpret_cast<const float4*>(w + i);
+                x[n].x *= g.x; x[n].y *= g.y; x[n].z *= g.z; x[n].w *= g.w;
+            }
+            x[n].x *= fac; x[n].y *= fac; x[n].z *= fac; x[n].w *= fac;
+            const int h = i / a.dim;
+            dst = (is_q ? q : k) + h * a.dim_pad + i - h * a.dim;
+        } else {
+            i -= nq + nk;
+            const int g = i / a.vdim;
+            dst = v + g * a.vdim_pad + i - g * a.vdim;
+        }
+        store4(dst, x[n]);
+    }
+    const int pd = a.dim_pad - a.dim, pv = a.vdim_pad - a.vdim;
+    for (int e = tid; e < a.heads * pd; e += kAppendThreads) q[e / pd * a.dim_pad + a.dim + e % pd] = from_f32<T>(0.f);
+    for (int e = tid; e < G * pd; e += kAppendThreads) k[e / pd * a.dim_pad + a.dim + e % pd] = from_f32<T>(0.f);
+    for (int e = tid; e < G * pv; e += kAppendThreads) v[e / pv * a.vdim_pad + a.vdim + e % pv] = from_f32<T>(0.f);
 }
 
 // Blocks first .. : mean of the block's keys / values as the ring holds them. One CTA per block.
@@ -70,7 +134,10 @@ __global__ void __launch_bounds__(kAttendThreads) window_pool_rows_kernel(const 
     const int t = blockIdx.x;
     const AttendPlan pl(a, kAttendThreads, n_max, kAttendSmemFloats);
     const T* row = q + (size_t)t * a.heads * a.dim_pad;
-    for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAttendThreads) sm[pl.q + e] = to_f32(row[e]) * a.scale;
+    for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAttendThreads) {
+        const int h = e / a.dim_pad;
+        put_query<T>(pl, sm, a.heads, h, e - h * a.dim_pad, to_f32(row[e]) * a.scale);
+    }
     __syncthreads();
     attend_query<T, T>(a, pl, sm, ws + (size_t)t * 2 * a.heads * pl.ldp, start + t, false, 0, 1,
                        out + (size_t)t * out_ld, out_scale);
@@ -91,8 +158,20 @@ int check_args(const leankv_window_pool_t* a) {
 template <typename T>
 int append(const leankv_window_pool_t& a, const float* qkv, int ld, const float* bias, void* q, int rows, int start,
            cudaStream_t st) {
-    LEANKV_CUDA_TRY(launch_kernel(window_pool_append_kernel<T>, dim3(rows), dim3(kAppendThreads), 0, st, a, qkv, ld,
-                                  bias, static_cast<T*>(q), start));
+    const int cols = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
+    const int nv = (cols + kAppendThreads * 4 - 1) / (kAppendThreads * 4);
+    const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && ld % 4 == 0 && nv <= 12 && aligned16(qkv) && aligned16(bias) &&
+                     aligned16(a.q_norm) && aligned16(a.k_norm) && aligned16(q);
+    auto go = [&](auto kernel) -> int {
+        LEANKV_CUDA_TRY(launch_kernel(kernel, dim3(rows), dim3(kAppendThreads), 0, st, a, qkv, ld, bias,
+                                      static_cast<T*>(q), start));
+        return LEANKV_OK;
+    };
+    const int rc = !vec      ? go(window_pool_append_kernel<T>)
+                   : nv <= 2 ? go(window_pool_append_vec_kernel<T, 2>)
+                   : nv <= 6 ? go(window_pool_append_vec_kernel<T, 6>)
+                             : go(window_pool_append_vec_kernel<T, 12>);
+    if (rc) return rc;
     const int b0 = start / a.pool, b1 = std::min((start + rows) / a.pool, a.max_blocks);
     if (b1 > b0)
         LEANKV_CUDA_TRY(launch_kernel(window_pool_blocks_kernel<T>, dim3(b1 - b0), dim3(256), 0, st, a, b0));

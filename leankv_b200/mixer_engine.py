@@ -106,7 +106,7 @@ class MixerDecodeEngine(DecodeLoop):
         W, V, t = cfg.hidden_size, cfg.vocab_size, {}
 
         def draw(name, *shape, std=0.02, mean=0.0):
-            t[name] = (torch.randn(*shape, generator=gen, device=device) * std + mean).bfloat16()
+            t[name] = (torch.randn(shape, generator=gen, device=device) * std + mean).bfloat16()
 
         draw("embed", V, W, std=1.0)
         draw("head", V, W)
