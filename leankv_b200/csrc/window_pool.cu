@@ -227,6 +227,9 @@ extern "C" int leankv_window_pool_attend(const leankv_window_pool_t* a, const vo
     if (rc) return rc;
     if (!q || !out || rows <= 0 || start < 0 || out_ld < a->heads * a->vdim) return LEANKV_EINVAL;
     if (VisibleKeys(start + rows - 1, a->size, a->pool).n_blk > a->max_blocks) return LEANKV_ELIMIT;
+    if (!aligned16(q)) return LEANKV_EALIGN;
+    const int tiled = window_pool_tile_attend(*a, q, out, out_ld, out_scale, rows, start, static_cast<cudaStream_t>(stream));
+    if (tiled != LEANKV_EUNSUPPORTED) return tiled;
     if (leankv_window_pool_workspace_bytes(a, rows, start + rows) > (ws ? ws_bytes : 0)) return LEANKV_EWORKSPACE;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     float* w = static_cast<float*>(ws);

@@ -24,6 +24,11 @@ struct VisibleKeys {
     }
 };
 
+// The tensor-core route of leankv_window_pool_attend (window_pool_tile.cu); LEANKV_EUNSUPPORTED for storage types,
+// head counts and sizes it does not take.
+int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* out, int out_ld, float out_scale, int rows,
+                            int start, cudaStream_t st);
+
 constexpr int kAttendHeads = 4;     // query heads a thread carries at once
 
 // Row length (elements) of bf16 operand rows in shared memory: 16-byte fragment reads of eight consecutive rows

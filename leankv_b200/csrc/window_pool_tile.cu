@@ -1,0 +1,424 @@
+// Window + pooled-block attention of a prompt portion on tensor cores (bf16): one CTA per eight queries, all heads.
+//
+// The weights of all heads of a (query, key) pair meet in the mix across heads, so they have to be in one CTA,
+// normalised, before the mix. Pass 1 computes every head's softmax statistics, pass 2 the scores again and from
+// them normalised weights, the mix and the product with the values. Scores and outputs are computed transposed
+// (keys or value columns as the 16 rows of an MMA tile, the eight queries as its columns), which keeps the
+// output accumulators of 32 heads x 128 columns in the registers of eight warps. Weights enter the mix as two
+// bf16 numbers each (16 bits); after it they are rounded once for the product with the values.
+//
+// A warp owns HPW query heads of one kv head; with few heads, several warps share a head and take every KS-th
+// key tile. Key rows go straight from L2 to registers (no other warp needs them), value rows through a
+// warp-private buffer because their fragments need the transposing load.
+
+#include <algorithm>
+
+#include "window_pool.cuh"
+
+namespace leankv {
+namespace {
+
+constexpr int kWarps = 8;
+constexpr int kThreads = 32 * kWarps;
+constexpr int kQ = 8;           // queries per CTA
+constexpr int kMaxNb = 4;       // blocks of 32 dimensions
+
+struct TileParams {
+    leankv_window_pool_t a;
+    const bf16* q;
+    bf16* out;
+    int out_ld, rows, start;
+    float out_scale;
+    int hs, ks;                 // head slots, key splits
+    int nb;                     // 32-blocks of dim_pad, the last may be half
+    int off_p, off_pm, off_v, off_t, off_stat, p_row, p_key, pm_q, pm_h, v_row;      // bytes, words for pm_*
+};
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <int HPW, int DVT>
+__global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_tile_kernel(const __grid_constant__ TileParams p) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    pdl_begin();
+    const leankv_window_pool_t& a = p.a;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int H = a.heads, G = a.kv_heads, rep = H / G, dp = a.dim_pad, vp = a.vdim_pad, nb = p.nb, KS = p.ks;
+    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kQ;           // the longest rows first
+    const int nq = min(kQ, p.rows - q0), i0 = p.start + q0, iL = i0 + nq - 1;
+    const VisibleKeys first(i0, a.size, a.pool), last(iL, a.size, a.pool);
+    const int tok0 = first.w0, ntok = iL - tok0 + 1, TB = (last.n_blk + 15) / 16, NT = TB + (ntok + 15) / 16;
+    const int hslot = warp % p.hs, ks = warp / p.hs, h0 = hslot * HPW, kv = h0 / rep;
+    const bool worker = ks < KS;
+    const float c = a.scale * 1.4426950408889634f;
+
+    // queries in fragment order: [head][block][lane] 16 bytes (query lane / 4, dimensions 8 (lane % 4) ..)
+    for (int e = tid; e < H * nb * 32; e += kThreads) {
+        const int l = e & 31, b = (e >> 5) % nb, h = (e >> 5) / nb, d = b * 32 + (l & 3) * 8;
+        const int row = min(q0 + (l >> 2), p.rows - 1);
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (d < dp) v = *reinterpret_cast<const uint4*>(p.q + ((size_t)row * H + h) * dp + d);
+        reinterpret_cast<uint4*>(smem)[e] = v;
+    }
+    // mixing matrix in fragment order, high then low parts: [row tile][column tile][2][lane] 16 bytes; lane t holds
+    // input heads 4 t .. 4 t + 3 of the column tile
+    const int MT = (H + 15) / 16;
+    for (int e = tid; e < MT * MT * 32; e += kThreads) {
+        const int l = e & 31, kt = (e >> 5) % MT, mt = (e >> 5) / MT;
+        const int r = mt * 16 + (l >> 2), col = kt * 16 + (l & 3) * 4;
+        auto at = [&](int h, int x) {
+            if (h >= H || x >= H) return 0.f;
+            return a.talk != nullptr ? __ldg(a.talk + h * H + x) : (h == x ? 1.f : 0.f);
+        };
+        uint32_t hi[4], lo[4];
+        split_bf16(at(r, col), at(r, col + 1), hi[0], lo[0]);
+        split_bf16(at(r + 8, col), at(r + 8, col + 1), hi[1], lo[1]);
+        split_bf16(at(r, col + 2), at(r, col + 3), hi[2], lo[2]);
+        split_bf16(at(r + 8, col + 2), at(r + 8, col + 3), hi[3], lo[3]);
+        uint4* dst = reinterpret_cast<uint4*>(smem + p.off_t) + (e >> 5) * 64 + l;
+        dst[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        dst[32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    // weights of padding heads stay zero
+    for (int e = tid; e < (p.off_pm - p.off_p) / 4; e += kThreads) reinterpret_cast<uint32_t*>(smem + p.off_p)[e] = 0;
+    __syncthreads();
+
+    // this thread's two queries
+    int iq[2], w0q[2], nbq[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        iq[x] = i0 + min(2 * t + x, nq - 1);
+        const VisibleKeys v(iq[x], a.size, a.pool);
+        w0q[x] = v.w0;
+        nbq[x] = v.n_blk;
+    }
+    const bf16* k_ring = static_cast<const bf16*>(a.k_ring);
+    const bf16* k_pool = static_cast<const bf16*>(a.k_pool);
+
+    // row of a tile's key r (clamped to the keys that exist): index into the pooled blocks or the ring
+    struct TileRows { bool pooled; int base, n, slot0; };
+    auto rows_of = [&](int tile) {
+        TileRows tr;
+        tile = min(tile, NT - 1);
+        tr.pooled = tile < TB;
+        tr.base = (tr.pooled ? tile : tile - TB) * 16;
+        tr.n = (tr.pooled ? last.n_blk : ntok) - tr.base;
+        tr.slot0 = tr.pooled ? tr.base : (tok0 + tr.base) % a.ring;
+        return tr;
+    };
+    auto index_of = [&](const TileRows& tr, int r) {
+        int s = tr.slot0 + min(r, tr.n - 1);
+        if (!tr.pooled && s >= a.ring) s -= a.ring;
+        return s;
+    };
+    uint4 x0[kMaxNb], x1[kMaxNb];
+    auto load_keys = [&](int tile) {
+        const TileRows tr = rows_of(tile);
+        const bf16* src = (tr.pooled ? k_pool : k_ring) + (size_t)kv * dp + t * 8;
+        const bf16* r0 = src + (size_t)index_of(tr, g) * G * dp;
+        const bf16* r1 = src + (size_t)index_of(tr, g + 8) * G * dp;
+#pragma unroll
+        for (int b = 0; b < kMaxNb; ++b)
+            if (b < nb) {
+                const bool on = b * 32 + t * 8 < dp;
+                x0[b] = on ? *reinterpret_cast<const uint4*>(r0 + b * 32) : make_uint4(0, 0, 0, 0);
+                x1[b] = on ? *reinterpret_cast<const uint4*>(r1 + b * 32) : make_uint4(0, 0, 0, 0);
+            }
+    };
+    float s[HPW][4];
+    auto score = [&](int tile) {        // scaled to base-2 exponents, -inf where the query does not see the key
+#pragma unroll
+        for (int h = 0; h < HPW; ++h)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) s[h][x] = 0.f;
+#pragma unroll
+        for (int b = 0; b < kMaxNb; ++b)
+            if (b < nb) {
+#pragma unroll
+                for (int h = 0; h < HPW; ++h) {
+                    const uint4 y = reinterpret_cast<const uint4*>(smem)[((h0 + h) * nb + b) * 32 + lane];
+                    mma_bf16(s[h], x0[b].x, x1[b].x, x0[b].y, x1[b].y, y.x, y.y);
+                    mma_bf16(s[h], x0[b].z, x1[b].z, x0[b].w, x1[b].w, y.z, y.w);
+                }
+            }
+        bool see[4] = {true, true, true, true};
+        const bool pooled = tile < TB;
+        const int base = pooled ? tile * 16 : tok0 + (tile - TB) * 16;
+        const bool all = tile < NT && (pooled ? base + 15 < first.n_blk : base >= last.w0 && base + 15 <= i0);
+        if (!all) {
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const int at = base + g + (x < 2 ? 0 : 8), qx = x & 1;
+                see[x] = tile < NT && (pooled ? at < nbq[qx] : at >= w0q[qx] && at <= iq[qx]);
+            }
+        }
+#pragma unroll
+        for (int h = 0; h < HPW; ++h)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) s[h][x] = see[x] ? s[h][x] * c : -INFINITY;
+    };
+
+    // ---- pass 1: log2 of the softmax denominators ----
+    float lse[HPW][2];
+    {
+        float m[HPW][2], l[HPW][2];
+#pragma unroll
+        for (int h = 0; h < HPW; ++h) m[h][0] = m[h][1] = -1e30f, l[h][0] = l[h][1] = 0.f;
+        if (worker) {
+            load_keys(ks);
+            for (int tile = ks; tile < NT; tile += KS) {
+                score(tile);
+                load_keys(tile + KS);
+#pragma unroll
+                for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const float mn = fmaxf(m[h][x], fmaxf(s[h][x], s[h][x + 2]));
+                        l[h][x] = l[h][x] * ex2(m[h][x] - mn) + ex2(s[h][x] - mn) + ex2(s[h][x + 2] - mn);
+                        m[h][x] = mn;
+                    }
+            }
+        }
+        float* stat = reinterpret_cast<float*>(smem + p.off_stat);       // [KS][H][8][2]
+#pragma unroll
+        for (int h = 0; h < HPW; ++h)
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+#pragma unroll
+                for (int o = 4; o < 32; o *= 2) {
+                    const float mo = __shfl_xor_sync(0xffffffffu, m[h][x], o), lo = __shfl_xor_sync(0xffffffffu, l[h][x], o);
+                    const float mn = fmaxf(m[h][x], mo);
+                    l[h][x] = l[h][x] * ex2(m[h][x] - mn) + lo * ex2(mo - mn);
+                    m[h][x] = mn;
+                }
+                if (worker && g == 0) {
+                    float* d = stat + (((size_t)ks * H + h0 + h) * kQ + 2 * t + x) * 2;
+                    d[0] = m[h][x];
+                    d[1] = l[h][x];
+                }
+            }
+        __syncthreads();
+        if (worker) {
+#pragma unroll
+            for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const float* d = stat + ((size_t)(h0 + h) * kQ + 2 * t + x) * 2;
+                    float mm = -1e30f, ll = 0.f;
+                    for (int k = 0; k < KS; ++k) mm = fmaxf(mm, d[(size_t)k * H * kQ * 2]);
+                    for (int k = 0; k < KS; ++k)
+                        ll += d[(size_t)k * H * kQ * 2 + 1] * ex2(d[(size_t)k * H * kQ * 2] - mm);
+                    lse[h][x] = mm + log2f(ll);
+                }
+        }
+    }
+
+    // ---- pass 2 ----
+    float o[HPW][DVT][4];
+#pragma unroll
+    for (int h = 0; h < HPW; ++h)
+#pragma unroll
+        for (int m = 0; m < DVT; ++m)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) o[h][m][x] = 0.f;
+    const int dvt = vp / 16;
+    unsigned char* vbuf = smem + p.off_v + (size_t)warp * 16 * p.v_row;
+    const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(vbuf);
+    uint32_t* pm = reinterpret_cast<uint32_t*>(smem + p.off_pm);
+    if (worker) load_keys(ks);
+    for (int base = 0; base < NT; base += KS) {
+        const int tile = base + ks;
+        if (worker) {
+            {       // this tile's values start their way
+                const TileRows tr = rows_of(tile);
+                const bf16* src = static_cast<const bf16*>(tr.pooled ? a.v_pool : a.v_ring) + (size_t)kv * vp;
+                const int per = vp / 8;
+                for (int e = lane; e < 16 * per; e += 32) {
+                    const int r = e / per, ch = e - r * per;
+                    const bf16* from = src + (size_t)index_of(tr, r) * G * vp + ch * 8;
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vaddr + r * p.v_row + ch * 16), "l"(from)
+                                 : "memory");
+                }
+                asm volatile("cp.async.commit_group;" ::: "memory");
+            }
+            score(tile);
+            if (base + KS < NT) load_keys(tile + KS);
+            // normalised weights as high + low bf16: [key][query][head / 4] {4 high, 4 low}
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                float w[HPW];
+#pragma unroll
+                for (int h = 0; h < HPW; ++h) w[h] = ex2(s[h][x] - lse[h][x & 1]);
+                const int key = ks * 16 + g + (x < 2 ? 0 : 8), qq = 2 * t + (x & 1);
+                unsigned char* dst = smem + p.off_p + key * p.p_key + qq * p.p_row + (h0 >> 2) * 16;
+                if constexpr (HPW == 4) {
+                    uint4 v;
+                    split_bf16(w[0], w[1], v.x, v.z);
+                    split_bf16(w[2], w[3], v.y, v.w);
+                    *reinterpret_cast<uint4*>(dst) = v;
+                } else if constexpr (HPW == 2) {
+                    uint32_t hi, lo;
+                    split_bf16(w[0], w[1], hi, lo);
+                    *reinterpret_cast<uint32_t*>(dst + (h0 & 2) * 2) = hi;
+                    *reinterpret_cast<uint32_t*>(dst + 8 + (h0 & 2) * 2) = lo;
+                } else {
+#pragma unroll
+                    for (int h = 0; h < HPW; ++h) {
+                        const int hh = h0 + h;
+                        unsigned char* d = smem + p.off_p + key * p.p_key + qq * p.p_row + (hh >> 2) * 16 + (hh & 3) * 2;
+                        const bf16 hi = from_f32<bf16>(w[h]);
+                        *reinterpret_cast<bf16*>(d) = hi;
+                        *reinterpret_cast<bf16*>(d + 8) = from_f32<bf16>(w[h] - to_f32(hi));
+                    }
+                }
+            }
+        }
+        __syncthreads();
+        // mix across heads, two keys at a time: [head][query][key] bf16
+        for (int pair = warp; pair < 8 * KS; pair += kWarps) {
+            const unsigned char* src = smem + p.off_p + (size_t)pair * 2 * p.p_key + g * p.p_row + t * 16;
+            for (int mt = 0; mt < MT; ++mt) {
+                float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int kt = 0; kt < MT; ++kt) {
+                    const uint4* tf = reinterpret_cast<const uint4*>(smem + p.off_t) + (mt * MT + kt) * 64 + lane;
+                    const uint4 ah = tf[0], al = tf[32];
+                    const uint4 b0 = *reinterpret_cast<const uint4*>(src + kt * 64);
+                    const uint4 b1 = *reinterpret_cast<const uint4*>(src + p.p_key + kt * 64);
+                    mma_bf16(d0, ah.x, ah.y, ah.z, ah.w, b0.x, b0.y);
+                    mma_bf16(d1, ah.x, ah.y, ah.z, ah.w, b1.x, b1.y);
+                    mma_bf16(d0, ah.x, ah.y, ah.z, ah.w, b0.z, b0.w);
+                    mma_bf16(d1, ah.x, ah.y, ah.z, ah.w, b1.z, b1.w);
+                    mma_bf16(d0, al.x, al.y, al.z, al.w, b0.x, b0.y);
+                    mma_bf16(d1, al.x, al.y, al.z, al.w, b1.x, b1.y);
+                }
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    const int h = mt * 16 + g + (x < 2 ? 0 : 8);
+                    if (h < H) pm[h * p.pm_h + (2 * t + (x & 1)) * p.pm_q + pair] = pack_bf16(d0[x], d1[x]);
+                }
+            }
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (worker) {
+            uint32_t b[HPW][2];
+#pragma unroll
+            for (int h = 0; h < HPW; ++h) {
+                const uint32_t* w = pm + (h0 + h) * p.pm_h + g * p.pm_q + ks * 8 + t;
+                b[h][0] = w[0];
+                b[h][1] = w[4];
+            }
+            const int mi = lane >> 3, r = (lane & 7) + (mi >= 2 ? 8 : 0);
+            const uint32_t from = vaddr + r * p.v_row + (mi & 1) * 16;
+#pragma unroll
+            for (int m = 0; m < DVT; ++m)
+                if (m < dvt) {
+                    uint32_t a0, a1, a2, a3;
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                 : "=r"(a0), "=r"(a1), "=r"(a2), "=r"(a3)
+                                 : "r"(from + m * 32));
+#pragma unroll
+                    for (int h = 0; h < HPW; ++h) mma_bf16(o[h][m], a0, a1, a2, a3, b[h][0], b[h][1]);
+                }
+            __syncwarp();
+        }
+    }
+
+    // ---- outputs: sum over the key splits, through the value buffers' space ----
+    if (KS > 1) {
+        float* red = reinterpret_cast<float*>(smem + p.off_v);           // [head][vp][8 queries]
+        for (int k = 1; k < KS; ++k) {
+            __syncthreads();
+            if (ks == k) {
+#pragma unroll
+                for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                    for (int m = 0; m < DVT; ++m)
+                        if (m < dvt)
+#pragma unroll
+                            for (int x = 0; x < 4; ++x)
+                                red[((h0 + h) * vp + m * 16 + g + (x < 2 ? 0 : 8)) * kQ + 2 * t + (x & 1)] = o[h][m][x];
+            }
+            __syncthreads();
+            if (ks == 0) {
+#pragma unroll
+                for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                    for (int m = 0; m < DVT; ++m)
+                        if (m < dvt)
+#pragma unroll
+                            for (int x = 0; x < 4; ++x)
+                                o[h][m][x] += red[((h0 + h) * vp + m * 16 + g + (x < 2 ? 0 : 8)) * kQ + 2 * t + (x & 1)];
+            }
+        }
+    }
+    if (ks == 0) {
+#pragma unroll
+        for (int h = 0; h < HPW; ++h)
+#pragma unroll
+            for (int m = 0; m < DVT; ++m)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    const int d = m * 16 + g + (x < 2 ? 0 : 8), qq = 2 * t + (x & 1);
+                    if (d < a.vdim && qq < nq)
+                        p.out[(size_t)(q0 + qq) * p.out_ld + (h0 + h) * a.vdim + d] = from_f32<bf16>(o[h][m][x] * p.out_scale);
+                }
+    }
+}
+
+template <int HPW, int DVT>
+int launch(const TileParams& p, size_t smem, cudaStream_t st) {
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(window_pool_tile_kernel<HPW, DVT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem));
+    LEANKV_CUDA_TRY(launch_kernel(window_pool_tile_kernel<HPW, DVT>, dim3((p.rows + kQ - 1) / kQ), dim3(kThreads), smem, st,
+                                  p));
+    return LEANKV_OK;
+}
+
+}  // namespace
+
+int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* out, int out_ld, float out_scale, int rows,
+                            int start, cudaStream_t st) {
+    const int rep = a.heads / a.kv_heads;
+    if (a.dtype != LEANKV_DT_BF16 || a.dim_pad > 32 * kMaxNb || a.vdim_pad > 128) return LEANKV_EUNSUPPORTED;
+    int hpw = 1;
+    while (hpw <= 4 && (rep % hpw != 0 || a.heads / hpw > kWarps)) ++hpw;
+    if (hpw > 4) return LEANKV_EUNSUPPORTED;
+    TileParams p{};
+    p.a = a;
+    p.q = static_cast<const bf16*>(q);
+    p.out = static_cast<bf16*>(out);
+    p.out_ld = out_ld;
+    p.out_scale = out_scale;
+    p.rows = rows;
+    p.start = start;
+    p.hs = a.heads / hpw;
+    p.ks = kWarps / p.hs;
+    p.nb = (a.dim_pad + 31) / 32;
+    const int hp = (a.heads + 15) / 16 * 16, mt = hp / 16;
+    p.p_row = hp * 4 + 16;              // fragment rows a few banks apart
+    p.p_key = kQ * p.p_row + 16;
+    p.pm_q = 8 * p.ks + 4;
+    p.pm_h = kQ * p.pm_q + 1;
+    p.v_row = a.vdim_pad * 2 + 16;
+    int at = a.heads * p.nb * 512;
+    const auto take = [&](int bytes) { const int o = at; at += (bytes + 127) / 128 * 128; return o; };
+    p.off_t = take(mt * mt * 1024);
+    p.off_stat = take(p.ks * a.heads * kQ * 8);
+    p.off_p = take(16 * p.ks * p.p_key);
+    p.off_pm = take(a.heads * p.pm_h * 4);
+    p.off_v = take(std::max(kWarps * 16 * p.v_row, p.ks > 1 ? a.heads * a.vdim_pad * kQ * 4 : 0));
+    if (at > 227 * 1024) return LEANKV_EUNSUPPORTED;
+    const bool narrow = a.vdim_pad <= 64;
+    switch (hpw) {
+        case 1: return narrow ? launch<1, 4>(p, at, st) : launch<1, 8>(p, at, st);
+        case 2: return narrow ? launch<2, 4>(p, at, st) : launch<2, 8>(p, at, st);
+        case 3: return narrow ? launch<3, 4>(p, at, st) : launch<3, 8>(p, at, st);
+        default: return narrow ? launch<4, 4>(p, at, st) : launch<4, 8>(p, at, st);
+    }
+}
+
+}  // namespace leankv
