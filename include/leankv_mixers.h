@@ -134,7 +134,8 @@ int leankv_time_mix_rows(const leankv_time_mix_t* a, const void* r, const void* 
 
 /* One decode step of both mixers in one launch (either may be NULL). y: fp32 projections of the step's
  * token, q | k | v at qkv_off and r | k | v | g at rkvg_off, low-rank decay input (rank numbers) at w1_off; w2
- * [heads * dim][rank] of the storage type. out fp32: left at 0, right at right_off, each times its scale. */
+ * [heads * dim][rank] of the storage type. The position state[0], the rings and the pooled blocks may be read
+ * before the launch just ahead of this one has finished: that launch must not write them. out fp32: left at 0, right at right_off, each times its scale. */
 typedef struct leankv_mixer_step {
     const float* y;
     int qkv_off, rkvg_off, w1_off, rank;

@@ -12,7 +12,6 @@ namespace leankv {
 namespace {
 
 constexpr int kStepThreads = 512;
-constexpr int kMaxCluster = 16;     // non-portable; 8 where the device does not place 16
 constexpr int kStepSmemFloats = 200 * 1024 / 4;
 
 struct StepParams {
@@ -22,35 +21,96 @@ struct StepParams {
     int has_left, has_right, n_max, cluster;
 };
 
+constexpr int kRowVecs = 6;        // float4s of the projection row a thread keeps: rows up to 12288 columns
+
 template <typename T>
 __device__ void left_step(const StepParams& p, float* sm, float* s_tmp, int rank) {
     const leankv_window_pool_t& a = p.left;
     const AttendPlan pl(a, kStepThreads, (p.n_max + p.cluster - 1) / p.cluster, kStepSmemFloats);
     const int tid = threadIdx.x, i = p.s.state[kPos], G = a.kv_heads;
-    const int nq = a.heads * a.dim, nk = G * a.dim;
+    const int nq = a.heads * a.dim, nk = G * a.dim, nv = G * a.vdim;
     const float* y = p.s.y + p.s.qkv_off;       // biases are already in
-    const RowFactors f = row_factors(y, nullptr, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
-    for (int e = tid; e < a.heads * a.dim_pad; e += kStepThreads) {
-        const int h = e / a.dim_pad, d = e - h * a.dim_pad, x = h * a.dim + d;
-        put_query<T>(pl, sm, a.heads, h, d, d < a.dim ? y[x] * f.q * (a.q_norm ? __ldg(a.q_norm + x) : 1.f) * a.scale : 0.f);
-    }
-    const int slot = i % a.ring;
     T* k_ring = static_cast<T*>(a.k_ring);
     T* v_ring = static_cast<T*>(a.v_ring);
+
+    // before the projections are there: the mix, and this CTA's key / value rows on their way into L2
+    put_talk(a, pl, sm);
+    {
+        const VisibleKeys vis(i, a.size, a.pool);
+        const int j0 = (int)((long long)vis.n * rank / p.cluster), j1 = (int)((long long)vis.n * (rank + 1) / p.cluster);
+        const int kb = G * a.dim_pad * (int)sizeof(T), per = (kb + 127) / 128;
+        const int vb = G * a.vdim_pad * (int)sizeof(T), perv = (vb + 127) / 128;
+        for (int e = tid; e < (j1 - j0) * (per + perv); e += kStepThreads) {
+            const int jl = e / (per + perv), c = e - jl * (per + perv), j = j0 + jl;
+            const int row = j < vis.n_blk ? j : (vis.w0 + j - vis.n_blk) % a.ring;
+            const char* base = c < per ? static_cast<const char*>(j < vis.n_blk ? a.k_pool : a.k_ring) + (size_t)row * kb + c * 128
+                                       : static_cast<const char*>(j < vis.n_blk ? a.v_pool : a.v_ring) + (size_t)row * vb + (c - per) * 128;
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(base));
+        }
+    }
+    pdl_begin();
+
+    const int slot = i % a.ring;
     T* k_new = reinterpret_cast<T*>(sm + pl.knew);
     T* v_new = reinterpret_cast<T*>(sm + pl.vnew);
-    for (int e = tid; e < G * a.dim_pad; e += kStepThreads) {
-        const int g = e / a.dim_pad, d = e - g * a.dim_pad, x = g * a.dim + d;
-        const T v = from_f32<T>(d < a.dim ? y[nq + x] * f.k * (a.k_norm ? __ldg(a.k_norm + x) : 1.f) : 0.f);
-        k_new[e] = v;
-        if (rank == 0) k_ring[(size_t)slot * G * a.dim_pad + e] = v;
+    auto put_k = [&](int g, int d, float v) {
+        const T r = from_f32<T>(v);
+        k_new[g * a.dim_pad + d] = r;
+        if (rank == 0) k_ring[((size_t)slot * G + g) * a.dim_pad + d] = r;
+    };
+    auto put_v = [&](int g, int d, float v) {
+        const T r = from_f32<T>(v);
+        v_new[g * a.vdim_pad + d] = r;
+        if (rank == 0) v_ring[((size_t)slot * G + g) * a.vdim_pad + d] = r;
+    };
+    if (a.dim % 4 == 0 && a.vdim % 4 == 0 && p.s.qkv_off % 4 == 0 && nq + nk + nv <= kStepThreads * 4 * kRowVecs) {
+        float4 x[kRowVecs];        // the row, read once
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int n = 0; n < kRowVecs; ++n) {
+            const int e = (tid + n * kStepThreads) * 4;
+            x[n] = e < nq + nk + nv ? ld_cg_f32x4(y + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int n = 0; n < kRowVecs; ++n) {
+            const int e = (tid + n * kStepThreads) * 4;
+            const float ss = x[n].x * x[n].x + x[n].y * x[n].y + x[n].z * x[n].z + x[n].w * x[n].w;
+            if (e < nq) sq += ss;
+            else if (e < nq + nk) sk += ss;
+        }
+        const RowFactors f = norm_factors(sq, sk, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
+#pragma unroll
+        for (int n = 0; n < kRowVecs; ++n) {
+            const int e = (tid + n * kStepThreads) * 4;
+            if (e >= nq + nk + nv) continue;
+            const float v[4] = {x[n].x, x[n].y, x[n].z, x[n].w};
+            if (e < nq) {
+                const int h = e / a.dim, d = e - h * a.dim;
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    put_query<T>(pl, sm, a.heads, h, d + c, v[c] * f.q * (a.q_norm ? __ldg(a.q_norm + e + c) : 1.f) * a.scale);
+            } else if (e < nq + nk) {
+                const int g = (e - nq) / a.dim, d = e - nq - g * a.dim;
+#pragma unroll
+                for (int c = 0; c < 4; ++c) put_k(g, d + c, v[c] * f.k * (a.k_norm ? __ldg(a.k_norm + e - nq + c) : 1.f));
+            } else {
+                const int g = (e - nq - nk) / a.vdim, d = e - nq - nk - g * a.vdim;
+#pragma unroll
+                for (int c = 0; c < 4; ++c) put_v(g, d + c, v[c]);
+            }
+        }
+    } else {
+        const RowFactors f = row_factors(y, nullptr, nq, nk, a.q_norm != nullptr, a.k_norm != nullptr, a.eps, s_tmp);
+        for (int e = tid; e < nq + nk + nv; e += kStepThreads) {
+            if (e < nq) put_query<T>(pl, sm, a.heads, e / a.dim, e % a.dim, y[e] * f.q * (a.q_norm ? __ldg(a.q_norm + e) : 1.f) * a.scale);
+            else if (e < nq + nk) put_k((e - nq) / a.dim, (e - nq) % a.dim, y[e] * f.k * (a.k_norm ? __ldg(a.k_norm + e - nq) : 1.f));
+            else put_v((e - nq - nk) / a.vdim, (e - nq - nk) % a.vdim, y[e]);
+        }
     }
-    for (int e = tid; e < G * a.vdim_pad; e += kStepThreads) {
-        const int g = e / a.vdim_pad, d = e - g * a.vdim_pad;
-        const T v = from_f32<T>(d < a.vdim ? y[nq + nk + g * a.vdim + d] : 0.f);
-        v_new[e] = v;
-        if (rank == 0) v_ring[(size_t)slot * G * a.vdim_pad + e] = v;
-    }
+    const int pd = a.dim_pad - a.dim, pv = a.vdim_pad - a.vdim;       // padding columns are zero
+    for (int e = tid; e < a.heads * pd; e += kStepThreads) put_query<T>(pl, sm, a.heads, e / pd, a.dim + e % pd, 0.f);
+    for (int e = tid; e < G * pd; e += kStepThreads) put_k(e / pd, a.dim + e % pd, 0.f);
+    for (int e = tid; e < G * pv; e += kStepThreads) put_v(e / pv, a.vdim + e % pv, 0.f);
     __syncthreads();
     float* p_gmem = static_cast<float*>(p.s.ws) + (size_t)rank * 2 * a.heads * pl.ldp;
     attend_query<T, float>(a, pl, sm, p_gmem, i, true, rank, p.cluster, p.s.out, p.s.left_scale);
@@ -74,6 +134,7 @@ template <typename T>
 __device__ void right_step(const StepParams& p, float* sm, float* s_tmp, int head) {
     const leankv_time_mix_t& a = p.right;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.dim, N = a.heads * d, c0 = head * d;
+    pdl_begin();
     float* s_r = sm;
     float* s_k = s_r + d;
     float* s_w = s_k + d;
@@ -128,7 +189,6 @@ template <typename T>
 __global__ void __launch_bounds__(kStepThreads) mixer_step_kernel(const __grid_constant__ StepParams p) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float s_tmp[32];
-    pdl_begin();
     const int first = p.has_left ? p.cluster : 0;
     if ((int)blockIdx.x < first) left_step<T>(p, sm, s_tmp, blockIdx.x);
     else if ((int)blockIdx.x - first < p.right.heads) right_step<T>(p, sm, s_tmp, blockIdx.x - first);
@@ -173,7 +233,7 @@ int launch_step(StepParams& p, cudaStream_t st) {
                 continue;
             }
         }
-        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(false, dim3(p.cluster), mixer_step_kernel<T>, dim3(grid),
+        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(true, dim3(p.cluster), mixer_step_kernel<T>, dim3(grid),
                                                  dim3(kStepThreads), smem, st, p));
         return LEANKV_OK;
     }

@@ -14,6 +14,7 @@ namespace {
 constexpr int kSlices = 8;       // lanes that share a column group, each with an eighth of the key channels
 constexpr int kColGroup = 4;     // value columns per thread: one read of r / k / w serves four columns
 constexpr int kMinPiece = 64;
+constexpr int kCtasPerSm = 4;
 
 // L: key channels per slice (a power of two from 4), kSlices * L >= dim.
 template <int L>
@@ -53,7 +54,7 @@ __device__ __forceinline__ void fetch8(const T* p, int n, bool vec, float (&v)[8
 }
 
 template <typename T, int L, bool OUT>
-__global__ void __launch_bounds__(ScanShape<L>::kThreads) time_mix_scan_kernel(const ScanParams<T> p, bool vec) {
+__global__ void __launch_bounds__(ScanShape<L>::kThreads, L <= 8 ? kCtasPerSm : L == 16 ? 2 : 1) time_mix_scan_kernel(const ScanParams<T> p, bool vec) {
     using Sh = ScanShape<L>;
     constexpr int kTok = Sh::kTok, kCols = Sh::kCols, kRow = Sh::kRow;
     __shared__ __align__(16) float s_r[OUT ? kTok : 1][kRow], s_k[kTok][kRow], s_w[kTok][kRow];
@@ -78,12 +79,8 @@ __global__ void __launch_bounds__(ScanShape<L>::kThreads) time_mix_scan_kernel(c
     // this thread's share of the staging: channels k8 .. k8 + 7 (and columns, for v) of token st_t
     const int st_t = tid / L, k8 = tid % L * 8, nk = d - k8;
     const int v_t = tid / (kCols / 8), v8 = tid % (kCols / 8) * 8;
-    float w0[8], u[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        w0[i] = i < nk ? __ldg(p.w0 + head * d + k8 + i) : 0.f;
-        u[i] = OUT && i < nk ? __ldg(p.u + head * d + k8 + i) : 0.f;
-    }
+    const float* w0 = p.w0 + head * d + k8;
+    const float* u = p.u + head * d + k8;
     float rr[8], kk[8], zz[8], vv[8], esum[8] = {};
     auto fetch = [&](int tb) {
         const bool on = tb + st_t < t1;
@@ -106,10 +103,10 @@ __global__ void __launch_bounds__(ScanShape<L>::kThreads) time_mix_scan_kernel(c
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const bool on = st_t < nt && h + i < nk;
-                const float e = on ? expf(zz[h + i] + w0[h + i]) : 0.f;      // -log of the decay
+                const float e = on ? expf(zz[h + i] + __ldg(w0 + h + i)) : 0.f;      // -log of the decay
                 w[i] = expf(-e);
                 if (!OUT) esum[h + i] += e;
-                else bonus = fmaf(rr[h + i] * u[h + i], kk[h + i], bonus);
+                else if (on) bonus = fmaf(rr[h + i] * __ldg(u + h + i), kk[h + i], bonus);
             }
             if (k < kSlices * L) {
                 *reinterpret_cast<float4*>(&s_k[st_t][at]) = make_float4(kk[h], kk[h + 1], kk[h + 2], kk[h + 3]);
@@ -214,30 +211,54 @@ __global__ void __launch_bounds__(256) time_mix_carry_kernel(const float* S, flo
     }
 }
 
-// out = out_scale * rms(o of the head) * norm * silu(g); one warp per (token, head).
+// out = out_scale * rms(o of the head) * norm * silu(g); a group of `lanes` lanes per (token, head), eight
+// channels per lane and pass (lanes: a power of two up to 32).
 template <typename T>
 __global__ void __launch_bounds__(256) time_mix_out_kernel(const float* o, const T* g, const float* norm, float eps,
-                                                           T* out, int out_ld, float out_scale, int rows, int heads,
-                                                           int dim) {
+                                                           T* out, int out_ld, float out_scale, long long groups, int heads,
+                                                           int dim, int lanes, bool vec) {
     pdl_begin();
-    const long long w = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
-    if (w >= (long long)rows * heads) return;
+    const long long at = ((long long)blockIdx.x * 256 + threadIdx.x) / lanes;
+    const int l = threadIdx.x % lanes;
+    const bool live = at < groups;
+    const long long w = live ? at : 0;
     const int t = (int)(w / heads), h = (int)(w - (long long)t * heads);
-    const size_t base = (size_t)t * heads * dim + (size_t)h * dim;
-    float ss = 0.f;
-    for (int i = lane; i < dim; i += 32) ss = fmaf(o[base + i], o[base + i], ss);
-    const float f = out_scale / sqrtf(warp_sum(ss) / (float)dim + eps);
-    for (int i = lane; i < dim; i += 32) {
-        const float gv = to_f32(g[base + i]);
-        out[(size_t)t * out_ld + h * dim + i] =
-            from_f32<T>(o[base + i] * f * __ldg(norm + h * dim + i) * gv * sigmoid_f32(gv));
+    const size_t base = (size_t)w * dim;
+    float v[8], ss = 0.f;
+    for (int i = l * 8; i < dim; i += lanes * 8) {
+        fetch8(o + base + i, dim - i, vec, v);
+#pragma unroll
+        for (int x = 0; x < 8; ++x) ss = fmaf(v[x], v[x], ss);
+    }
+    for (int s = lanes / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+    if (!live) return;
+    const float f = out_scale / sqrtf(ss / (float)dim + eps);
+    T* dst = out + (size_t)t * out_ld + h * dim;
+    for (int i = l * 8; i < dim; i += lanes * 8) {
+        float gv[8];
+        if (dim > lanes * 8) fetch8(o + base + i, dim - i, vec, v);      // else still in registers
+        fetch8(g + base + i, dim - i, vec, gv);
+#pragma unroll
+        for (int x = 0; x < 8; ++x)
+            if (i + x < dim) v[x] *= f * __ldg(norm + h * dim + i + x) * gv[x] * sigmoid_f32(gv[x]);
+        if (vec) {
+            T r[8];
+#pragma unroll
+            for (int x = 0; x < 8; ++x) r[x] = from_f32<T>(v[x]);
+            Raw8<T> raw;
+            memcpy(&raw, r, sizeof(raw));
+            *reinterpret_cast<Raw8<T>*>(dst + i) = raw;
+        } else {
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+                if (i + x < dim) dst[i + x] = from_f32<T>(v[x]);
+        }
     }
 }
 
 int pieces_for(int heads, int dim, int rows) {
     const int base = heads * ((dim + 63) / 64);
-    const int want = std::max(1, sm_count() * 4 / base);
+    const int want = std::max(1, sm_count() * kCtasPerSm / base);
     const int n = std::min(want, rows / kMinPiece);
     return n < 3 ? 1 : n;
 }
@@ -293,10 +314,13 @@ int rows_all(const leankv_time_mix_t& a, const void* r, const void* k, const voi
     else if (a.dim <= 8 * 16) rc = scan<T, 16>(a, r, k, v, z, ws, rows, st);
     else if (a.dim <= 8 * 32) rc = scan<T, 32>(a, r, k, v, z, ws, rows, st);
     if (rc) return rc;
-    const long long warps = (long long)rows * a.heads;
-    LEANKV_CUDA_TRY(launch_kernel(time_mix_out_kernel<T>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, st,
+    int lanes = 1;
+    while (lanes < 32 && lanes * 8 < a.dim) lanes *= 2;
+    const long long groups = (long long)rows * a.heads, threads = groups * lanes;
+    const bool vec = a.dim % 8 == 0 && out_ld % 8 == 0 && aligned16(ws) && aligned16(g) && aligned16(out);
+    LEANKV_CUDA_TRY(launch_kernel(time_mix_out_kernel<T>, dim3((unsigned)((threads + 255) / 256)), dim3(256), 0, st,
                                   static_cast<const float*>(ws), static_cast<const T*>(g), a.norm, a.eps,
-                                  static_cast<T*>(out), out_ld, out_scale, rows, a.heads, a.dim));
+                                  static_cast<T*>(out), out_ld, out_scale, groups, a.heads, a.dim, lanes, vec));
     return LEANKV_OK;
 }
 

@@ -106,22 +106,35 @@ __global__ void __launch_bounds__(kAppendThreads) window_pool_append_vec_kernel(
     for (int e = tid; e < G * pv; e += kAppendThreads) v[e / pv * a.vdim_pad + a.vdim + e % pv] = from_f32<T>(0.f);
 }
 
-// Blocks first .. : mean of the block's keys / values as the ring holds them. One CTA per block.
+// Blocks first .. : mean of the block's keys / values as the ring holds them. One CTA per block, eight columns
+// per thread (both paddings are multiples of 16).
 template <typename T>
 __global__ void __launch_bounds__(256) window_pool_blocks_kernel(const leankv_window_pool_t a, int first) {
     pdl_begin();
-    const int b = first + blockIdx.x, p0 = b * a.pool;
-    const float inv = (float)a.pool;
-    auto mean = [&](const void* ring, void* dst, int n) {
-        const T* src = static_cast<const T*>(ring);
-        for (int e = threadIdx.x; e < n; e += blockDim.x) {
-            float t = 0.f;
-            for (int i = 0; i < a.pool; ++i) t += to_f32(src[(size_t)((p0 + i) % a.ring) * n + e]);
-            static_cast<T*>(dst)[(size_t)b * n + e] = from_f32<T>(t / inv);
+    const int b = first + blockIdx.x, slot0 = (int)((long long)b * a.pool % a.ring);
+    const int nk = a.kv_heads * a.dim_pad, nv = a.kv_heads * a.vdim_pad;
+    const float size = (float)a.pool;
+    for (int e = threadIdx.x * 8; e < nk + nv; e += 256 * 8) {
+        const bool key = e < nk;
+        const int n = key ? nk : nv, col = key ? e : e - nk;
+        const T* src = static_cast<const T*>(key ? a.k_ring : a.v_ring) + col;
+        float t[8] = {};
+        int slot = slot0;
+#pragma unroll 8
+        for (int i = 0; i < a.pool; ++i) {
+            Raw8<T> r;
+            load8(src + (size_t)slot * n, r);
+            float v[8];
+            unpack8(r, v);
+#pragma unroll
+            for (int x = 0; x < 8; ++x) t[x] += v[x];
+            slot = slot + 1 == a.ring ? 0 : slot + 1;
         }
-    };
-    mean(a.k_ring, a.k_pool, a.kv_heads * a.dim_pad);
-    mean(a.v_ring, a.v_pool, a.kv_heads * a.vdim_pad);
+        T* dst = static_cast<T*>(key ? a.k_pool : a.v_pool) + (size_t)b * n + col;
+#pragma unroll
+        for (int x = 0; x < 8; x += 4)
+            store4(dst + x, make_float4(t[x] / size, t[x + 1] / size, t[x + 2] / size, t[x + 3] / size));
+    }
 }
 
 // One CTA per query row (the fp32 route, and shapes the tile kernel does not take).
@@ -134,6 +147,7 @@ __global__ void __launch_bounds__(kAttendThreads) window_pool_rows_kernel(const 
     const int t = blockIdx.x;
     const AttendPlan pl(a, kAttendThreads, n_max, kAttendSmemFloats);
     const T* row = q + (size_t)t * a.heads * a.dim_pad;
+    put_talk(a, pl, sm);
     for (int e = threadIdx.x; e < a.heads * a.dim_pad; e += kAttendThreads) {
         const int h = e / a.dim_pad;
         put_query<T>(pl, sm, a.heads, h, e - h * a.dim_pad, to_f32(row[e]) * a.scale);

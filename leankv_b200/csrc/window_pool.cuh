@@ -29,6 +29,7 @@ struct VisibleKeys {
 int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* out, int out_ld, float out_scale, int rows,
                             int start, cudaStream_t st);
 
+constexpr int kMaxCluster = 16;     // non-portable; 8 where the device does not place 16
 constexpr int kAttendHeads = 4;     // query heads a thread carries at once
 
 // Row length (elements) of bf16 operand rows in shared memory: 16-byte fragment reads of eight consecutive rows
@@ -54,7 +55,7 @@ struct AttendPlan {
         const int slots = a.kv_heads * (a.vdim_pad / 8);
         const int split = threads / slots > 1 ? threads / slots : 1;
         part = take(split > 1 ? split * a.kv_heads * kAttendHeads * a.vdim_pad : 0);
-        talk = take(a.talk && !half ? a.heads * ((a.heads + 7) / 8 * 8) : 0);
+        talk = take(a.talk ? a.heads * ((a.heads + 7) / 8 * 8) : 0);
         ldp = (n_local + 3) / 4 * 4 + 4;
         const int need = 2 * a.heads * ldp;
         p_in_smem = o + need <= max_floats;
@@ -170,21 +171,26 @@ __device__ __forceinline__ void scores(const leankv_window_pool_t& a, const Atte
     }
 }
 
+// The mixing matrix into shared memory, transposed and its rows padded to 8 ([from head][to head]).
+__device__ __forceinline__ void put_talk(const leankv_window_pool_t& a, const AttendPlan& pl, float* sm) {
+    if (a.talk == nullptr) return;
+    const int H = a.heads, Hr = (H + 7) / 8 * 8;
+    for (int e = threadIdx.x; e < H * Hr; e += blockDim.x) {
+        const int h = e / H, g = e - h * H;
+        sm[pl.talk + g * Hr + h] = h < H ? __ldg(a.talk + e) : 0.f;
+    }
+}
+
 // pm[h][j] = sum over g of talk[h][g] * (p[g][j] * factor[g]). fp32 on FMA units.
 __device__ __forceinline__ void mix_heads(const leankv_window_pool_t& a, const AttendPlan& pl, float* sm,
                                           const float* factor, const float* p, float* pm, int n, float) {
     const int H = a.heads, Hr = (H + 7) / 8 * 8, nb = Hr / 8;
-    for (int e = threadIdx.x; e < H * Hr; e += blockDim.x) {      // talk^T, rows padded, times the factor
-        const int g = e / Hr, h = e - g * Hr;
-        sm[pl.talk + e] = h < H ? __ldg(a.talk + h * H + g) * factor[g] : 0.f;
-    }
-    __syncthreads();
     for (int e = threadIdx.x; e < n * nb; e += blockDim.x) {
         const int hb = e / n, jl = e - hb * n;
         float acc[8] = {};
         const float* tk = sm + pl.talk + hb * 8;
         for (int g = 0; g < H; ++g) {
-            const float w = p[g * pl.ldp + jl];
+            const float w = p[g * pl.ldp + jl] * factor[g];
 #pragma unroll
             for (int x = 0; x < 8; ++x) acc[x] = fmaf(tk[g * Hr + x], w, acc[x]);
         }
@@ -196,15 +202,15 @@ __device__ __forceinline__ void mix_heads(const leankv_window_pool_t& a, const A
 
 // The same on tensor cores: output heads as rows, keys as columns, both operands as high + low bf16 parts
 // (the product of the two low parts, 2^-16 of the result, is dropped).
-__device__ __forceinline__ void mix_heads(const leankv_window_pool_t& a, const AttendPlan& pl, float*,
+__device__ __forceinline__ void mix_heads(const leankv_window_pool_t& a, const AttendPlan& pl, float* sm,
                                           const float* factor, const float* p, float* pm, int n, bf16) {
-    const int H = a.heads, ht = (H + 15) / 16, kt = (n + 7) / 8;
+    const int H = a.heads, Hr = (H + 7) / 8 * 8, ht = (H + 15) / 16, kt = (n + 7) / 8;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, gl = lane >> 2, t = lane & 3;
     for (int e = warp; e < ht * kt; e += nw) {
         const int m0 = (e / kt) * 16, j = (e % kt) * 8 + gl;
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         for (int g0 = 0; g0 < H; g0 += 16) {
-            auto tk = [&](int h, int g) { return h < H && g < H ? __ldg(a.talk + h * H + g) : 0.f; };
+            auto tk = [&](int h, int g) { return h < H && g < H ? sm[pl.talk + g * Hr + h] : 0.f; };
             auto wt = [&](int g) { return g < H && j < n ? p[g * pl.ldp + j] * factor[g] : 0.f; };
             const int c = g0 + 2 * t;
             uint32_t ah[4], al[4], bh[2], bl[2];
@@ -228,7 +234,7 @@ __device__ __forceinline__ void mix_heads(const leankv_window_pool_t& a, const A
 
 // Attention of position i over this CTA's share (rank of C) of its visible keys; scores, softmax and the mix
 // across heads in fp32 (bf16 operands enter as exact parts).
-// sm: shared memory laid out by `pl`, with the normed queries in place (put_query). If `fresh`, the key / value
+// sm: shared memory laid out by `pl`, with the normed queries (put_query) and the mix (put_talk) in place. If `fresh`, the key / value
 // rows of position i are those at sm[pl.knew] / sm[pl.vnew] instead of the ring's (not written yet).
 // p_gmem: weight buffers (2 * heads * ldp floats of this CTA) when they do not fit into shared memory.
 // Writes out[h * vdim + d] times out_scale; with C > 1 the CTAs are a cluster and each writes its share.
@@ -243,13 +249,15 @@ __device__ void attend_query(const leankv_window_pool_t& a, const AttendPlan& pl
     float* pm = a.talk ? p + H * ldp : p;
     float* stat = sm + pl.stat;            // local max | local sum | factor of this CTA's exponentials
 
+    const int slot_w0 = vis.w0 % a.ring;
     // row of local key jl in the pooled blocks, the ring, or the fresh row
     auto row = [&](int jl, int g, const void* pool, const void* ring, int fresh_at, int width) -> const T* {
         const int j = j0 + jl;
         if (j < vis.n_blk) return static_cast<const T*>(pool) + ((size_t)j * G + g) * width;
-        const int pos = vis.w0 + j - vis.n_blk;
-        if (fresh && pos == i) return reinterpret_cast<const T*>(sm + fresh_at) + g * width;
-        return static_cast<const T*>(ring) + ((size_t)(pos % a.ring) * G + g) * width;
+        if (fresh && j == vis.n - 1) return reinterpret_cast<const T*>(sm + fresh_at) + g * width;
+        int slot = slot_w0 + j - vis.n_blk;              // a window fits into the ring once
+        if (slot >= a.ring) slot -= a.ring;
+        return static_cast<const T*>(ring) + ((size_t)slot * G + g) * width;
     };
     if (n > 0) scores(a, pl, sm, p, n, [&](int jl, int g) { return row(jl, g, a.k_pool, a.k_ring, pl.knew, dp); }, T{});
     __syncthreads();
@@ -274,11 +282,18 @@ __device__ void attend_query(const leankv_window_pool_t& a, const AttendPlan& pl
         float m = -INFINITY, l = 0.f;
         if (C > 1) {
             auto cl = cg::this_cluster();
-            for (int r = 0; r < C; ++r) m = fmaxf(m, cl.map_shared_rank(stat, r)[h]);
-            for (int r = 0; r < C; ++r) {
-                const float* s = cl.map_shared_rank(stat, r);
-                if (s[H + h] > 0.f) l += s[H + h] * expf(s[h] - m);
+            float mr[kMaxCluster], lr[kMaxCluster];      // all remote reads in flight together
+#pragma unroll
+            for (int r = 0; r < kMaxCluster; ++r) {
+                const float* s = cl.map_shared_rank(stat, r < C ? r : 0);
+                mr[r] = s[h];
+                lr[r] = r < C ? s[H + h] : 0.f;
             }
+#pragma unroll
+            for (int r = 0; r < kMaxCluster; ++r) m = fmaxf(m, mr[r]);
+#pragma unroll
+            for (int r = 0; r < kMaxCluster; ++r)
+                if (lr[r] > 0.f) l += lr[r] * expf(mr[r] - m);
         } else {
             m = stat[h];
             l = stat[H + h];
@@ -300,7 +315,7 @@ __device__ void attend_query(const leankv_window_pool_t& a, const AttendPlan& pl
     // ---- weights times values: a thread owns 8 value columns of one kv head and a range of keys ----
     const int per_g = vp / 8, slots = G * per_g;
     const int split = nt / slots > 1 ? nt / slots : 1;
-    const int per_split = ((n + split - 1) / split + 3) / 4 * 4;
+    const int per_split = ((n + split - 1) / split + 3) / 4 * 4;      // 16-byte reads of the weights
     float* s_out = sm + pl.out;
     for (int hb = 0; hb < rep; hb += kAttendHeads) {
         const int nh = min(kAttendHeads, rep - hb);
@@ -309,28 +324,35 @@ __device__ void attend_query(const leankv_window_pool_t& a, const AttendPlan& pl
             float acc[kAttendHeads][8] = {};
             const float* w = pm + (g * rep + hb) * ldp;
             const int e0 = min(n, ks * per_split), e1 = min(n, e0 + per_split);
-            for (int jl = e0; jl < e1; jl += 4) {
-                Raw8<T> raw[4];
+            constexpr int kBatch = sizeof(T) == 2 ? 8 : 4;      // value rows in flight per thread
+            for (int jb = e0; jb < e1; jb += kBatch) {
+                Raw8<T> raw[kBatch];
 #pragma unroll
-                for (int x = 0; x < 4; ++x) load8(row(min(jl + x, e1 - 1), g, a.v_pool, a.v_ring, pl.vnew, vp) + d, raw[x]);
-                float wr[kAttendHeads][4];
+                for (int x = 0; x < kBatch; ++x)
+                    load8(row(min(jb + x, e1 - 1), g, a.v_pool, a.v_ring, pl.vnew, vp) + d, raw[x]);
 #pragma unroll
-                for (int r = 0; r < kAttendHeads; ++r)
-                    if (r < nh) {
-                        const float4 w4 = *reinterpret_cast<const float4*>(w + r * ldp + jl);
-                        wr[r][0] = w4.x; wr[r][1] = w4.y; wr[r][2] = w4.z; wr[r][3] = w4.w;
-                    }
+                for (int q = 0; q < kBatch; q += 4) {
+                    const int jl = jb + q;
+                    if (jl >= e1) break;
+                    float wr[kAttendHeads][4];
 #pragma unroll
-                for (int x = 0; x < 4; ++x)
-                    if (jl + x < e1) {
-                        float vv[8];
-                        unpack8(raw[x], vv);
+                    for (int r = 0; r < kAttendHeads; ++r)
+                        if (r < nh) {
+                            const float4 w4 = *reinterpret_cast<const float4*>(w + r * ldp + jl);
+                            wr[r][0] = w4.x; wr[r][1] = w4.y; wr[r][2] = w4.z; wr[r][3] = w4.w;
+                        }
 #pragma unroll
-                        for (int r = 0; r < kAttendHeads; ++r)
-                            if (r < nh)
+                    for (int x = 0; x < 4; ++x)
+                        if (jl + x < e1) {
+                            float vv[8];
+                            unpack8(raw[q + x], vv);
 #pragma unroll
-                                for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(wr[r][x], vv[c], acc[r][c]);
-                    }
+                            for (int r = 0; r < kAttendHeads; ++r)
+                                if (r < nh)
+#pragma unroll
+                                    for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(wr[r][x], vv[c], acc[r][c]);
+                        }
+                }
             }
             float* dst = split > 1 ? sm + pl.part + (size_t)(ks * G + g) * kAttendHeads * vp : nullptr;
 #pragma unroll
@@ -359,7 +381,11 @@ __device__ void attend_query(const leankv_window_pool_t& a, const AttendPlan& pl
         float t = 0.f;
         if (C > 1) {
             auto cl = cg::this_cluster();
-            for (int r = 0; r < C; ++r) t += cl.map_shared_rank(s_out, r)[h * vp + d];
+            float part[kMaxCluster];
+#pragma unroll
+            for (int r = 0; r < kMaxCluster; ++r) part[r] = r < C ? cl.map_shared_rank(s_out, r)[h * vp + d] : 0.f;
+#pragma unroll
+            for (int r = 0; r < kMaxCluster; ++r) t += part[r];
         } else {
             t = s_out[h * vp + d];
         }

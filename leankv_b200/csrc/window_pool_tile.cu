@@ -40,13 +40,16 @@ __device__ __forceinline__ float ex2(float x) {
     return y;
 }
 
-template <int HPW, int DVT>
-__global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_tile_kernel(const __grid_constant__ TileParams p) {
+// HPW query heads per warp, NB blocks of 32 dimensions and DVT tiles of 16 value columns; EXACT: the sizes are
+// those, otherwise at most those.
+template <int HPW, int NB, int DVT, bool EXACT>
+__global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_kernel(const __grid_constant__ TileParams p) {
     extern __shared__ __align__(128) unsigned char smem[];
     pdl_begin();
     const leankv_window_pool_t& a = p.a;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int H = a.heads, G = a.kv_heads, rep = H / G, dp = a.dim_pad, vp = a.vdim_pad, nb = p.nb, KS = p.ks;
+    const int H = a.heads, G = a.kv_heads, rep = H / G, KS = p.ks;
+    const int dp = EXACT ? NB * 32 : a.dim_pad, vp = EXACT ? DVT * 16 : a.vdim_pad, nb = EXACT ? NB : p.nb;
     const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kQ;           // the longest rows first
     const int nq = min(kQ, p.rows - q0), i0 = p.start + q0, iL = i0 + nq - 1;
     const VisibleKeys first(i0, a.size, a.pool), last(iL, a.size, a.pool);
@@ -99,52 +102,55 @@ __global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_t
     const bf16* k_pool = static_cast<const bf16*>(a.k_pool);
 
     // row of a tile's key r (clamped to the keys that exist): index into the pooled blocks or the ring
-    struct TileRows { bool pooled; int base, n, slot0; };
+    struct TileRows { bool pooled; int n, slot0; };
+    const int ring0 = tok0 % a.ring;
     auto rows_of = [&](int tile) {
         TileRows tr;
         tile = min(tile, NT - 1);
         tr.pooled = tile < TB;
-        tr.base = (tr.pooled ? tile : tile - TB) * 16;
-        tr.n = (tr.pooled ? last.n_blk : ntok) - tr.base;
-        tr.slot0 = tr.pooled ? tr.base : (tok0 + tr.base) % a.ring;
+        const int base = (tr.pooled ? tile : tile - TB) * 16;
+        tr.n = (tr.pooled ? last.n_blk : ntok) - base - 1;
+        tr.slot0 = tr.pooled ? base : ring0 + base;              // the tokens of a portion fit into the ring once
         return tr;
     };
     auto index_of = [&](const TileRows& tr, int r) {
-        int s = tr.slot0 + min(r, tr.n - 1);
+        int s = tr.slot0 + min(r, tr.n);
         if (!tr.pooled && s >= a.ring) s -= a.ring;
         return s;
     };
-    uint4 x0[kMaxNb], x1[kMaxNb];
-    auto load_keys = [&](int tile) {
+    struct Keys { uint4 x0[NB], x1[NB]; };
+    const size_t k_stride = (size_t)G * dp;
+    auto load_keys = [&](int tile, Keys& k) {
         const TileRows tr = rows_of(tile);
         const bf16* src = (tr.pooled ? k_pool : k_ring) + (size_t)kv * dp + t * 8;
-        const bf16* r0 = src + (size_t)index_of(tr, g) * G * dp;
-        const bf16* r1 = src + (size_t)index_of(tr, g + 8) * G * dp;
+        const bf16* r0 = src + index_of(tr, g) * k_stride;
+        const bf16* r1 = src + index_of(tr, g + 8) * k_stride;
 #pragma unroll
-        for (int b = 0; b < kMaxNb; ++b)
+        for (int b = 0; b < NB; ++b)
             if (b < nb) {
                 const bool on = b * 32 + t * 8 < dp;
-                x0[b] = on ? *reinterpret_cast<const uint4*>(r0 + b * 32) : make_uint4(0, 0, 0, 0);
-                x1[b] = on ? *reinterpret_cast<const uint4*>(r1 + b * 32) : make_uint4(0, 0, 0, 0);
+                k.x0[b] = on ? *reinterpret_cast<const uint4*>(r0 + b * 32) : make_uint4(0, 0, 0, 0);
+                k.x1[b] = on ? *reinterpret_cast<const uint4*>(r1 + b * 32) : make_uint4(0, 0, 0, 0);
             }
     };
+    const uint4* q_frag = reinterpret_cast<const uint4*>(smem) + h0 * nb * 32 + lane;
     float s[HPW][4];
-    auto score = [&](int tile) {        // scaled to base-2 exponents, -inf where the query does not see the key
+    auto score = [&](int tile, const Keys& k) {        // -inf where the query does not see the key
 #pragma unroll
         for (int h = 0; h < HPW; ++h)
 #pragma unroll
             for (int x = 0; x < 4; ++x) s[h][x] = 0.f;
 #pragma unroll
-        for (int b = 0; b < kMaxNb; ++b)
+        for (int b = 0; b < NB; ++b)
             if (b < nb) {
+                uint4 y[HPW];
 #pragma unroll
-                for (int h = 0; h < HPW; ++h) {
-                    const uint4 y = reinterpret_cast<const uint4*>(smem)[((h0 + h) * nb + b) * 32 + lane];
-                    mma_bf16(s[h], x0[b].x, x1[b].x, x0[b].y, x1[b].y, y.x, y.y);
-                    mma_bf16(s[h], x0[b].z, x1[b].z, x0[b].w, x1[b].w, y.z, y.w);
-                }
+                for (int h = 0; h < HPW; ++h) y[h] = q_frag[(h * nb + b) * 32];
+#pragma unroll
+                for (int h = 0; h < HPW; ++h) mma_bf16(s[h], k.x0[b].x, k.x1[b].x, k.x0[b].y, k.x1[b].y, y[h].x, y[h].y);
+#pragma unroll
+                for (int h = 0; h < HPW; ++h) mma_bf16(s[h], k.x0[b].z, k.x1[b].z, k.x0[b].w, k.x1[b].w, y[h].z, y[h].w);
             }
-        bool see[4] = {true, true, true, true};
         const bool pooled = tile < TB;
         const int base = pooled ? tile * 16 : tok0 + (tile - TB) * 16;
         const bool all = tile < NT && (pooled ? base + 15 < first.n_blk : base >= last.w0 && base + 15 <= i0);
@@ -152,34 +158,57 @@ __global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_t
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int at = base + g + (x < 2 ? 0 : 8), qx = x & 1;
-                see[x] = tile < NT && (pooled ? at < nbq[qx] : at >= w0q[qx] && at <= iq[qx]);
+                const bool see = tile < NT && (pooled ? at < nbq[qx] : at >= w0q[qx] && at <= iq[qx]);
+#pragma unroll
+                for (int h = 0; h < HPW; ++h) s[h][x] = see ? s[h][x] : -INFINITY;
             }
         }
-#pragma unroll
-        for (int h = 0; h < HPW; ++h)
-#pragma unroll
-            for (int x = 0; x < 4; ++x) s[h][x] = see[x] ? s[h][x] * c : -INFINITY;
     };
 
     // ---- pass 1: log2 of the softmax denominators ----
     float lse[HPW][2];
     {
+        // m: a reference exponent per (head, query) and lane, raised only when a score exceeds it by kSlack: the
+        // exponentials stay below 2^kSlack and most tiles need no rescaling
+        constexpr float kSlack = 12.f;
         float m[HPW][2], l[HPW][2];
 #pragma unroll
         for (int h = 0; h < HPW; ++h) m[h][0] = m[h][1] = -1e30f, l[h][0] = l[h][1] = 0.f;
-        if (worker) {
-            load_keys(ks);
-            for (int tile = ks; tile < NT; tile += KS) {
-                score(tile);
-                load_keys(tile + KS);
+        auto count = [&]() {
+            bool raise = false;
+#pragma unroll
+            for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                for (int x = 0; x < 2; ++x) raise = raise || fmaxf(s[h][x], s[h][x + 2]) * c > m[h][x] + kSlack;
+            if (__any_sync(0xffffffffu, raise)) {
 #pragma unroll
                 for (int h = 0; h < HPW; ++h)
 #pragma unroll
                     for (int x = 0; x < 2; ++x) {
-                        const float mn = fmaxf(m[h][x], fmaxf(s[h][x], s[h][x + 2]));
-                        l[h][x] = l[h][x] * ex2(m[h][x] - mn) + ex2(s[h][x] - mn) + ex2(s[h][x + 2] - mn);
+                        const float mn = fmaxf(m[h][x], fmaxf(s[h][x], s[h][x + 2]) * c);
+                        l[h][x] *= ex2(m[h][x] - mn);
                         m[h][x] = mn;
                     }
+            }
+#pragma unroll
+            for (int h = 0; h < HPW; ++h)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) l[h][x & 1] += ex2(fmaf(s[h][x], c, -m[h][x & 1]));
+        };
+        if (worker) {
+            Keys ka, kb;
+            load_keys(ks, ka);
+            load_keys(ks + KS, kb);
+#pragma unroll 1
+            for (int tile = ks; tile < NT; tile += 2 * KS) {
+                score(tile, ka);
+                load_keys(tile + 2 * KS, ka);
+                count();
+                if (tile + KS < NT) {
+                    score(tile + KS, kb);
+                    load_keys(tile + 3 * KS, kb);
+                    count();
+                }
             }
         }
         float* stat = reinterpret_cast<float*>(smem + p.off_stat);       // [KS][H][8][2]
@@ -228,30 +257,36 @@ __global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_t
     unsigned char* vbuf = smem + p.off_v + (size_t)warp * 16 * p.v_row;
     const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(vbuf);
     uint32_t* pm = reinterpret_cast<uint32_t*>(smem + p.off_pm);
-    if (worker) load_keys(ks);
+    Keys keys;
+    if (worker) load_keys(ks, keys);
+    const int v_per = vp / 8, v_r0 = lane / v_per, v_c0 = lane % v_per, v_dr = 32 / v_per, v_dc = 32 % v_per;
+    const size_t v_stride = (size_t)G * vp;
+#pragma unroll 1
     for (int base = 0; base < NT; base += KS) {
         const int tile = base + ks;
         if (worker) {
             {       // this tile's values start their way
                 const TileRows tr = rows_of(tile);
                 const bf16* src = static_cast<const bf16*>(tr.pooled ? a.v_pool : a.v_ring) + (size_t)kv * vp;
-                const int per = vp / 8;
-                for (int e = lane; e < 16 * per; e += 32) {
-                    const int r = e / per, ch = e - r * per;
-                    const bf16* from = src + (size_t)index_of(tr, r) * G * vp + ch * 8;
+                int r = v_r0, ch = v_c0;
+                while (r < 16) {
+                    const bf16* from = src + index_of(tr, r) * v_stride + ch * 8;
                     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vaddr + r * p.v_row + ch * 16), "l"(from)
                                  : "memory");
+                    r += v_dr;
+                    ch += v_dc;
+                    if (ch >= v_per) { ch -= v_per; ++r; }
                 }
                 asm volatile("cp.async.commit_group;" ::: "memory");
             }
-            score(tile);
-            if (base + KS < NT) load_keys(tile + KS);
+            score(tile, keys);
+            if (base + KS < NT) load_keys(tile + KS, keys);
             // normalised weights as high + low bf16: [key][query][head / 4] {4 high, 4 low}
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 float w[HPW];
 #pragma unroll
-                for (int h = 0; h < HPW; ++h) w[h] = ex2(s[h][x] - lse[h][x & 1]);
+                for (int h = 0; h < HPW; ++h) w[h] = ex2(fmaf(s[h][x], c, -lse[h][x & 1]));
                 const int key = ks * 16 + g + (x < 2 ? 0 : 8), qq = 2 * t + (x & 1);
                 unsigned char* dst = smem + p.off_p + key * p.p_key + qq * p.p_row + (h0 >> 2) * 16;
                 if constexpr (HPW == 4) {
@@ -277,29 +312,30 @@ __global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_t
             }
         }
         __syncthreads();
-        // mix across heads, two keys at a time: [head][query][key] bf16
-        for (int pair = warp; pair < 8 * KS; pair += kWarps) {
+        // mix across heads, two keys and 16 output heads at a time: [head][query][key] bf16
+        for (int e = warp; e < 8 * KS * MT; e += kWarps) {
+            const int pair = e / MT, mt = e - pair * MT;
             const unsigned char* src = smem + p.off_p + (size_t)pair * 2 * p.p_key + g * p.p_row + t * 16;
-            for (int mt = 0; mt < MT; ++mt) {
-                float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-                for (int kt = 0; kt < MT; ++kt) {
-                    const uint4* tf = reinterpret_cast<const uint4*>(smem + p.off_t) + (mt * MT + kt) * 64 + lane;
-                    const uint4 ah = tf[0], al = tf[32];
-                    const uint4 b0 = *reinterpret_cast<const uint4*>(src + kt * 64);
-                    const uint4 b1 = *reinterpret_cast<const uint4*>(src + p.p_key + kt * 64);
-                    mma_bf16(d0, ah.x, ah.y, ah.z, ah.w, b0.x, b0.y);
-                    mma_bf16(d1, ah.x, ah.y, ah.z, ah.w, b1.x, b1.y);
-                    mma_bf16(d0, ah.x, ah.y, ah.z, ah.w, b0.z, b0.w);
-                    mma_bf16(d1, ah.x, ah.y, ah.z, ah.w, b1.z, b1.w);
-                    mma_bf16(d0, al.x, al.y, al.z, al.w, b0.x, b0.y);
-                    mma_bf16(d1, al.x, al.y, al.z, al.w, b1.x, b1.y);
-                }
-#pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    const int h = mt * 16 + g + (x < 2 ? 0 : 8);
-                    if (h < H) pm[h * p.pm_h + (2 * t + (x & 1)) * p.pm_q + pair] = pack_bf16(d0[x], d1[x]);
-                }
+            float d0[2][4] = {}, d1[2][4] = {};
+#pragma unroll 2
+            for (int kt = 0; kt < MT; ++kt) {
+                const uint4* tf = reinterpret_cast<const uint4*>(smem + p.off_t) + (mt * MT + kt) * 64 + lane;
+                const uint4 ah = tf[0], al = tf[32];
+                const uint4 b0 = *reinterpret_cast<const uint4*>(src + kt * 64);
+                const uint4 b1 = *reinterpret_cast<const uint4*>(src + p.p_key + kt * 64);
+                mma_bf16(d0[0], ah.x, ah.y, ah.z, ah.w, b0.x, b0.y);
+                mma_bf16(d1[0], ah.x, ah.y, ah.z, ah.w, b1.x, b1.y);
+                mma_bf16(d0[1], ah.x, ah.y, ah.z, ah.w, b0.z, b0.w);
+                mma_bf16(d1[1], ah.x, ah.y, ah.z, ah.w, b1.z, b1.w);
+                mma_bf16(d0[1], al.x, al.y, al.z, al.w, b0.x, b0.y);
+                mma_bf16(d1[1], al.x, al.y, al.z, al.w, b1.x, b1.y);
             }
+            uint32_t* dst = pm + (mt * 16 + g) * p.pm_h + 2 * t * p.pm_q + pair;
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+                if (mt * 16 + g + (x < 2 ? 0 : 8) < H)
+                    dst[(x < 2 ? 0 : 8) * p.pm_h + (x & 1) * p.pm_q] =
+                        pack_bf16(d0[0][x] + d0[1][x], d1[0][x] + d1[1][x]);
         }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
@@ -369,13 +405,20 @@ __global__ void __launch_bounds__(kThreads, HPW* DVT <= 8 ? 2 : 1) window_pool_t
     }
 }
 
-template <int HPW, int DVT>
+template <int HPW, int NB, int DVT, bool EXACT>
 int launch(const TileParams& p, size_t smem, cudaStream_t st) {
-    LEANKV_CUDA_TRY(cudaFuncSetAttribute(window_pool_tile_kernel<HPW, DVT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)smem));
-    LEANKV_CUDA_TRY(launch_kernel(window_pool_tile_kernel<HPW, DVT>, dim3((p.rows + kQ - 1) / kQ), dim3(kThreads), smem, st,
-                                  p));
+    auto kernel = window_pool_tile_kernel<HPW, NB, DVT, EXACT>;
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LEANKV_CUDA_TRY(launch_kernel(kernel, dim3((p.rows + kQ - 1) / kQ), dim3(kThreads), smem, st, p));
     return LEANKV_OK;
+}
+
+template <int HPW>
+int launch_sizes(const TileParams& p, size_t smem, cudaStream_t st) {
+    const int dp = p.a.dim_pad, vp = p.a.vdim_pad;
+    if (dp == 64 && vp == 64) return launch<HPW, 2, 4, true>(p, smem, st);
+    if (dp == 128 && vp == 128) return launch<HPW, 4, 8, true>(p, smem, st);
+    return launch<HPW, 4, 8, false>(p, smem, st);
 }
 
 }  // namespace
@@ -412,12 +455,11 @@ int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* 
     p.off_pm = take(a.heads * p.pm_h * 4);
     p.off_v = take(std::max(kWarps * 16 * p.v_row, p.ks > 1 ? a.heads * a.vdim_pad * kQ * 4 : 0));
     if (at > 227 * 1024) return LEANKV_EUNSUPPORTED;
-    const bool narrow = a.vdim_pad <= 64;
     switch (hpw) {
-        case 1: return narrow ? launch<1, 4>(p, at, st) : launch<1, 8>(p, at, st);
-        case 2: return narrow ? launch<2, 4>(p, at, st) : launch<2, 8>(p, at, st);
-        case 3: return narrow ? launch<3, 4>(p, at, st) : launch<3, 8>(p, at, st);
-        default: return narrow ? launch<4, 4>(p, at, st) : launch<4, 8>(p, at, st);
+        case 1: return launch_sizes<1>(p, at, st);
+        case 2: return launch_sizes<2>(p, at, st);
+        case 3: return launch_sizes<3>(p, at, st);
+        default: return launch_sizes<4>(p, at, st);
     }
 }
 
