@@ -18,7 +18,7 @@ struct StepParams {
     leankv_window_pool_t left;
     leankv_time_mix_t right;
     leankv_mixer_step_t s;
-    int has_left, has_right, n_max, cluster;
+    int has_left, has_right, n_max, cluster, norms_aligned;
 };
 
 constexpr int kRowVecs = 6;        // float4s of the projection row a thread keeps: rows up to 12288 columns
@@ -63,7 +63,7 @@ __device__ void left_step(const StepParams& p, float* sm, float* s_tmp, int rank
         v_new[g * a.vdim_pad + d] = r;
         if (rank == 0) v_ring[((size_t)slot * G + g) * a.vdim_pad + d] = r;
     };
-    if (a.dim % 4 == 0 && a.vdim % 4 == 0 && p.s.qkv_off % 4 == 0 && nq + nk + nv <= kStepThreads * 4 * kRowVecs) {
+    if (a.dim % 4 == 0 && a.vdim % 4 == 0 && p.s.qkv_off % 4 == 0 && p.norms_aligned && nq + nk + nv <= kStepThreads * 4 * kRowVecs) {
         float4 x[kRowVecs];        // the row, read once
         float sq = 0.f, sk = 0.f;
 #pragma unroll
@@ -83,20 +83,23 @@ __device__ void left_step(const StepParams& p, float* sm, float* s_tmp, int rank
         for (int n = 0; n < kRowVecs; ++n) {
             const int e = (tid + n * kStepThreads) * 4;
             if (e >= nq + nk + nv) continue;
-            const float v[4] = {x[n].x, x[n].y, x[n].z, x[n].w};
-            if (e < nq) {
-                const int h = e / a.dim, d = e - h * a.dim;
-#pragma unroll
-                for (int c = 0; c < 4; ++c)
-                    put_query<T>(pl, sm, a.heads, h, d + c, v[c] * f.q * (a.q_norm ? __ldg(a.q_norm + e + c) : 1.f) * a.scale);
-            } else if (e < nq + nk) {
-                const int g = (e - nq) / a.dim, d = e - nq - g * a.dim;
-#pragma unroll
-                for (int c = 0; c < 4; ++c) put_k(g, d + c, v[c] * f.k * (a.k_norm ? __ldg(a.k_norm + e - nq + c) : 1.f));
+            const bool is_q = e < nq, is_k = !is_q && e < nq + nk;
+            const int at = is_q ? e : is_k ? e - nq : e - nq - nk, width = is_q || is_k ? a.dim : a.vdim;
+            const int h = at / width, d = at - h * width;
+            const float* w = is_q ? a.q_norm : is_k ? a.k_norm : nullptr;
+            const float fac = is_q ? f.q * a.scale : is_k ? f.k : 1.f;
+            float4 v = make_float4(x[n].x * fac, x[n].y * fac, x[n].z * fac, x[n].w * fac);
+            if (w != nullptr) {
+                const float4 g = *reinterpret_cast<const float4*>(w + at);
+                v.x *= g.x; v.y *= g.y; v.z *= g.z; v.w *= g.w;
+            }
+            if (is_q) {
+                put_query4<T>(pl, sm, a.heads, h, d, v);
             } else {
-                const int g = (e - nq - nk) / a.vdim, d = e - nq - nk - g * a.vdim;
-#pragma unroll
-                for (int c = 0; c < 4; ++c) put_v(g, d + c, v[c]);
+                const int to = h * (is_k ? a.dim_pad : a.vdim_pad) + d;
+                store4((is_k ? k_new : v_new) + to, v);
+                if (rank == 0)
+                    store4((is_k ? k_ring : v_ring) + (size_t)slot * G * (is_k ? a.dim_pad : a.vdim_pad) + to, v);
             }
         }
     } else {
@@ -273,6 +276,7 @@ extern "C" int leankv_mixer_step(const leankv_window_pool_t* left, const leankv_
         if (leankv_mixer_step_workspace_bytes(left, s->max_pos) > (s->ws ? s->ws_bytes : 0)) return LEANKV_EWORKSPACE;
         p.left = *left;
         p.has_left = 1;
+        p.norms_aligned = aligned16(left->q_norm) && aligned16(left->k_norm) && aligned16(s->y);
         p.n_max = keys_bound(*left, s->max_pos);
         dtype = left->dtype;
     }

@@ -53,15 +53,8 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const leankv_s
     }
 }
 
-// The same with 4-element accesses and rows in registers (width % 4 == 0, width <= kRowThreads * 4 * NV). A CTA
-// walks `per_cta` consecutive rows and keeps the row above, so only its first row is normed twice.
 template <typename T>
-__device__ __forceinline__ void store4(T* p, const float (&v)[4]) {
-    if constexpr (sizeof(T) == 4)
-        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    else
-        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
-}
+__device__ __forceinline__ void store4(T* p, const float (&v)[4]) { leankv::store4(p, make_float4(v[0], v[1], v[2], v[3])); }
 __device__ __forceinline__ void fetch4(const float* p, float (&v)[4]) {
     const float4 a = *reinterpret_cast<const float4*>(p);
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
@@ -72,6 +65,8 @@ __device__ __forceinline__ void fetch4(const bf16* p, float (&v)[4]) {
     v[2] = __uint_as_float(a.y << 16); v[3] = __uint_as_float(a.y & 0xffff0000u);
 }
 
+// The same with 4-element accesses and rows in registers (width % 4 == 0, width <= kRowThreads * 4 * NV). A CTA
+// walks `per_cta` consecutive rows and keeps the row above, so only its first row is normed twice.
 template <typename T, typename D, int NV>
 __global__ void __launch_bounds__(kRowThreads) stream_norm_vec_kernel(const leankv_stream_norm_t a, int per_cta) {
     __shared__ float s_tmp[32];

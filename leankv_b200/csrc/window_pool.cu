@@ -43,11 +43,6 @@ __global__ void __launch_bounds__(kAppendThreads) window_pool_append_kernel(cons
 
 // The same with 4-element accesses, the row in registers (dim, vdim and ld multiples of 4, at most
 // kAppendThreads * 4 * NV columns).
-template <typename T>
-__device__ __forceinline__ void store4(T* p, float4 v) {
-    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = v;
-    else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-}
 template <typename T, int NV>
 __global__ void __launch_bounds__(kAppendThreads) window_pool_append_vec_kernel(const leankv_window_pool_t a,
                                                                                 const float* qkv, int ld,

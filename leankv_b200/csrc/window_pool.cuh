@@ -84,6 +84,20 @@ __device__ __forceinline__ void put_query(const AttendPlan& pl, float* sm, int h
     }
 }
 
+template <typename T>
+__device__ __forceinline__ void put_query4(const AttendPlan& pl, float* sm, int heads, int h, int d, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        store4(sm + pl.q + h * pl.ldq + d, v);
+    } else {
+        bf16* q = reinterpret_cast<bf16*>(sm + pl.q);
+        uint2 hi, lo;
+        split_bf16(v.x, v.y, hi.x, lo.x);
+        split_bf16(v.z, v.w, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(q + h * pl.ldq + d) = hi;
+        *reinterpret_cast<uint2*>(q + (heads + h) * pl.ldq + d) = lo;
+    }
+}
+
 // Scores of the keys of one kv head, row_of(jl, g) -> key row. fp32: a thread per (key, kv head), the
 // group's query heads kAttendHeads at a time.
 template <typename RowOf>

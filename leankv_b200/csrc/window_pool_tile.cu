@@ -8,8 +8,8 @@
 // bf16 numbers each (16 bits); after it they are rounded once for the product with the values.
 //
 // A warp owns HPW query heads of one kv head; with few heads, several warps share a head and take every KS-th
-// key tile. Key rows go straight from L2 to registers (no other warp needs them), value rows through a
-// warp-private buffer because their fragments need the transposing load.
+// key tile. Key rows go straight from L2 to registers, value rows through shared memory because their
+// fragments need the transposing load.
 
 #include <algorithm>
 
@@ -140,6 +140,7 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
         for (int h = 0; h < HPW; ++h)
 #pragma unroll
             for (int x = 0; x < 4; ++x) s[h][x] = 0.f;
+        float s2[4] = {};          // with one head, a second accumulator halves the chain of dependent products
 #pragma unroll
         for (int b = 0; b < NB; ++b)
             if (b < nb) {
@@ -149,8 +150,12 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
 #pragma unroll
                 for (int h = 0; h < HPW; ++h) mma_bf16(s[h], k.x0[b].x, k.x1[b].x, k.x0[b].y, k.x1[b].y, y[h].x, y[h].y);
 #pragma unroll
-                for (int h = 0; h < HPW; ++h) mma_bf16(s[h], k.x0[b].z, k.x1[b].z, k.x0[b].w, k.x1[b].w, y[h].z, y[h].w);
+                for (int h = 0; h < HPW; ++h)
+                    mma_bf16(HPW == 1 ? s2 : s[h], k.x0[b].z, k.x1[b].z, k.x0[b].w, k.x1[b].w, y[h].z, y[h].w);
             }
+        if (HPW == 1)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) s[0][x] += s2[x];
         const bool pooled = tile < TB;
         const int base = pooled ? tile * 16 : tok0 + (tile - TB) * 16;
         const bool all = tile < NT && (pooled ? base + 15 < first.n_blk : base >= last.w0 && base + 15 <= i0);
@@ -254,16 +259,19 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
 #pragma unroll
             for (int x = 0; x < 4; ++x) o[h][m][x] = 0.f;
     const int dvt = vp / 16;
-    unsigned char* vbuf = smem + p.off_v + (size_t)warp * 16 * p.v_row;
-    const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(vbuf);
+    // value rows of a (key split, kv head) are shared by the warps of that head's queries, in two buffers
+    const int sharers = rep / HPW, v_buf = 16 * p.v_row, v_half = KS * G * v_buf;
+    const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(smem + p.off_v) + (ks * G + kv) * v_buf;
     uint32_t* pm = reinterpret_cast<uint32_t*>(smem + p.off_pm);
     Keys keys;
     if (worker) load_keys(ks, keys);
-    const int v_per = vp / 8, v_r0 = lane / v_per, v_c0 = lane % v_per, v_dr = 32 / v_per, v_dc = 32 % v_per;
+    const int v_per = vp / 8, v_id = hslot % sharers * 32 + lane, v_r0 = v_id / v_per, v_c0 = v_id % v_per;
+    const int v_dr = sharers * 32 / v_per, v_dc = sharers * 32 % v_per;
     const size_t v_stride = (size_t)G * vp;
 #pragma unroll 1
-    for (int base = 0; base < NT; base += KS) {
+    for (int base = 0, half = 0; base < NT; base += KS, half ^= 1) {
         const int tile = base + ks;
+        const uint32_t v_now = vaddr + half * v_half;
         if (worker) {
             {       // this tile's values start their way
                 const TileRows tr = rows_of(tile);
@@ -271,7 +279,7 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
                 int r = v_r0, ch = v_c0;
                 while (r < 16) {
                     const bf16* from = src + index_of(tr, r) * v_stride + ch * 8;
-                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vaddr + r * p.v_row + ch * 16), "l"(from)
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(v_now + r * p.v_row + ch * 16), "l"(from)
                                  : "memory");
                     r += v_dr;
                     ch += v_dc;
@@ -348,7 +356,7 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
                 b[h][1] = w[4];
             }
             const int mi = lane >> 3, r = (lane & 7) + (mi >= 2 ? 8 : 0);
-            const uint32_t from = vaddr + r * p.v_row + (mi & 1) * 16;
+            const uint32_t from = v_now + r * p.v_row + (mi & 1) * 16;
 #pragma unroll
             for (int m = 0; m < DVT; ++m)
                 if (m < dvt) {
@@ -359,7 +367,6 @@ __global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_k
 #pragma unroll
                     for (int h = 0; h < HPW; ++h) mma_bf16(o[h][m], a0, a1, a2, a3, b[h][0], b[h][1]);
                 }
-            __syncwarp();
         }
     }
 
@@ -453,7 +460,7 @@ int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* 
     p.off_stat = take(p.ks * a.heads * kQ * 8);
     p.off_p = take(16 * p.ks * p.p_key);
     p.off_pm = take(a.heads * p.pm_h * 4);
-    p.off_v = take(std::max(kWarps * 16 * p.v_row, p.ks > 1 ? a.heads * a.vdim_pad * kQ * 4 : 0));
+    p.off_v = take(std::max(2 * p.ks * a.kv_heads * 16 * p.v_row, p.ks > 1 ? a.heads * a.vdim_pad * kQ * 4 : 0));
     if (at > 227 * 1024) return LEANKV_EUNSUPPORTED;
     switch (hpw) {
         case 1: return launch_sizes<1>(p, at, st);
