@@ -43,7 +43,7 @@ __device__ __forceinline__ float ex2(float x) {
 // HPW query heads per warp, NB blocks of 32 dimensions and DVT tiles of 16 value columns; EXACT: the sizes are
 // those, otherwise at most those.
 template <int HPW, int NB, int DVT, bool EXACT>
-__global__ void __launch_bounds__(kThreads, HPW == 1 ? 2 : 1) window_pool_tile_kernel(const __grid_constant__ TileParams p) {
+__global__ void __launch_bounds__(kThreads, 1) window_pool_tile_kernel(const __grid_constant__ TileParams p) {
     extern __shared__ __align__(128) unsigned char smem[];
     pdl_begin();
     const leankv_window_pool_t& a = p.a;
@@ -434,9 +434,10 @@ int window_pool_tile_attend(const leankv_window_pool_t& a, const void* q, void* 
                             int start, cudaStream_t st) {
     const int rep = a.heads / a.kv_heads;
     if (a.dtype != LEANKV_DT_BF16 || a.dim_pad > 32 * kMaxNb || a.vdim_pad > 128) return LEANKV_EUNSUPPORTED;
-    int hpw = 1;
-    while (hpw <= 4 && (rep % hpw != 0 || a.heads / hpw > kWarps)) ++hpw;
-    if (hpw > 4) return LEANKV_EUNSUPPORTED;
+    // the most heads per warp: fewer warps read the same key and value rows, and more key tiles go in parallel
+    int hpw = 4;
+    while (hpw > 1 && rep % hpw != 0) --hpw;
+    if (a.heads / hpw > kWarps) return LEANKV_EUNSUPPORTED;
     TileParams p{};
     p.a = a;
     p.q = static_cast<const bf16*>(q);
