@@ -65,8 +65,8 @@ def read_weights(model_dir: str) -> dict[str, torch.Tensor]:
 
 
 class TensorBag:
-    """The tensors of a checkpoint, taken by name and expected shape; what is missing, misshapen or left
-    over is an error."""
+    """The tensors of a checkpoint, taken by name and expected shape; what is missing or misshapen is an
+    error, what is left over a warning."""
 
     def __init__(self, tensors: dict[str, torch.Tensor]):
         self._t, self._used = tensors, set()
@@ -88,4 +88,4 @@ class TensorBag:
     def finish(self) -> None:
         left = sorted(set(self._t) - self._used)
         if left:
-            raise ValueError(f"checkpoint has tensors that no layer uses: {', '.join(left[:8])}")
+            warnings.warn(f"checkpoint has tensors that no layer uses: {', '.join(left[:8])}")

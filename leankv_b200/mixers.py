@@ -9,7 +9,7 @@ the kernels, so a model combines them as its configuration says.
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 
 import torch
 
@@ -51,6 +51,11 @@ class WindowPoolSpec:
         if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.size, spec.pool) < 1 or spec.heads % spec.kv_heads:
             raise ValueError(f"bad attention sizes: {spec}")
         return spec
+
+    def bounded(self, max_seq_len: int) -> "WindowPoolSpec":
+        """The same visibility for sequences of at most ``max_seq_len`` tokens, with no larger ring than they
+        need: a longer window shows every token, a longer block is never complete."""
+        return replace(self, size=min(self.size, max_seq_len), pool=min(self.pool, max_seq_len + 1))
 
     @property
     def q_width(self) -> int:
@@ -102,7 +107,8 @@ class WindowPoolAttention:
     """Window + pooled-block attention over normed queries and keys, weights mixed across heads."""
 
     def __init__(self, spec: WindowPoolSpec, p: Parameters, seq: SequenceState, eps: float):
-        self.spec, self.seq = spec, seq
+        self.spec = spec = spec.bounded(seq.max_seq_len)
+        self.seq = seq
         self.lib = _native.mixers()
         self.q_norm = p.vector("q.norm", spec.q_width)
         self.k_norm = p.vector("k.norm", spec.kv_heads * spec.dim)

@@ -493,6 +493,15 @@ def test_constants_come_from_the_configuration(eps, left, right):
     assert rel(got, plain.forward(cfg, w, ids)[40:]) < MODEL_TOL[F32]
 
 
+def test_window_and_block_longer_than_the_sequence():
+    cfg = config([layer(size=1000, pool=3), layer(size=5, pool=700), layer(size=4000, pool=2000, ff=None)])
+    w, ids = weights(cfg, 5), tokens(cfg, 64)
+    eng = MixerDecodeEngine(MixerModelConfig.from_dict(cfg), w, DEV, max_seq_len=64, dtype=F32)
+    want = plain.forward(cfg, w, ids)
+    assert rel(eng.extend(ids[:50], list(range(50))), want[:50]) < MODEL_TOL[F32]
+    assert rel(torch.cat([eng.extend([t], [0]) for t in ids[50:]]), want[50:]) < MODEL_TOL[F32]
+
+
 def test_engine_refuses_what_does_not_fit():
     cfg, w, eng = engine("small", F32, limit=10)
     with pytest.raises(ValueError):

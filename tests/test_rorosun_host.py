@@ -125,7 +125,7 @@ def test_tensor_bag_refuses_what_does_not_fit():
         bag.take("b", 5)
     with pytest.raises(ValueError, match="no tensor"):
         bag.take("c", 5)
-    with pytest.raises(ValueError, match="no layer uses"):
+    with pytest.warns(UserWarning, match="no layer uses"):
         bag.finish()
 
 
@@ -188,6 +188,15 @@ def test_replay_loop(tmp_path):
            {"step": 1, "entries": [{"id": "b", "tokens": [1], "want": []}], "end": []}]
     with pytest.raises(ValueError, match="before a has ended"):
         trace.replay(_FakeEngine(), map(json.dumps, bad), str(tmp_path), said.append)
+
+
+def test_windows_longer_than_the_sequence_take_no_more_memory():
+    spec = WindowPoolSpec(4, 2, 16, 24, size=1 << 20, pool=1 << 16, scale=1.0)
+    assert spec.bounded(100) == WindowPoolSpec(4, 2, 16, 24, size=100, pool=101, scale=1.0)
+    assert spec.bounded(1 << 21) == spec
+    for n in (1, 2, 50, 100):            # no position below the bound sees anything else
+        a, b = plain.visible(n, spec.size, spec.pool), plain.visible(n, 100, 101)
+        assert torch.equal(a[0], b[0]) and a[1].shape[1] == b[1].shape[1] == 0
 
 
 def test_sequence_state_sizes_and_reset():
