@@ -120,9 +120,9 @@ def mixer_leg(size, dev, steps, peaks):
     x, d = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
     h = torch.empty(T, W, dtype=eng.dtype, device=dev)
     mixed = torch.empty(5, T, W, dtype=eng.dtype, device=dev)
-    mem("stream_norm_shift", _graphed(lambda i: eng._stream_norm(x, L[i].norm1, h, d, L[i].ls1, L[i].mixer, mixed), layers),
+    mem("stream_norm_shift", _graphed(lambda i: eng._stream_norm(x, L[i].first.norm, h, d, L[i].first, L[i].mixer, mixed), layers),
         T * W * (4 * 3 + 2 * 6))
-    mem("stream_norm", _graphed(lambda i: eng._stream_norm(x, L[i].norm2, h, d, L[i].ls2), layers), T * W * (4 * 3 + 2))
+    mem("stream_norm", _graphed(lambda i: eng._stream_norm(x, L[i].second.norm, h, d, L[i].second), layers), T * W * (4 * 3 + 2))
     gu = torch.randn(T, 2 * ff, device=dev).bfloat16()
     act = torch.empty(T, ff, dtype=eng.dtype, device=dev)
     mem("silu_mul", _graphed(lambda i: lib.leankv_silu_mul(gu.data_ptr(), act.data_ptr(), 1, T, ff, st()), 4), T * ff * 6)

@@ -1,7 +1,8 @@
 /*
  * leankv_b200 — C ABI of the token mixers and dense layers beside the TEAL / TurboQuant paths:
- * row-major dense GEMV with fused norm / token shift / gating / residual, window + pooled-block
- * attention with mixed heads, and the matrix-state time mixing recurrence.
+ * row-major dense GEMV with fused norms / token shift / gating / residual, window + pooled-block
+ * attention with mixed heads, the matrix-state time mixing recurrence, and causal attention (whole sequence or
+ * window) over per-head keys or a shared latent.
  *
  * Conventions are those of leankv_b200.h (device pointers unless marked host, stream as void*, status
  * codes, nothing allocated or synchronised, every call may be captured into a CUDA graph). Storage types
@@ -28,10 +29,14 @@ extern "C" {
 
 /* y[rows] = epilogue( W x' ), W row-major [rows][cols] ([2 rows][cols], gate rows first, if gated).
  *   x' = x                                                   gain == NULL
- *   x' = h := gain * x / sqrt(mean(x^2) + eps)               gain: one number
+ *   x' = h := gain * x / sqrt(mean(x^2) + eps)               gain: one number, or one per column
  *   x' = h + (prev - h) * mu_s                               rows of segment s, mu[s] != NULL
  * prev is [2][cols]: half state[6] is read, h is written to the other half.
+ *   delta != NULL: a branch joins the stream first, x := x + post_mult * post_gain * delta / sqrt(mean(delta^2) + eps)
+ *     (post_gain per column), and that x goes to x_out (not x itself, not read by this launch).
+ *   group_rows > 0: rows g * group_rows .. belong to group g and multiply x + g * group_stride (no gain, no delta).
  *   epilogue: y = acc + bias (first bias_rows rows);  gated: y = silu(acc_gate) * acc_up;
+ *             softcap > 0: y = softcap * tanh(y / softcap);
  *             residual != NULL: y = residual + scale * acc (y may be residual; x may not be y). */
 typedef struct leankv_dense_gemv {
     const void* w;
@@ -49,6 +54,13 @@ typedef struct leankv_dense_gemv {
     int bias_rows;
     const float* scale;
     const float* residual;
+    int gain_per_col;
+    const float* delta;
+    const float* post_gain;
+    float post_mult;
+    float* x_out;
+    int group_rows, group_stride;
+    float softcap;
 } leankv_dense_gemv_t;
 
 int leankv_dense_gemv(const leankv_dense_gemv_t* args, void* stream);
@@ -60,7 +72,8 @@ int leankv_greedy_end(const float* logits, int vocab, long long* token, long lon
                       int32_t* state, void* stream);
 
 /* Rows of a prompt portion: x_out = x_in + scale * delta (delta NULL: x_out is not written and may be
- * NULL), h = gain * rms(x_out), and for each of n_mix coefficient vectors mixed[i] = h + (h' - h) * mu[i], h' the row
+ * NULL; post_gain given, per column: x_in + post_mult * post_gain * rms(delta), no scale), h = gain * rms(x_out) (gain one
+ * number, or one per column; NULL with h: only the sum), and for each of n_mix coefficient vectors mixed[i] = h + (h' - h) * mu[i], h' the row
  * above (row 0: prev_in). h may be NULL. h of the last row goes to prev_out. delta is of type
  * delta_dtype, h and mixed [n_mix][rows][width] of type dtype. prev_in and prev_out must differ. */
 typedef struct leankv_stream_norm {
@@ -76,12 +89,18 @@ typedef struct leankv_stream_norm {
     float* prev_out;
     int dtype, delta_dtype, rows, width, n_mix;
     float eps;
+    int gain_per_col;
+    const float* post_gain;
+    float post_mult;
 } leankv_stream_norm_t;
 
 int leankv_stream_norm(const leankv_stream_norm_t* args, void* stream);
 
 /* out = silu(gate) * up; gate_up [rows][2 * inter], gate columns first. */
 int leankv_silu_mul(const void* gate_up, void* out, int dtype, int rows, int inter, void* stream);
+
+/* x = cap * tanh(x / cap), in place. */
+int leankv_softcap(float* x, long long n, float cap, void* stream);
 
 /* bf16: out [rows][2 n] = {hi, lo} with hi + lo = tanh(in) to 16 bits; fp32: out [rows][n] = tanh(in). */
 int leankv_tanh_split(const float* in, void* out, int dtype, int rows, int n, void* stream);
@@ -152,6 +171,80 @@ typedef struct leankv_mixer_step {
 size_t leankv_mixer_step_workspace_bytes(const leankv_window_pool_t* left, int max_pos);
 int leankv_mixer_step(const leankv_window_pool_t* left, const leankv_time_mix_t* right,
                       const leankv_mixer_step_t* step, void* stream);
+
+/* ---- causal attention over a ring of keys -------------------------------------------------------------
+ * Position i sees the positions j with 0 <= i - j < size. A key is `dim` numbers of its kv head and, after them,
+ * shared_dim numbers common to all heads (0: none); query head h reads kv head h / (heads / kv_heads). Position p
+ * lies in slot (p - base) % ring. v NULL: the value is the first vdim numbers of the key's own part (a latent).
+ * Paddings are multiples of 16 and zero; slots hold finite numbers. */
+typedef struct leankv_causal_attn {
+    int dtype, heads, kv_heads;
+    int dim, shared_dim, vdim, dim_pad, shared_pad, vdim_pad;
+    int size;
+    float scale;
+    void* k;                  /* [k_ring][kv_heads][dim_pad], the first k_rows slots are there */
+    void* v;                  /* [k_ring][kv_heads][vdim_pad] */
+    int k_base, k_ring, k_rows;
+    void* shared;             /* [s_ring][shared_pad], base 0 */
+    int s_ring;
+} leankv_causal_attn_t;
+
+/* Rows of a portion on their way into operand buffers and rings. Segment: element i < n of head h of row r at
+ * src[r * ld + h * head_stride + i] -> dst[slot * dst_ld + h * dst_head_stride + i] (storage type), i in n .. n_pad
+ * zero; slot = (start + r) % ring, or r without a ring. gain (heads == 1): RMS-normed over n. rot: coordinates
+ * 2i, 2i + 1 < rot of every head turn by (start + r) * rate[i]. */
+#define LEANKV_MAX_SEGMENTS 4
+typedef struct leankv_row_segment {
+    const float* src;
+    int ld, heads, head_stride, n;
+    void* dst;
+    int dst_ld, dst_head_stride, n_pad, ring;
+    const float* gain;
+    int rot;
+} leankv_row_segment_t;
+typedef struct leankv_place_rows {
+    int dtype, rows, start, n_seg;
+    leankv_row_segment_t seg[LEANKV_MAX_SEGMENTS];
+    const float* rate;
+    float eps;
+} leankv_place_rows_t;
+
+int leankv_place_rows(const leankv_place_rows_t* args, void* stream);
+
+/* Attention of `rows` tokens at positions start.., whose keys are in place. q [rows][heads][dim_pad + shared_pad] of the
+ * storage type; out [rows][heads * vdim] (storage type, row stride out_ld), times the logistic function of gate (fp32,
+ * row stride gate_ld; NULL: none). status: int32 set non-zero if a wait inside the kernel ran out. */
+int leankv_causal_attend(const leankv_causal_attn_t* a, const void* q, const float* gate, int gate_ld, void* out,
+                         int out_ld, int rows, int start, int32_t* status, void* stream);
+
+/* One decode step at position state[0] < max_pos: rotates the query and the new key, stores the key / value, attends.
+ * fp32 inputs: q [heads] x dim numbers (stride q_stride), q_shared [heads] x shared_dim (stride qs_stride), k_new
+ * [kv_heads][dim], shared_new [shared_dim], v_new [kv_heads][vdim] (unused if a->v is NULL). k_gain: k_new is RMS-normed
+ * over dim (kv_heads == 1). rot_own / rot_shared: rotated coordinates of either part. out fp32 [heads][vdim]; gate
+ * fp32 [heads * vdim] or NULL. state[0] and the rings may be read before the launch just ahead has finished: that
+ * launch must not write them. ws: leankv_causal_step_workspace_bytes, zeroed once before the first call. */
+typedef struct leankv_causal_step {
+    const float* q;
+    const float* q_shared;
+    const float* k_new;
+    const float* shared_new;
+    const float* v_new;
+    int q_stride, qs_stride;
+    const float* k_gain;
+    float eps;
+    const float* rate;
+    int rot_own, rot_shared;
+    const float* gate;
+    float* out;
+    const int32_t* state;
+    int max_pos;
+    void* ws;
+    size_t ws_bytes;
+    int32_t* status;
+} leankv_causal_step_t;
+
+size_t leankv_causal_step_workspace_bytes(const leankv_causal_attn_t* a, int max_pos);
+int leankv_causal_step(const leankv_causal_attn_t* a, const leankv_causal_step_t* step, void* stream);
 
 #ifdef __cplusplus
 }

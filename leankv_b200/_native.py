@@ -141,7 +141,9 @@ class DenseGemv(Structure):
                 ("n_mix", c_int), ("mix_end", c_int * MAX_MIX), ("mu", c_void_p * MAX_MIX),
                 ("prev", c_void_p), ("state", c_void_p),
                 ("bias", c_void_p), ("bias_rows", c_int),
-                ("scale", c_void_p), ("residual", c_void_p)]
+                ("scale", c_void_p), ("residual", c_void_p),
+                ("gain_per_col", c_int), ("delta", c_void_p), ("post_gain", c_void_p), ("post_mult", c_float),
+                ("x_out", c_void_p), ("group_rows", c_int), ("group_stride", c_int), ("softcap", c_float)]
 
 
 class StreamNorm(Structure):
@@ -151,7 +153,7 @@ class StreamNorm(Structure):
                 ("gain", c_void_p), ("h", c_void_p), ("mixed", c_void_p), ("mu", c_void_p * MAX_MIX),
                 ("prev_in", c_void_p), ("prev_out", c_void_p),
                 ("dtype", c_int), ("delta_dtype", c_int), ("rows", c_int), ("width", c_int), ("n_mix", c_int),
-                ("eps", c_float)]
+                ("eps", c_float), ("gain_per_col", c_int), ("post_gain", c_void_p), ("post_mult", c_float)]
 
 
 class WindowPool(Structure):
@@ -181,12 +183,52 @@ class MixerStep(Structure):
                 ("ws", c_void_p), ("ws_bytes", c_size_t)]
 
 
+class CausalAttn(Structure):
+    """Mirror of ``leankv_causal_attn_t``."""
+
+    _fields_ = [("dtype", c_int), ("heads", c_int), ("kv_heads", c_int),
+                ("dim", c_int), ("shared_dim", c_int), ("vdim", c_int),
+                ("dim_pad", c_int), ("shared_pad", c_int), ("vdim_pad", c_int),
+                ("size", c_int), ("scale", c_float),
+                ("k", c_void_p), ("v", c_void_p), ("k_base", c_int), ("k_ring", c_int), ("k_rows", c_int),
+                ("shared", c_void_p), ("s_ring", c_int)]
+
+
+class RowSegment(Structure):
+    """Mirror of ``leankv_row_segment_t``."""
+
+    _fields_ = [("src", c_void_p), ("ld", c_int), ("heads", c_int), ("head_stride", c_int), ("n", c_int),
+                ("dst", c_void_p), ("dst_ld", c_int), ("dst_head_stride", c_int), ("n_pad", c_int), ("ring", c_int),
+                ("gain", c_void_p), ("rot", c_int)]
+
+
+MAX_ROW_SEGMENTS = 4
+
+
+class PlaceRows(Structure):
+    """Mirror of ``leankv_place_rows_t``."""
+
+    _fields_ = [("dtype", c_int), ("rows", c_int), ("start", c_int), ("n_seg", c_int),
+                ("seg", RowSegment * MAX_ROW_SEGMENTS), ("rate", c_void_p), ("eps", c_float)]
+
+
+class CausalStep(Structure):
+    """Mirror of ``leankv_causal_step_t``."""
+
+    _fields_ = [("q", c_void_p), ("q_shared", c_void_p), ("k_new", c_void_p), ("shared_new", c_void_p),
+                ("v_new", c_void_p), ("q_stride", c_int), ("qs_stride", c_int),
+                ("k_gain", c_void_p), ("eps", c_float), ("rate", c_void_p), ("rot_own", c_int), ("rot_shared", c_int),
+                ("gate", c_void_p), ("out", c_void_p), ("state", c_void_p), ("max_pos", c_int),
+                ("ws", c_void_p), ("ws_bytes", c_size_t), ("status", c_void_p)]
+
+
 MIXER_SIGNATURES = {
     "leankv_dense_gemv": (c_int, [POINTER(DenseGemv), c_void_p]),
     "leankv_embed_begin": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]),
     "leankv_greedy_end": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "leankv_stream_norm": (c_int, [POINTER(StreamNorm), c_void_p]),
     "leankv_silu_mul": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "leankv_softcap": (c_int, [c_void_p, c_longlong, c_float, c_void_p]),
     "leankv_tanh_split": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "leankv_window_pool_append": (c_int, [POINTER(WindowPool), c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                           c_void_p]),
@@ -198,6 +240,11 @@ MIXER_SIGNATURES = {
                                      c_int, c_float, c_int, c_void_p, c_size_t, c_void_p]),
     "leankv_mixer_step_workspace_bytes": (c_size_t, [POINTER(WindowPool), c_int]),
     "leankv_mixer_step": (c_int, [POINTER(WindowPool), POINTER(TimeMix), POINTER(MixerStep), c_void_p]),
+    "leankv_place_rows": (c_int, [POINTER(PlaceRows), c_void_p]),
+    "leankv_causal_attend": (c_int, [POINTER(CausalAttn), c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                                     c_void_p, c_void_p]),
+    "leankv_causal_step_workspace_bytes": (c_size_t, [POINTER(CausalAttn), c_int]),
+    "leankv_causal_step": (c_int, [POINTER(CausalAttn), POINTER(CausalStep), c_void_p]),
 }
 _COMMON = ("leankv_strerror", "leankv_last_cuda_error", "leankv_abi_version")     # capi.cu, in both libraries
 

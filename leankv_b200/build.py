@@ -25,7 +25,8 @@ LIBRARIES = {
     "libleankv_b200.so": ["capi.cu", "teal_gemv.cu", "tq_quantize.cu", "tq_attn.cu", "decoder_ops.cu",
                           "decode_fused.cu"],
     "libleankv_mixers.so": ["capi.cu", "dense_gemv.cu", "stream_ops.cu", "window_pool.cu",
-                            "window_pool_tile.cu", "time_mix.cu", "mixer_step.cu"],
+                            "window_pool_tile.cu", "time_mix.cu", "mixer_step.cu", "causal_rows.cu", "causal_tile.cu",
+                            "causal_step.cu"],
 }
 LIB_PATH = os.path.join(PKG_DIR, "libleankv_b200.so")
 MIXERS_PATH = os.path.join(PKG_DIR, "libleankv_mixers.so")

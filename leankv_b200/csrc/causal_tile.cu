@@ -1,0 +1,301 @@
+// Causal attention of a prompt portion on the fifth-generation tensor cores (bf16 operands, fp32 scores and
+// weights). A CTA holds 128 rows, (token, query head) pairs of one kv head, and walks the 128-key tiles they see:
+//
+//   copy thread     Q once, then K and V tiles by TMA into swizzled shared memory (one buffer each: a K tile is free once the
+//                   scores are computed, a V tile once the outputs are)
+//   MMA thread      S = Q K^T into tensor memory; O += P V with P from tensor memory
+//   128 row threads a thread a row: mask, running maximum, exponentials; P goes back over S as two bf16 numbers per
+//                   weight (16 bits), so two products per V tile
+//
+// Two CTAs share an SM and fill each other's waits. O stays in tensor memory; it is rescaled only when a row's
+// maximum grows by more than 2^kSlack. Tiles start at positions that are multiples of 128 and rings are
+// multiples of 128 slots, so a tile never wraps.
+
+#include <algorithm>
+
+#include "causal_attn.cuh"
+#include "tma.cuh"
+
+namespace leankv {
+namespace {
+
+constexpr int kTile = 128;                       // rows of a CTA, keys of a tile
+constexpr int kThreads = 192;
+constexpr uint32_t kBlock = kTile * 128;         // one 128-row block of 64 columns: 16 KB
+constexpr float kSlack = 8.f;
+
+struct TileArgs {
+    CUtensorMap q, k, shared, v;
+    const float* gate;
+    bf16* out;
+    int32_t* status;
+    int gate_ld, out_ld, rows, start, size, vec;
+    int heads, rep, tq;                          // query heads, per kv head, tokens of a CTA
+    int dim_pad, shared_pad, vdim, vdim_pad;
+    int k_base, k_ring, s_ring, v_from_k;
+    int nb1, nb2, nbv;                           // 64-column blocks
+    uint32_t q_box, tmem_cols;
+    float c;                                     // scale * log2(e)
+};
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+enum { kQ, kKFull, kVFull, kS, kP, kKFree, kVFree, kO, kBars };
+
+__global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_constant__ TileArgs p) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    __shared__ __align__(8) uint64_t s_bar[kBars];
+    __shared__ uint32_t s_tmem;
+    pdl_begin();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t base = (umma::smem_addr(raw) + 1023u) & ~1023u;
+    const uint32_t sq = base, sk = sq + (p.nb1 + p.nb2) * kBlock, sv = p.v_from_k ? sk : sk + (p.nb1 + p.nb2) * kBlock;
+    auto bar = [&](int b) { return umma::smem_addr(&s_bar[b]); };
+    if (tid == 0)
+        for (int b = 0; b < kBars; ++b) umma::bar_init_n(bar(b), b == kP ? kTile : 1);
+    if (warp == 4) umma::tmem_alloc_n(umma::smem_addr(&s_tmem), p.tmem_cols);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    umma::fence_before_sync();
+    __syncthreads();
+    umma::fence_after_sync();
+    const uint32_t tmem = s_tmem, tm_s = tmem, tm_o = tmem + kTile;
+
+    const int g = blockIdx.y, q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * p.tq;      // the longest rows first
+    const int nt = min(p.tq, p.rows - q0);
+    const int lo = first_visible(p.start + q0, p.size), hi = p.start + q0 + nt - 1;
+    const int t0 = lo / kTile, n_tiles = hi / kTile - t0 + 1;
+    bool ok = true;
+
+    if (tid == 128) {                                    // ---- copies ----
+        tma::expect(bar(kQ), (p.nb1 + p.nb2) * p.q_box);
+        for (int b = 0; b < p.nb1 + p.nb2; ++b)
+            tma::load3(sq + b * kBlock, &p.q, b < p.nb1 ? b * 64 : p.dim_pad + (b - p.nb1) * 64, g * p.rep, q0, bar(kQ));
+        int nk = 0, nv = 0;
+        for (int j = 0; j < n_tiles && ok; ++j) {
+            const int at = (t0 + j) * kTile, slot = ring_slot(at, p.k_base, p.k_ring);
+            if (j > 0) ok = umma::bar_wait(bar(p.v_from_k ? kVFree : kKFree), (j - 1) & 1);
+            if (!ok) break;
+            tma::expect(bar(kKFull), (p.nb1 + p.nb2) * kBlock);
+            for (int b = 0; b < p.nb1; ++b) tma::load3(sk + b * kBlock, &p.k, b * 64, g, slot, bar(kKFull));
+            for (int b = 0; b < p.nb2; ++b)
+                tma::load3(sk + (p.nb1 + b) * kBlock, &p.shared, b * 64, 0, ring_slot(at, 0, p.s_ring), bar(kKFull));
+            ++nk;
+            if (p.v_from_k) continue;
+            if (j > 0) ok = umma::bar_wait(bar(kVFree), (j - 1) & 1);
+            if (!ok) break;
+            tma::expect(bar(kVFull), p.nbv * kBlock);
+            for (int b = 0; b < p.nbv; ++b) tma::load3(sv + b * kBlock, &p.v, b * 64, g, slot, bar(kVFull));
+            ++nv;
+        }
+        if (!ok) {                                       // give up only once the copies in flight have landed
+            umma::bar_wait(bar(kQ), 0);
+            if (nk > 0) umma::bar_wait(bar(kKFull), (nk - 1) & 1);
+            if (nv > 0) umma::bar_wait(bar(kVFull), (nv - 1) & 1);
+        }
+    } else if (tid == 160) {                             // ---- products ----
+        constexpr uint32_t idesc_s = tma::idesc_bf16(kTile, false);
+        const uint32_t idesc_o = tma::idesc_bf16(p.vdim_pad, true);
+        ok = umma::bar_wait(bar(kQ), 0);
+        for (int j = 0; j < n_tiles && ok; ++j) {
+            ok = umma::bar_wait(bar(kKFull), j & 1);
+            if (!ok) break;
+            umma::fence_after_sync();
+            uint32_t first = 0;
+            for (int part = 0; part < 2; ++part) {
+                const int steps = (part == 0 ? p.dim_pad : p.shared_pad) / 16;
+                const uint32_t off = part == 0 ? 0 : p.nb1 * kBlock;
+                for (int s = 0; s < steps; ++s, first = 1) {
+                    const uint32_t o = off + (s >> 2) * kBlock + (s & 3) * 32;
+                    umma::mma_f16_n(tm_s, tma::swizzled(sq + o, 16), tma::swizzled(sk + o, 16), idesc_s, first);
+                }
+            }
+            umma::commit(bar(kS));
+            umma::commit(bar(kKFree));
+            if (!p.v_from_k) ok = umma::bar_wait(bar(kVFull), j & 1);
+            ok = ok && umma::bar_wait(bar(kP), j & 1);
+            if (!ok) break;
+            umma::fence_after_sync();
+            for (int s = 0; s < kTile / 16; ++s) {       // 16 keys: high parts, then low parts
+                const uint64_t v = tma::swizzled(sv + s * 2048, kBlock);
+                const uint32_t pa = tm_s + (s >> 1) * 32 + (s & 1) * 8;
+                umma::mma_f16_ts(tm_o, pa, v, idesc_o, j > 0 || s > 0);
+                umma::mma_f16_ts(tm_o, pa + 16, v, idesc_o, 1);
+            }
+            umma::commit(bar(kVFree));
+            // the next scores go over these weights
+            ok = umma::bar_wait(bar(kVFree), j & 1);
+        }
+        umma::commit(bar(kO));
+        if (!ok) umma::bar_wait(bar(kO), 0);
+    } else if (tid < kTile) {                            // ---- rows ----
+        const int row0 = warp * 32, used = p.rep * nt;
+        const int r = min(tid, used - 1), t = q0 + r / p.rep, h = g * p.rep + r % p.rep, i = p.start + t;
+        const int see0 = first_visible(i, p.size);
+        float m = -1e30f, l = 0.f;
+        for (int j = 0; j < n_tiles; ++j) {
+            ok = __all_sync(0xffffffffu, umma::bar_wait(bar(kS), j & 1));      // the warp stays together
+            if (!ok) break;
+            umma::fence_after_sync();
+            const int at = (t0 + j) * kTile;
+            // this row's keys of the tile: from k0 to k1
+            const int k0 = max(see0 - at, 0), k1 = min(i - at, kTile - 1);
+            const bool all = k0 == 0 && k1 == kTile - 1;
+            float best = -INFINITY;
+#pragma unroll 1
+            for (int c = 0; c < 4; ++c) {
+                uint32_t s[32];
+                umma::ld32(s, tm_s, row0, c * 32);
+                if (all) {
+#pragma unroll
+                    for (int x = 0; x < 32; ++x) best = fmaxf(best, __uint_as_float(s[x]));
+                } else {
+#pragma unroll
+                    for (int x = 0; x < 32; ++x) {
+                        const int k = c * 32 + x;
+                        best = fmaxf(best, k >= k0 && k <= k1 ? __uint_as_float(s[x]) : -INFINITY);
+                    }
+                }
+            }
+            const bool raise = best * p.c > m + kSlack;
+            if (__any_sync(0xffffffffu, raise)) {
+                const float mn = raise ? best * p.c : m, f = ex2(m - mn);
+                m = mn;
+                l *= f;
+                if (j > 0)
+#pragma unroll 1
+                    for (int c = 0; c < p.vdim_pad; c += 32) {
+                        uint32_t o[32];
+                        umma::ld32(o, tm_o, row0, c);
+#pragma unroll
+                        for (int x = 0; x < 32; ++x) o[x] = __float_as_uint(__uint_as_float(o[x]) * f);
+                        umma::st32(o, tm_o, row0, c);
+                    }
+            }
+#pragma unroll 1
+            for (int c = 0; c < 4; ++c) {
+                uint32_t s[32], ph[16], pl[16];
+                umma::ld32(s, tm_s, row0, c * 32);
+#pragma unroll
+                for (int x = 0; x < 32; x += 2) {
+                    float w[2];
+#pragma unroll
+                    for (int y = 0; y < 2; ++y) {
+                        const int k = c * 32 + x + y;
+                        const float e = ex2(fmaf(__uint_as_float(s[x + y]), p.c, -m));
+                        w[y] = all || (k >= k0 && k <= k1) ? e : 0.f;
+                        l += w[y];
+                    }
+                    split_bf16(w[0], w[1], ph[x / 2], pl[x / 2]);
+                }
+                umma::st16(ph, tm_s, row0, c * 32);
+                umma::st16(pl, tm_s, row0, c * 32 + 16);
+            }
+            umma::fence_before_sync();
+            umma::bar_arrive(bar(kP));
+        }
+        if (ok) ok = __all_sync(0xffffffffu, umma::bar_wait(bar(kO), 0));
+        umma::fence_after_sync();
+        const float inv = 1.f / l;
+        bf16* out = p.out + (size_t)t * p.out_ld + h * p.vdim;
+        const float* gate = p.gate != nullptr ? p.gate + (size_t)t * p.gate_ld + h * p.vdim : nullptr;
+        const bool vec = p.vec != 0;
+#pragma unroll 1
+        for (int c = 0; c < p.vdim_pad; c += 32) {
+            uint32_t o[32];
+            umma::ld32(o, tm_o, row0, c);
+            if (tid >= used || !ok) continue;
+#pragma unroll
+            for (int x = 0; x < 32; x += 8) {
+                if (c + x >= p.vdim) break;
+                float w[8];
+#pragma unroll
+                for (int y = 0; y < 8; ++y) w[y] = __uint_as_float(o[x + y]) * inv;
+                if (vec) {
+                    if (gate != nullptr) {
+                        const float4 g0 = *reinterpret_cast<const float4*>(gate + c + x);
+                        const float4 g1 = *reinterpret_cast<const float4*>(gate + c + x + 4);
+                        w[0] *= sigmoid_f32(g0.x); w[1] *= sigmoid_f32(g0.y); w[2] *= sigmoid_f32(g0.z); w[3] *= sigmoid_f32(g0.w);
+                        w[4] *= sigmoid_f32(g1.x); w[5] *= sigmoid_f32(g1.y); w[6] *= sigmoid_f32(g1.z); w[7] *= sigmoid_f32(g1.w);
+                    }
+                    *reinterpret_cast<uint4*>(out + c + x) = make_uint4(pack_bf16(w[0], w[1]), pack_bf16(w[2], w[3]),
+                                                                         pack_bf16(w[4], w[5]), pack_bf16(w[6], w[7]));
+                } else {
+#pragma unroll
+                    for (int y = 0; y < 8; ++y) {
+                        const int d = c + x + y;
+                        if (d < p.vdim) out[d] = from_f32<bf16>(gate != nullptr ? w[y] * sigmoid_f32(gate[d]) : w[y]);
+                    }
+                }
+            }
+        }
+    }
+    if (!ok && p.status != nullptr) *p.status = 1;
+    __syncwarp();
+    umma::fence_before_sync();
+    __syncthreads();
+    if (warp == 4) {
+        umma::fence_after_sync();
+        umma::tmem_free_n(tmem, p.tmem_cols);
+    }
+    (void)lane;
+}
+
+}  // namespace
+
+int causal_tile_attend(const leankv_causal_attn_t& a, const void* q, const float* gate, int gate_ld, void* out, int out_ld,
+                       int rows, int start, int32_t* status, cudaStream_t st) {
+    const int rep = a.heads / a.kv_heads;
+    if (a.dtype != LEANKV_DT_BF16 || rep > kTile || a.vdim_pad > 256 || a.kv_heads > 65535 || a.k_base % kTile ||
+        a.k_ring % kTile || (a.shared_dim > 0 && a.s_ring % kTile))
+        return LEANKV_EUNSUPPORTED;
+    TileArgs p{};
+    p.nb1 = (a.dim_pad + 63) / 64;
+    p.nb2 = a.shared_dim > 0 ? (a.shared_pad + 63) / 64 : 0;
+    p.nbv = (a.vdim_pad + 63) / 64;
+    p.v_from_k = a.v == nullptr;
+    size_t smem = (size_t)(2 * (p.nb1 + p.nb2) + (p.v_from_k ? 0 : p.nbv)) * kBlock + 1024;
+    if (smem > 226 * 1024) return LEANKV_EUNSUPPORTED;
+    p.tmem_cols = kTile + (a.vdim_pad + 31) / 32 * 32 <= 256 ? 256 : 512;
+    if (p.tmem_cols == 512) smem = std::max(smem, (size_t)116 * 1024);       // tensor memory for one CTA per SM
+    p.gate = gate;
+    p.gate_ld = gate_ld;
+    p.out = static_cast<bf16*>(out);
+    p.out_ld = out_ld;
+    p.status = status;
+    p.vec = a.vdim % 8 == 0 && out_ld % 8 == 0 && aligned16(out) && (!gate || (gate_ld % 4 == 0 && aligned16(gate)));
+    p.rows = rows;
+    p.start = start;
+    p.size = a.size;
+    p.heads = a.heads;
+    p.rep = rep;
+    p.tq = kTile / rep;
+    p.dim_pad = a.dim_pad;
+    p.shared_pad = a.shared_dim > 0 ? a.shared_pad : 0;
+    p.vdim = a.vdim;
+    p.vdim_pad = a.vdim_pad;
+    p.k_base = a.k_base;
+    p.k_ring = a.k_ring;
+    p.s_ring = a.s_ring;
+    p.q_box = 128u * rep * p.tq;
+    p.c = a.scale * 1.4426950408889634f;
+    const cuuint64_t dq = a.dim_pad + p.shared_pad, G = a.kv_heads, H = a.heads;
+    const auto map = [](CUtensorMap* m, const void* base, cuuint64_t d, cuuint64_t h, cuuint64_t n, cuuint32_t bh, cuuint32_t bn) {
+        const cuuint64_t dims[3] = {d, h, n}, strides[2] = {d, d * h};
+        const cuuint32_t box[3] = {(cuuint32_t)tma::kBoxCols, bh, bn};
+        return tma::make_map(m, base, 3, dims, strides, box);
+    };
+    int rc = map(&p.q, q, dq, H, rows, rep, p.tq);
+    if (!rc) rc = map(&p.k, a.k, a.dim_pad, G, a.k_rows, 1, kTile);
+    if (!rc && p.nb2) rc = map(&p.shared, a.shared, a.shared_pad, 1, a.s_ring, 1, kTile);
+    if (!rc && a.v) rc = map(&p.v, a.v, a.vdim_pad, G, a.k_rows, 1, kTile);
+    if (rc) return rc;
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(causal_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LEANKV_CUDA_TRY(launch_kernel(causal_tile_kernel, dim3((rows + p.tq - 1) / p.tq, a.kv_heads), dim3(kThreads), smem, st, p));
+    return LEANKV_OK;
+}
+
+}  // namespace leankv

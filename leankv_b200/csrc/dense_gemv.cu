@@ -1,7 +1,7 @@
 // Dense matrix-vector product over row-major [out][in] weights (bf16 or fp32), fp32 vectors and arithmetic,
 // with the steps around a projection fused in: RMS norm with one gain, token shift (a mix of the normed
 // vector with the previous token's, per row segment), bias, silu gating of row pairs, and the scaled
-// residual sum.
+// residual sum; or a branch's post-norm and residual sum ahead of the norm, and row groups with an input slice each.
 //
 // A CTA owns a contiguous range of rows; its warps split the columns and every warp walks all rows of the
 // range, so a lane's share of x stays in registers for the whole range and the weight stream needs no
@@ -9,6 +9,7 @@
 // bit-reproducible.
 
 #include <algorithm>
+#include <type_traits>
 
 #include "decode_frame.cuh"
 #include "leankv_mixers.h"
@@ -18,11 +19,13 @@ namespace {
 
 constexpr int kMaxWarps = 16;
 constexpr int kSmemPartials = 96 * 1024;
+constexpr int kMaxStaged = 32 * 1024;        // columns of a launch that prepares its input in shared memory
 
 struct GemvParams {
     leankv_dense_gemv_t a;
     int slabs;          // column passes of (warps * 32 * 8 * CH)
     int vec;            // cols % 8 == 0: 16-byte loads
+    int x_smem;         // floats of shared memory in front of the partial sums: the prepared input
 };
 
 template <typename T>
@@ -80,10 +83,15 @@ __device__ __forceinline__ float warp_reduce_rows(float (&acc)[R], int lane) {
 template <int R>
 __device__ __forceinline__ int row_of_lane(int lane) { return (lane * R) >> 5; }
 
-template <typename T, int CH>
+// kStaged: the input is prepared once in shared memory (a branch joins it, or a gain per column). kGrouped: row
+// groups with an input slice each.
+enum class Input { kPlain, kStaged, kGrouped };
+template <typename T, int CH, Input IN>
 __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel(const GemvParams p) {
+    constexpr bool STAGED = IN == Input::kStaged, GROUPED = IN == Input::kGrouped;
     constexpr int R = 8 / CH;                        // rows in flight: R * CH 16-byte loads per lane (bf16)
-    extern __shared__ float s_part[];                // [rows of this CTA (x2 if gated)][warps]
+    extern __shared__ __align__(16) float s_dyn[];
+    float* s_part = STAGED ? s_dyn + p.x_smem : s_dyn;      // [rows of this CTA (x2 if gated)][warps]
     __shared__ float s_tmp[32];
     const leankv_dense_gemv_t& a = p.a;
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -107,7 +115,30 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
     pdl_begin();
 
     float rs = 1.f;
-    if (a.gain != nullptr) {
+    if constexpr (STAGED) {         // the normed input x', after a branch joined x, into shared memory
+        float f = 0.f, ss = 0.f;
+        if (a.delta != nullptr) {
+            float sd = 0.f;
+            for (int k = threadIdx.x; k < cols; k += blockDim.x) {
+                const float d = ld_cg_f32(a.delta + k);
+                s_dyn[k] = d;
+                sd = fmaf(d, d, sd);
+            }
+            f = a.post_mult / sqrtf(cta_sum(sd, s_tmp) / (float)cols + a.eps);
+        }
+        for (int k = threadIdx.x; k < cols; k += blockDim.x) {
+            float x = ld_cg_f32(a.x + k);
+            if (a.delta != nullptr) {
+                x = fmaf(s_dyn[k] * f, __ldg(a.post_gain + k), x);
+                if (blockIdx.x == 0) a.x_out[k] = x;
+            }
+            s_dyn[k] = x;
+            ss = fmaf(x, x, ss);
+        }
+        if (a.gain != nullptr) rs = (a.gain_per_col ? 1.f : __ldg(a.gain)) / sqrtf(cta_sum(ss, s_tmp) / (float)cols + a.eps);
+        for (int k = threadIdx.x; k < cols; k += blockDim.x) s_dyn[k] *= rs * (a.gain_per_col ? __ldg(a.gain + k) : 1.f);
+        __syncthreads();
+    } else if (a.gain != nullptr) {
         float ss = 0.f;
         for (int s = 0; s < p.slabs; ++s)
 #pragma unroll
@@ -125,13 +156,15 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
         prev = a.prev + (size_t)par * cols;
         float* next = a.prev + (size_t)(par ^ 1) * cols;
         if (blockIdx.x == 0)
-            for (int k = threadIdx.x; k < cols; k += blockDim.x) next[k] = ld_cg_f32(a.x + k) * rs;
+            for (int k = threadIdx.x; k < cols; k += blockDim.x)
+                next[k] = STAGED ? s_dyn[k] : ld_cg_f32(a.x + k) * rs;
     }
+    const int m0 = GROUPED ? lo / a.group_rows : 0, m1 = GROUPED ? (hi - 1) / a.group_rows + 1 : max(a.n_mix, 1);
 
     for (int s = 0; s < p.slabs; ++s) {
-        int seg_lo = 0;
-        for (int m = 0; m < max(a.n_mix, 1); ++m) {
-            const int seg_hi = a.n_mix > 0 ? a.mix_end[m] : a.rows;
+        int seg_lo = GROUPED ? m0 * a.group_rows : 0;
+        for (int m = m0; m < m1; ++m) {
+            const int seg_hi = a.n_mix > 0 ? a.mix_end[m] : GROUPED ? seg_lo + a.group_rows : a.rows;
             const int r0 = max(lo, seg_lo), r1 = min(hi, seg_hi);
             seg_lo = seg_hi;
             if (r0 >= r1) continue;
@@ -140,9 +173,20 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
 #pragma unroll
             for (int c = 0; c < CH; ++c) {
                 const int k = s * slab_cols + (c * warps + warp) * 256 + lane * 8;
-                load_x8(a.x, k, cols, vec, xs[c]);
+                if constexpr (STAGED) {
+                    const bool on = vec && k < cols;
+                    const float4 lo4 = on ? *reinterpret_cast<const float4*>(s_dyn + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float4 hi4 = on ? *reinterpret_cast<const float4*>(s_dyn + k + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    xs[c][0] = lo4.x; xs[c][1] = lo4.y; xs[c][2] = lo4.z; xs[c][3] = lo4.w;
+                    xs[c][4] = hi4.x; xs[c][5] = hi4.y; xs[c][6] = hi4.z; xs[c][7] = hi4.w;
+                    if (!vec)
 #pragma unroll
-                for (int i = 0; i < 8; ++i) xs[c][i] *= rs;
+                        for (int i = 0; i < 8; ++i) xs[c][i] = k + i < cols ? s_dyn[k + i] : 0.f;
+                } else {
+                    load_x8(GROUPED ? a.x + (size_t)m * a.group_stride : a.x, k, cols, vec, xs[c]);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) xs[c][i] *= rs;
+                }
                 if (mu != nullptr) {
                     float pv[8], mv[8];
                     load_x8(prev, k, cols, vec, pv);
@@ -199,12 +243,13 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
             y = total(i);
             if (a.bias != nullptr && row < a.bias_rows) y += __ldg(a.bias + row);
         }
+        if (a.softcap > 0.f) y = a.softcap * tanhf(y / a.softcap);
         if (a.residual != nullptr) y = a.residual[row] + y * __ldg(a.scale + row);
         a.y[row] = y;
     }
 }
 
-template <typename T, int CH>
+template <typename T, int CH, Input IN>
 int launch_gemv(const GemvParams& p, int warps, cudaStream_t st) {
     const int per_sm = std::max(1, (sizeof(T) == 2 ? 2 : 1) * kMaxWarps / warps);
     const int mult = p.a.gated ? 2 : 1;
@@ -212,11 +257,11 @@ int launch_gemv(const GemvParams& p, int warps, cudaStream_t st) {
     grid = std::max(grid, 1);
     const auto smem_for = [&](int g) { return (size_t)((p.a.rows + g - 1) / g) * mult * warps * sizeof(float); };
     while (smem_for(grid) > (size_t)kSmemPartials / 2 && grid < p.a.rows) grid = std::min(p.a.rows, grid * 2);
-    const size_t smem = smem_for(grid);
+    const size_t smem = smem_for(grid) + (size_t)p.x_smem * sizeof(float);
     if (smem > 48 * 1024)
-        LEANKV_CUDA_TRY(cudaFuncSetAttribute(dense_gemv_kernel<T, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                             kSmemPartials));
-    LEANKV_CUDA_TRY(launch_kernel_ex(true, dense_gemv_kernel<T, CH>, dim3(grid), dim3(warps * 32), smem, st, p));
+        LEANKV_CUDA_TRY(cudaFuncSetAttribute(dense_gemv_kernel<T, CH, IN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             kSmemPartials + kMaxStaged * (int)sizeof(float)));
+    LEANKV_CUDA_TRY(launch_kernel_ex(true, dense_gemv_kernel<T, CH, IN>, dim3(grid), dim3(warps * 32), smem, st, p));
     return LEANKV_OK;
 }
 
@@ -237,10 +282,18 @@ extern "C" int leankv_dense_gemv(const leankv_dense_gemv_t* a, void* stream) {
     } else if (a->prev) {
         return LEANKV_EINVAL;
     }
-    if (!aligned16(a->w) || !aligned16(a->x)) return LEANKV_EALIGN;
+    if (a->delta && (!a->post_gain || !a->x_out || a->x_out == a->x || a->x_out == a->delta || a->delta == a->y))
+        return LEANKV_EINVAL;
+    if ((a->delta || a->gain_per_col) && a->cols > kMaxStaged) return LEANKV_ELIMIT;
+    if (a->group_rows < 0 || (a->group_rows > 0 && (a->rows % a->group_rows || a->group_stride < 0 || a->gain || a->delta ||
+                                                    a->n_mix > 0 || a->gated)))
+        return LEANKV_EINVAL;
+    if (!aligned16(a->w) || !aligned16(a->x) || (a->gain_per_col && !aligned16(a->gain))) return LEANKV_EALIGN;
     GemvParams p{};
     p.a = *a;
-    p.vec = a->cols % 8 == 0;
+    p.vec = a->cols % 8 == 0 && (a->group_rows == 0 || a->group_stride % 4 == 0);
+    const bool staged = a->delta || (a->gain && a->gain_per_col);
+    p.x_smem = staged ? (a->cols + 3) / 4 * 4 : 0;
     // warps x slabs x CH column chunks of 256: the widest CTA that pads least
     const int chunks = (a->cols + 255) / 256;
     int warps = 1, per = 1;
@@ -253,7 +306,15 @@ extern "C" int leankv_dense_gemv(const leankv_dense_gemv_t* a, void* stream) {
         }
     p.slabs = (chunks + warps * per - 1) / (warps * per);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    if (a->dtype == LEANKV_DT_BF16)
-        return per == 1 ? launch_gemv<bf16, 1>(p, warps, st) : launch_gemv<bf16, 2>(p, warps, st);
-    return per == 1 ? launch_gemv<float, 1>(p, warps, st) : launch_gemv<float, 2>(p, warps, st);
+    const auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        const auto with = [&](auto in) -> int {
+            constexpr Input IN = decltype(in)::value;
+            return per == 1 ? launch_gemv<T, 1, IN>(p, warps, st) : launch_gemv<T, 2, IN>(p, warps, st);
+        };
+        if (staged) return with(std::integral_constant<Input, Input::kStaged>{});
+        if (a->group_rows > 0) return with(std::integral_constant<Input, Input::kGrouped>{});
+        return with(std::integral_constant<Input, Input::kPlain>{});
+    };
+    return a->dtype == LEANKV_DT_BF16 ? go(bf16{}) : go(float{});
 }

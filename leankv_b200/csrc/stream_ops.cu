@@ -19,12 +19,24 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const leankv_s
     pdl_begin();
     const int t = blockIdx.x, W = a.width;
     const D* delta = static_cast<const D*>(a.delta);
+    const float* scale = a.post_gain != nullptr ? a.post_gain : a.scale;
+    const bool shift = a.n_mix > 0;
+    auto branch_factor = [&](int row) {         // of a branch that is normed before it joins the stream
+        if (a.post_gain == nullptr) return 1.f;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < W; i += kRowThreads) {
+            const float d = to_f32(delta[(size_t)row * W + i]);
+            ss = fmaf(d, d, ss);
+        }
+        return a.post_mult / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+    };
+    const float f_here = branch_factor(t), f_above = shift && t > 0 ? branch_factor(t - 1) : 1.f;
     auto value = [&](int row, int i) {
         float x = a.x_in[(size_t)row * W + i];
-        if (delta != nullptr) x = fmaf(to_f32(delta[(size_t)row * W + i]), __ldg(a.scale + i), x);
+        if (delta != nullptr)
+            x = fmaf(to_f32(delta[(size_t)row * W + i]) * (row == t ? f_here : f_above), __ldg(scale + i), x);
         return x;
     };
-    const bool shift = a.n_mix > 0;
     float ss = 0.f, ss_above = 0.f;
     for (int i = threadIdx.x; i < W; i += kRowThreads) {
         const float x = value(t, i);
@@ -35,17 +47,19 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_kernel(const leankv_s
             ss_above = fmaf(y, y, ss_above);
         }
     }
-    const float gain = __ldg(a.gain);
+    if (a.gain == nullptr) return;
+    const float gain = a.gain_per_col ? 1.f : __ldg(a.gain);
     const float rs = gain / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
     float rs_above = 0.f;
     if (shift && t > 0) rs_above = gain / sqrtf(cta_sum(ss_above, s_tmp) / (float)W + a.eps);
     T* h = static_cast<T*>(a.h);
     T* mixed = static_cast<T*>(a.mixed);
     for (int i = threadIdx.x; i < W; i += kRowThreads) {
-        const float hv = value(t, i) * rs;
+        const float ci = a.gain_per_col ? __ldg(a.gain + i) : 1.f;
+        const float hv = value(t, i) * rs * ci;
         if (h != nullptr) h[(size_t)t * W + i] = from_f32<T>(hv);
         if (shift) {
-            const float d = (t > 0 ? value(t - 1, i) * rs_above : a.prev_in[i]) - hv;
+            const float d = (t > 0 ? value(t - 1, i) * rs_above * ci : a.prev_in[i]) - hv;
             for (int m = 0; m < a.n_mix; ++m)
                 mixed[((size_t)m * a.rows + t) * W + i] = from_f32<T>(fmaf(d, __ldg(a.mu[m] + i), hv));
         }
@@ -75,11 +89,25 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_vec_kernel(const lean
     const D* delta = static_cast<const D*>(a.delta);
     T* h = static_cast<T*>(a.h);
     T* mixed = static_cast<T*>(a.mixed);
-    const bool shift = a.n_mix > 0;
-    const float gain = __ldg(a.gain);
+    const bool shift = a.n_mix > 0, post = a.post_gain != nullptr, per_col = a.gain_per_col != 0;
+    const float gain = a.gain == nullptr || per_col ? 1.f : __ldg(a.gain);
+    const float* scale = post ? a.post_gain : a.scale;
     float cur[NV][4], above[NV][4];
     auto load = [&](int row, bool store) -> float {       // the updated stream of `row` into cur; its norm factor
-        float ss = 0.f;
+        float ss = 0.f, f = 1.f;
+        if (post) {                                       // the branch is normed before it joins
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int i = (tid + n * kRowThreads) * 4;
+                if (i >= W) continue;
+                float dv[4];
+                fetch4(delta + (size_t)row * W + i, dv);
+#pragma unroll
+                for (int q = 0; q < 4; ++q) ss = fmaf(dv[q], dv[q], ss);
+            }
+            f = a.post_mult / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+            ss = 0.f;
+        }
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
             const int i = (tid + n * kRowThreads) * 4;
@@ -88,24 +116,33 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_vec_kernel(const lean
                 if (delta != nullptr) {
                     float dv[4], sv[4];
                     fetch4(delta + (size_t)row * W + i, dv);
-                    fetch4(a.scale + i, sv);
+                    fetch4(scale + i, sv);
 #pragma unroll
-                    for (int q = 0; q < 4; ++q) cur[n][q] = fmaf(dv[q], sv[q], cur[n][q]);
+                    for (int q = 0; q < 4; ++q) cur[n][q] = fmaf(dv[q] * f, sv[q], cur[n][q]);
                     if (store) store4(a.x_out + (size_t)row * W + i, cur[n]);
                 }
 #pragma unroll
                 for (int q = 0; q < 4; ++q) ss = fmaf(cur[n][q], cur[n][q], ss);
             }
         }
-        return gain / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+        return a.gain == nullptr ? 1.f : gain / sqrtf(cta_sum(ss, s_tmp) / (float)W + a.eps);
+    };
+    auto norm = [&](int n, float rs) {
+        const int i = (tid + n * kRowThreads) * 4;
+        float g[4] = {1.f, 1.f, 1.f, 1.f};
+        if (per_col && i < W) fetch4(a.gain + i, g);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) cur[n][q] *= rs * g[q];
     };
     if (shift) {
         if (r0 > 0) {
             const float rs = load(r0 - 1, false);
 #pragma unroll
-            for (int n = 0; n < NV; ++n)
+            for (int n = 0; n < NV; ++n) {
+                norm(n, rs);
 #pragma unroll
-                for (int q = 0; q < 4; ++q) above[n][q] = cur[n][q] * rs;
+                for (int q = 0; q < 4; ++q) above[n][q] = cur[n][q];
+            }
         } else {
 #pragma unroll
             for (int n = 0; n < NV; ++n) {
@@ -116,12 +153,12 @@ __global__ void __launch_bounds__(kRowThreads) stream_norm_vec_kernel(const lean
     }
     for (int row = r0; row < r1; ++row) {
         const float rs = load(row, true);
+        if (a.gain == nullptr) continue;
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
             const int i = (tid + n * kRowThreads) * 4;
             if (i >= W) continue;
-#pragma unroll
-            for (int q = 0; q < 4; ++q) cur[n][q] *= rs;
+            norm(n, rs);
             if (h != nullptr) store4(h + (size_t)row * W + i, cur[n]);
             if (shift) {
                 for (int m = 0; m < a.n_mix; ++m) {
@@ -190,11 +227,18 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float* in, T* out
     }
 }
 
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+    pdl_begin();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+        x[i] = cap * tanhf(x[i] / cap);
+}
+
 template <typename T, typename D>
 int launch_stream_norm(const leankv_stream_norm_t* a, cudaStream_t st) {
     bool vec = a->width % 4 == 0 && a->width <= kRowThreads * 4 * 8 && aligned16(a->x_in) && aligned16(a->x_out) &&
                aligned16(a->delta) && aligned16(a->scale) && aligned16(a->h) && aligned16(a->mixed) &&
-               aligned16(a->prev_in) && aligned16(a->prev_out);
+               aligned16(a->prev_in) && aligned16(a->prev_out) && aligned16(a->post_gain) &&
+               (!a->gain_per_col || aligned16(a->gain));
     for (int i = 0; i < a->n_mix; ++i) vec = vec && aligned16(a->mu[i]);
     if (!vec) {
         LEANKV_CUDA_TRY(launch_kernel(stream_norm_kernel<T, D>, dim3(a->rows), dim3(kRowThreads), 0, st, *a));
@@ -242,9 +286,10 @@ extern "C" int leankv_greedy_end(const float* logits, int vocab, long long* toke
 }
 
 extern "C" int leankv_stream_norm(const leankv_stream_norm_t* a, void* stream) {
-    if (!a || !a->x_in || !a->gain || a->rows <= 0 || a->width <= 0 || a->n_mix < 0 || a->n_mix > LEANKV_MAX_MIX)
-        return LEANKV_EINVAL;
-    if (a->delta && (!a->x_out || !a->scale || a->x_out == a->x_in)) return LEANKV_EINVAL;
+    if (!a || !a->x_in || a->rows <= 0 || a->width <= 0 || a->n_mix < 0 || a->n_mix > LEANKV_MAX_MIX) return LEANKV_EINVAL;
+    if (!a->gain && (a->h || a->n_mix > 0 || !a->delta)) return LEANKV_EINVAL;
+    if (a->delta && (!a->x_out || (!a->scale && !a->post_gain) || a->x_out == a->x_in)) return LEANKV_EINVAL;
+    if (a->post_gain && !a->delta) return LEANKV_EINVAL;
     if (a->n_mix > 0) {
         if (!a->mixed || !a->prev_in || !a->prev_out || a->prev_in == a->prev_out) return LEANKV_EINVAL;
         for (int i = 0; i < a->n_mix; ++i)
@@ -287,4 +332,11 @@ extern "C" int leankv_tanh_split(const float* in, void* out, int dtype, int rows
         return LEANKV_OK;
     };
     return dtype == LEANKV_DT_BF16 ? go(bf16{}) : go(float{});
+}
+
+extern "C" int leankv_softcap(float* x, long long n, float cap, void* stream) {
+    if (!x || n <= 0 || !(cap > 0.f)) return LEANKV_EINVAL;
+    const int grid = (int)std::min<long long>((n + 255) / 256, (long long)sm_count() * 8);
+    LEANKV_CUDA_TRY(launch_kernel(softcap_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream), x, n, cap));
+    return LEANKV_OK;
 }

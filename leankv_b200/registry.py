@@ -94,6 +94,7 @@ def _llama_model(config, tensors, device, dtype, max_seq_len, **kw):
     return DecodeEngine(cfg, DecodeEngine.shard_weights(full, cfg, 0, 1), device, max_seq_len=max_seq_len, **kw)
 
 
-register("Rorosun", ModelEntry("libleankv_mixers.so", ("bfloat16", "float32"), _mixer_model))
+for _name in ("Rorosun", "Pefitar"):
+    register(_name, ModelEntry("libleankv_mixers.so", ("bfloat16", "float32"), _mixer_model))
 for _name in ("LlamaForCausalLM", "MistralForCausalLM"):
     register(_name, ModelEntry("libleankv_b200.so", ("float16",), _llama_model))

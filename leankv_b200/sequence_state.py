@@ -1,5 +1,6 @@
-"""What one sequence keeps between steps in a model whose layers hold bounded state: rings of recent keys and
-values, pooled blocks of older ones, recurrent matrices, and the previous token's inputs.
+"""What one sequence keeps between steps in a mixer model: rings of keys and values (a window, or the whole
+sequence), latents with the key part all heads share, pooled blocks of older keys, recurrent matrices, and the
+previous token's inputs.
 
 Memory of a window + pooled-block layer does not grow with the raw sequence: the ring holds the window and
 one prompt portion, and every ``pool`` tokens add one pooled key / value per kv head.
@@ -8,6 +9,7 @@ one prompt portion, and every ``pool`` tokens add one pooled key / value per kv 
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -32,6 +34,20 @@ class WindowState:
         return self.k_pool.shape[0]
 
 
+RING_STEP = 128          # causal rings are a multiple of the prompt kernel's key tile
+
+
+@dataclass
+class CausalState:
+    k: torch.Tensor                        # [ring][kv_heads][pad16(dim)], position p in slot p % ring
+    v: Optional[torch.Tensor]              # [ring][kv_heads][pad16(vdim)]; None: values come from the keys (a latent)
+    shared: Optional[torch.Tensor]         # [ring][pad16(shared dim)]: the part of a key that all heads share
+
+    @property
+    def ring(self) -> int:
+        return self.k.shape[0]
+
+
 class SequenceState:
     """Allocates and resets the per-layer state of a single sequence of at most ``max_seq_len`` tokens that
     is fed in portions of at most ``max_chunk``."""
@@ -39,6 +55,7 @@ class SequenceState:
     def __init__(self, device, dtype: torch.dtype, max_seq_len: int, max_chunk: int):
         self.dev, self.dtype = device, dtype
         self.max_seq_len, self.max_chunk = max_seq_len, max_chunk
+        self.status = torch.zeros(1, dtype=torch.int32, device=device)      # set by a kernel whose wait ran out
         self._all: list[torch.Tensor] = []
         self._carried: list[torch.Tensor] = []       # state a new sequence starts from zero
 
@@ -55,6 +72,15 @@ class SequenceState:
                            self._new(ring, kv_heads, vd, dtype=self.dtype),
                            self._new(blocks, kv_heads, kd, dtype=self.dtype),
                            self._new(blocks, kv_heads, vd, dtype=self.dtype))
+
+    def causal(self, kv_heads: int, dim: int, vdim: int, shared: int, size: int) -> CausalState:
+        """``size``: visible positions (a window, or at least ``max_seq_len`` for the whole sequence); a portion is
+        appended whole before it attends. ``vdim`` or ``shared`` 0: not there."""
+        slots = min(size + self.max_chunk - 1, self.max_seq_len)
+        ring = (slots + RING_STEP - 1) // RING_STEP * RING_STEP
+        return CausalState(self._new(ring, kv_heads, pad16(dim), dtype=self.dtype),
+                           self._new(ring, kv_heads, pad16(vdim), dtype=self.dtype) if vdim else None,
+                           self._new(ring, pad16(shared), dtype=self.dtype) if shared else None)
 
     def carried(self, *shape: int) -> torch.Tensor:
         """fp32 state that is updated in place token by token and is zero before the first."""
