@@ -1184,11 +1184,11 @@ def main():
     ap.add_argument("--no-comparators", action="store_true", help="skip the GPU comparator legs of the default run")
     ap.add_argument("--only-exchange", action="store_true",
                     help="under torchrun: time the GEMV + all-reduce leg alone and print its JSON")
-    ap.add_argument("--workload", choices=["decode", "batched", "rorosun"], default="decode",
+    ap.add_argument("--workload", choices=["decode", "batched", "rorosun", "pefitar"], default="decode",
                     help="decode: batch-1 TEAL + TurboQuant decode loop (the headline metric), with a short "
                          "batched leg attached; batched: only the 80-sequence long-context decode, its own line; "
-                         "rorosun: the mixer engine beside the closest model at a few layer sizes")
-    ap.add_argument("--sizes", default="1k,2k,4k", help="with --workload rorosun: layer sizes to run")
+                         "rorosun, pefitar: the mixer engine beside the closest model at a few layer sizes")
+    ap.add_argument("--sizes", default="1k,2k,4k", help="with --workload rorosun or pefitar: layer sizes to run")
     ap.add_argument("--no-batched", action="store_true", help="skip the batched-decode leg of the default run")
     ap.add_argument("--batched-steps", type=int, default=32)
     args = ap.parse_args()
@@ -1215,7 +1215,7 @@ def main():
         dist.destroy_process_group()
     elif args.workload == "batched":
         run_batched(args)
-    elif args.workload == "rorosun":
+    elif args.workload in ("rorosun", "pefitar"):
         import bench_mixers
 
         bench_mixers.run(args, ClockSampler)

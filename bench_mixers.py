@@ -1,6 +1,6 @@
-"""``bench.py --workload rorosun``: the mixer engine beside the framework's closest model at equal size.
+"""``bench.py --workload {rorosun,pefitar}``: the mixer engine beside the framework's closest model at equal size.
 
-For a few layer sizes (random weights): prefill and decode throughput of a Rorosun model and of the
+For a few layer sizes (random weights): prefill and decode throughput of a Rorosun or Pefitar model and of the
 Llama-shaped TEAL + TurboQuant engine with the same width, attention heads and feed-forward (TEAL off: both
 stream every weight), then every hot kernel alone with its share of the roofline, next to the like kernel of
 the other engine. Launches rotate over the layers, whose weights exceed L2 together.
@@ -17,6 +17,7 @@ ROOT = os.path.dirname(os.path.abspath(__file__))
 # name -> width, attention heads / kv heads (x 128), time-mixing heads (x 64), ff, layers
 SIZES = {"1k": (1024, 8, 2, 16, 3584, 24), "2k": (2048, 16, 4, 32, 7168, 12), "4k": (4096, 32, 8, 64, 14336, 6)}
 VOCAB, WINDOW, POOL, PROMPT = 32768, 1024, 16, 2048
+KV_RANK, ROT_DIM, LONG = 512, 64, 32768          # Pefitar's latent layers; positions of the long-context step
 
 
 def model_config(width, heads, kv, right, ff, layers):
@@ -25,6 +26,19 @@ def model_config(width, heads, kv, right, ff, layers):
              "right": {"heads": right, "dim": 64}, "left_scale": 0.7, "right_scale": 0.7}
     return {"architecture": "Rorosun", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5},
             "layers": [{"type": "parallel", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}}] * layers}
+
+
+def pefitar_config(width, heads, kv, _, ff, layers):
+    """Attention and latent-attention layers in turn."""
+    rot = lambda dims: {"base": 10000.0, "dims": dims}
+    mlp = {"kind": "dense", "ff": ff}
+    attn = {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128,
+                                                       "scale": 128 ** -0.5, "rot": rot(128)}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": ROT_DIM, "vdim": 128, "q_rank": width // 2, "kv_rank": KV_RANK,
+        "mask": {"size": WINDOW}, "scale": (128 + ROT_DIM) ** -0.5, "rot": rot(ROT_DIM)}}
+    return {"architecture": "Pefitar", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5},
+            "layers": [attn, latent] * (layers // 2), "residual_mult": 0.5, "logit_softcap": 30.0}
 
 
 def _timed(fn, n_variants, iters, warmup=5):
@@ -151,6 +165,82 @@ def mixer_leg(size, dev, steps, peaks):
     return out
 
 
+def pefitar_leg(size, dev, steps, peaks):
+    import torch
+
+    from leankv_b200 import _native
+    from leankv_b200.mixer_engine import MixerDecodeEngine, MixerModelConfig
+    from leankv_b200.mixers import pad16
+
+    width, heads, kv, _, ff, layers = SIZES[size]
+    cfg = MixerModelConfig.from_dict(pefitar_config(*SIZES[size]))
+    eng = MixerDecodeEngine(cfg, MixerDecodeEngine.random_tensors(cfg, dev), dev, max_seq_len=LONG, max_chunk=PROMPT)
+    prompt = torch.randint(0, VOCAB, (PROMPT,), generator=torch.Generator().manual_seed(1)).tolist()
+
+    def prefill():
+        eng.reset()
+        return eng.extend(prompt, [PROMPT - 1])
+    pre, dec = _loops(eng, prompt, steps, prefill)
+    lib, hbm, tflops = eng.lib, *peaks
+    out = {"prefill_tok_s": pre, "decode_tok_s": dec, "launches_per_step": eng.launches_per_step,
+           "state_bytes": eng.seq.bytes(), "kernels": {}}
+    st = lambda: torch.cuda.current_stream().cuda_stream
+    runs, attn, latent = eng.layers, eng.layers[0::2], eng.layers[1::2]
+    n = len(attn)
+
+    def mem(name, seconds, nbytes):
+        out["kernels"][name] = {"us": seconds * 1e6, "gbs": nbytes / seconds / 1e9, "frac": nbytes / seconds / 1e9 / hbm,
+                                "bound": "hbm"}
+
+    def math_(name, seconds, flops):
+        out["kernels"][name] = {"us": seconds * 1e6, "tflops": flops / seconds / 1e12,
+                                "frac": flops / seconds / 1e12 / tflops, "bound": "tensor"}
+
+    gemv = lambda a: _native.check(lib.leankv_dense_gemv(ctypes.byref(a), st()), "gemv", lib)
+    A, L = attn[0].mixer, latent[0].mixer
+    mem("gemv_qkvg_join_norm", _graphed(lambda i: gemv(attn[i].mixer._step_args[0]), n), 2 * A.w_in.numel())
+    mem("gemv_out", _graphed(lambda i: gemv(attn[i].mixer._step_args[2]), n), 2 * A.w_out.numel())
+    for k, name, w in ((0, "gemv_latent_in", L.w_down), (1, "gemv_latent_q", L.w_q), (2, "gemv_latent_fold", L.w_fold),
+                       (4, "gemv_latent_unfold", L.w_unfold), (5, "gemv_latent_out", L.w_out)):
+        mem(name, _graphed(lambda i: gemv(latent[i].mixer._step_args[k]), n), 2 * w.numel())
+    mem("gemv_gate_up_silu", _graphed(lambda i: gemv(runs[i].mlp._step_args[0]), layers), 2 * runs[0].mlp.w_gu.numel())
+    mem("gemv_down", _graphed(lambda i: gemv(runs[i].mlp._step_args[1]), layers), 2 * runs[0].mlp.w_down.numel())
+    mem("gemv_head", _graphed(lambda i: gemv(eng._head_args), 4), 2 * eng.head.numel())
+
+    def step(r, k):
+        m = r.mixer
+        _native.check(lib.leankv_causal_step(ctypes.byref(m.c), ctypes.byref(m._step_args[k]), st()), "causal_step", lib)
+    for name, pos in (("causal_step", eng.pos), ("causal_step_32k", LONG - 1)):
+        eng.state[0] = pos
+        mem(name, _graphed(lambda i: step(attn[i], 1), n), 2 * pos * kv * 256)
+    mem("causal_step_latent", _graphed(lambda i: step(latent[i], 3), n), 2 * WINDOW * (KV_RANK + ROT_DIM))
+
+    # prompt kernels on a portion of PROMPT tokens
+    T, W = PROMPT, width
+    x, d = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+    h = torch.empty(T, W, dtype=eng.dtype, device=dev)
+    mem("stream_norm_join", _graphed(lambda i: eng._stream_norm(x, runs[i].second.norm, h, d, runs[i].second), layers),
+        T * W * (4 * 3 + 2))
+    gu = torch.randn(T, 2 * ff, device=dev).bfloat16()
+    act = torch.empty(T, ff, dtype=eng.dtype, device=dev)
+    mem("silu_mul", _graphed(lambda i: lib.leankv_silu_mul(gu.data_ptr(), act.data_ptr(), 1, T, ff, st()), 4), T * ff * 6)
+    y = torch.randn(T, A.in_width, device=dev)
+    mem("place_rows", _graphed(lambda i: attn[i].mixer.place(y, 0), n), T * A.at_g * 6)
+    q = attn[0].mixer.place(y, 0)
+    gate = y[:, A.at_g:]
+    math_("causal_attend", _graphed(lambda i: attn[i].mixer._attend(attn[i].mixer.c, q, gate, 0), n),
+          2 * T * (T + 1) // 2 * heads * 256)
+    z = torch.randn(T, heads * (128 + ROT_DIM), device=dev)
+    ql = L.place_q(z, 0)
+    mem("place_rows_latent_q", _graphed(lambda i: latent[i].mixer.place_q(z, 0), n), T * z.shape[1] * 6)
+    math_("latent_expand", _graphed(lambda i: latent[i].mixer._expanded(0, T), n), 2 * T * KV_RANK * heads * 256)
+    e, keep = L._expanded(0, T)
+    pairs = sum(min(i + 1, WINDOW) for i in range(T))
+    math_("causal_attend_latent", _graphed(lambda i: L._attend(e, ql, None, 0), n), 2 * pairs * heads * (256 + ROT_DIM))
+    del keep
+    return out
+
+
 def llama_leg(size, dev, steps, peaks):
     """The Llama-shaped engine (3-bit KV pages, TEAL off) at the same width, heads, ff and layers."""
     import torch
@@ -228,20 +318,23 @@ def run(args, sampler_cls):
     sizes = [s for s in args.sizes.split(",") if s]
     sampler = sampler_cls(0)
     sampler.start()
-    result = {}
+    result, name = {}, args.workload
+    legs = {"rorosun": mixer_leg, "pefitar": pefitar_leg}
     for s in sizes:
-        result[s] = {"rorosun": mixer_leg(s, dev, steps, peaks)}
+        result[s] = {name: legs[name](s, dev, steps, peaks)}
         torch.cuda.empty_cache()
         result[s]["llama_same_size"] = llama_leg(s, dev, steps, peaks)
         torch.cuda.empty_cache()
     sampler.stop()
-    last = result[sizes[-1]]["rorosun"]
+    last = result[sizes[-1]][name]
+    more = {"pool": POOL} if name == "rorosun" else {"kv_rank": KV_RANK, "rot_dim": ROT_DIM, "long_context": LONG}
+    columns = ("width", "heads", "kv_heads", "time_mix_heads" if name == "rorosun" else None, "ff", "layers")
     print(json.dumps({
-        "metric": "B=1 decode tok/s (Rorosun layers, largest size)", "value": last["decode_tok_s"], "unit": "tok/s",
-        "n_gpus": 1, "steps": steps, "warmup": 8, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
-        "data": "synthetic", "clocks": sampler.summary(), "peaks": {"hbm_gbs": peaks[0], "bf16_tflops": peaks[1],
-                                                                    "source": source},
-        "config": {"sizes": {s: dict(zip(("width", "heads", "kv_heads", "time_mix_heads", "ff", "layers"), SIZES[s]))
-                             for s in sizes}, "vocab": VOCAB, "window": WINDOW, "pool": POOL, "prompt_len": PROMPT,
+        "metric": f"B=1 decode tok/s ({name.capitalize()} layers, largest size)", "value": last["decode_tok_s"],
+        "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": 8, "higher_is_better": True, "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic", "clocks": sampler.summary(),
+        "peaks": {"hbm_gbs": peaks[0], "bf16_tflops": peaks[1], "source": source},
+        "config": {"sizes": {s: {c: v for c, v in zip(columns, SIZES[s]) if c} for s in sizes},
+                   "vocab": VOCAB, "window": WINDOW, "prompt_len": PROMPT, **more,
                    "l2": "launches rotate over the layers; their weights exceed L2 together"},
         "sizes": result}))

@@ -240,7 +240,6 @@ typedef struct leankv_causal_step {
     int max_pos;
     void* ws;
     size_t ws_bytes;
-    int32_t* status;
 } leankv_causal_step_t;
 
 size_t leankv_causal_step_workspace_bytes(const leankv_causal_attn_t* a, int max_pos);

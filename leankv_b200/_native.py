@@ -219,7 +219,7 @@ class CausalStep(Structure):
                 ("v_new", c_void_p), ("q_stride", c_int), ("qs_stride", c_int),
                 ("k_gain", c_void_p), ("eps", c_float), ("rate", c_void_p), ("rot_own", c_int), ("rot_shared", c_int),
                 ("gate", c_void_p), ("out", c_void_p), ("state", c_void_p), ("max_pos", c_int),
-                ("ws", c_void_p), ("ws_bytes", c_size_t), ("status", c_void_p)]
+                ("ws", c_void_p), ("ws_bytes", c_size_t)]
 
 
 MIXER_SIGNATURES = {

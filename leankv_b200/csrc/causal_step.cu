@@ -1,19 +1,23 @@
 // One decode step of causal attention over a ring of keys, split over the keys. A CTA takes up to 16 query heads of one
-// kv head and a range of 64-key tiles: the rows of a tile come by bulk copies through a few stages, so several
-// tiles are in flight while one is computed, and the first ones are on their way before the launch ahead has
-// finished. The last CTA of a head block to finish merges the partial outputs (in split order) and gates them.
+// kv head and a range of 64-key tiles, which come by asynchronous copies through a few stages; the first are on their
+// way before the launch ahead has finished. The CTAs of a cluster merge their outputs through distributed
+// shared memory, each a slice of the columns. A long sequence takes several clusters per head block: there the
+// last cluster to finish a slice merges the clusters' results, in cluster order.
 //
 // bf16: scores and outputs on tensor cores (16 heads x 8 keys, 16 heads x 8 columns). Queries and softmax weights enter
 // as two bf16 numbers each, so a 32-bit query meets the stored keys exactly. fp32: the same walk on FMA units.
 
 #include <algorithm>
 
+#include <cooperative_groups.h>
+
 #include "causal_attn.cuh"
 #include "decode_frame.cuh"
-#include "umma.cuh"
 
 namespace leankv {
 namespace {
+
+namespace cg = cooperative_groups;
 
 constexpr int kWarps = 8;
 constexpr int kThreads = 32 * kWarps;
@@ -21,6 +25,8 @@ constexpr int kHeads = 16;                // query heads of a CTA
 constexpr int kMaxStages = 4;
 constexpr int kMaxCols = 1024;            // value columns
 constexpr int kMaxPairs = 512;            // rotated pairs
+constexpr int kMaxCluster = 16;           // non-portable; 8 where the device does not place 16
+constexpr int kTilesPerCta = 4;           // a further cluster joins when every CTA would have more tiles
 
 template <typename T> constexpr int kTileOf = sizeof(T) == 2 ? 64 : 32;      // keys of a tile
 
@@ -28,7 +34,7 @@ template <typename T> constexpr int kTileOf = sizeof(T) == 2 ? 64 : 32;      // 
 // fragment fall into different banks.
 struct StepPlan {
     int k_row, v_row, stages, stage_bytes;             // bytes of a key row (own part, then shared), of a value row
-    int q, q_row, s, p, stat, trig, fresh, stage, total;
+    int q, q_row, s, p, stat, factor, trig, fresh, stage, total;
     __host__ __device__ static constexpr int row(int bytes) { return (bytes + 127) / 128 * 128 + 16; }
     __host__ __device__ StepPlan(const leankv_causal_attn_t& a, int tile, int limit) {
         const int es = a.dtype == LEANKV_DT_BF16 ? 2 : 4, kd = a.dim_pad + a.shared_pad;
@@ -41,12 +47,15 @@ struct StepPlan {
         s = take(kHeads * (tile + 4) * 4);
         p = take(kHeads * row(tile * 2) * 2);
         stat = take(kHeads * 4 * 4);                    // maximum, sum, rescale factor
+        factor = take(kHeads * kMaxCluster * 4 + kHeads * 8);
         trig = take(kMaxPairs * 8);
         fresh = take(k_row + v_row);
         stage = o;
         stage_bytes = (tile * (k_row + v_row) + 127) / 128 * 128;
         stages = (limit - o) / stage_bytes;
         if (stages > kMaxStages) stages = kMaxStages;
+        const int out = kHeads * a.vdim_pad * 4;        // the outputs take the stages' place
+        if (stages * stage_bytes < out) stages = 0;
         total = o + stages * stage_bytes;
     }
 };
@@ -54,16 +63,15 @@ struct StepPlan {
 struct StepArgs {
     leankv_causal_attn_t a;
     leankv_causal_step_t s;
-    int blocks, splits, limit;            // head blocks per kv head, splits, shared memory
-    float* part;                          // [kv head][block][split][kHeads][vdim_pad]
-    float* ml;                            // [kv head][block][split][kHeads][2]
-    unsigned* tickets;                    // [kv head][block]
+    int blocks, cluster, clusters, limit; // head blocks per kv head, CTAs of a cluster, clusters of a head block
+    float* part;                          // [head block][cluster][kHeads][vdim_pad]
+    float* ml;                            // [head block][cluster][rank][kHeads][2]
+    unsigned* tickets;                    // [head block][rank]
 };
 
-__device__ __forceinline__ void bulk_row(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src),
-                 "r"(bytes), "r"(bar)
-                 : "memory");
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void copy16(uint32_t dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
 __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -78,9 +86,8 @@ __device__ __forceinline__ void ldmatrix4_t(uint32_t (&r)[4], uint32_t addr) {
 
 // NP: 16-column pieces of the values that a warp accumulates at most (bf16).
 template <typename T, int NP>
-__global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(const __grid_constant__ StepArgs p) {
+__global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) causal_step_kernel(const __grid_constant__ StepArgs p) {
     extern __shared__ __align__(128) unsigned char sm[];
-    __shared__ __align__(8) uint64_t s_bar[kMaxStages];
     __shared__ float s_tmp[32];
     __shared__ int s_last;
     constexpr bool HALF = sizeof(T) == 2;
@@ -88,46 +95,45 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
     const leankv_causal_attn_t& a = p.a;
     const StepPlan pl(a, KT, p.limit);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int g = blockIdx.y / p.blocks, hb = blockIdx.y % p.blocks, rep = a.heads / a.kv_heads;
+    const int gb = blockIdx.y, g = gb / p.blocks, hb = gb % p.blocks, rep = a.heads / a.kv_heads;
     const int h0 = g * rep + hb * kHeads, nh = min(kHeads, rep - hb * kHeads);
+    const int C = p.cluster, rank = blockIdx.x % C, cluster = blockIdx.x / C;
     const int i = p.s.state[kPos], lo = first_visible(i, a.size), n = i + 1 - lo, tiles = (n + KT - 1) / KT;
-    const int active = min(p.splits, tiles), split = blockIdx.x;
-    if (split >= active) {
+    const int active = max(1, min(p.clusters, (tiles + C * kTilesPerCta - 1) / (C * kTilesPerCta)));
+    if (cluster >= active) {
         pdl_begin();
         return;
     }
-    const int j0 = (int)((long long)tiles * split / active), j1 = (int)((long long)tiles * (split + 1) / active);
+    const int split = cluster * C + rank, splits = active * C;
+    const int j0 = (int)((long long)tiles * split / splits), j1 = (int)((long long)tiles * (split + 1) / splits);
     const int kd = a.dim_pad + a.shared_pad;
     const T* K = static_cast<const T*>(a.k);
     const T* V = static_cast<const T*>(a.v);
     const T* S = static_cast<const T*>(a.shared);
-    auto bar = [&](int s) { return umma::smem_addr(&s_bar[s]); };
-    if (tid < pl.stages) umma::bar_init_n(bar(tid), 1);
-    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    __syncthreads();
 
-    // tile j into its stage; the position of this step is not in the ring yet
-    auto fetch = [&](int j) {                             // warp 0
-        const int st = (j - j0) % pl.stages, first = lo + j * KT, cnt = min(KT, i - first);       // rows that are in the ring
-        const uint32_t row_bytes = (uint32_t)(kd + (V != nullptr ? a.vdim_pad : 0)) * sizeof(T);
-        if (lane == 0)
-            asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar(st)), "r"((uint32_t)max(cnt, 0) * row_bytes)
-                         : "memory");
-        __syncwarp();
-        const uint32_t kb = umma::smem_addr(sm + pl.stage + st * pl.stage_bytes), vb = kb + KT * pl.k_row;
-        for (int r = lane; r < cnt; r += 32) {
-            const size_t slot = ring_slot(first + r, a.k_base, a.k_ring);
-            bulk_row(kb + r * pl.k_row, K + (slot * a.kv_heads + g) * a.dim_pad, a.dim_pad * sizeof(T), bar(st));
-            if (a.shared_dim > 0)
-                bulk_row(kb + r * pl.k_row + a.dim_pad * sizeof(T), S + (size_t)ring_slot(first + r, 0, a.s_ring) * a.shared_pad,
-                         a.shared_pad * sizeof(T), bar(st));
-            if (V != nullptr)
-                bulk_row(vb + r * pl.v_row, V + (slot * a.kv_heads + g) * a.vdim_pad, a.vdim_pad * sizeof(T), bar(st));
+    // tile j into its stage, a warp a row; the position of this step is not in the ring yet
+    constexpr int E16 = 16 / (int)sizeof(T);
+    const int c_own = a.dim_pad / E16, c_key = kd / E16, c_all = c_key + (V != nullptr ? a.vdim_pad / E16 : 0);
+    auto fetch = [&](int j) {
+        if (j < j1) {
+            const int st = (j - j0) % pl.stages, first = lo + j * KT, cnt = min(KT, i - first);
+            const uint32_t kb = smem_addr(sm + pl.stage + st * pl.stage_bytes), vb = kb + KT * pl.k_row;
+            const int slot0 = ring_slot(first, a.k_base, a.k_ring), sslot0 = a.shared_dim > 0 ? ring_slot(first, 0, a.s_ring) : 0;
+            for (int r = warp; r < cnt; r += kWarps) {
+                int slot = slot0 + r, sslot = sslot0 + r;           // a window fits into the ring once
+                if (slot >= a.k_ring) slot -= a.k_ring;
+                if (sslot >= a.s_ring) sslot -= a.s_ring;
+                const T* k_src = K + ((size_t)slot * a.kv_heads + g) * a.dim_pad;
+                for (int c = lane; c < c_all; c += 32) {
+                    if (c < c_own) copy16(kb + r * pl.k_row + c * 16, k_src + c * E16);
+                    else if (c < c_key) copy16(kb + r * pl.k_row + c * 16, S + (size_t)sslot * a.shared_pad + (c - c_own) * E16);
+                    else copy16(vb + r * pl.v_row + (c - c_key) * 16, V + ((size_t)slot * a.kv_heads + g) * a.vdim_pad + (c - c_key) * E16);
+                }
+            }
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    int issued = j0;
-    for (; issued < j1 && issued < j0 + pl.stages; ++issued)
-        if (warp == 0) fetch(issued);
+    for (int x = 0; x < pl.stages; ++x) fetch(j0 + x);
     float* s_sin = reinterpret_cast<float*>(sm + pl.trig);
     float* s_cos = s_sin + kMaxPairs;
     for (int x = tid; x < max(p.s.rot_own, p.s.rot_shared) / 2; x += kThreads)
@@ -137,16 +143,27 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
 
     // ---- queries, and the new key / value row ----
     const float c = a.scale * 1.4426950408889634f;        // scores in units of log2
-    auto pair_at = [&](const float* x, int d, int dim, int rot) {
-        float2 v = make_float2(d < dim ? ld_cg_f32(x + d) : 0.f, d + 1 < dim ? ld_cg_f32(x + d + 1) : 0.f);
-        return d < rot ? turn(v.x, v.y, s_sin[d >> 1], s_cos[d >> 1]) : v;
+    auto pair_of = [&](const float* x, int d, int dim) {
+        return make_float2(d < dim ? __ldcg(x + d) : 0.f, d + 1 < dim ? __ldcg(x + d + 1) : 0.f);
     };
-    for (int e = tid; e < kHeads * (kd / 2); e += kThreads) {
-        const int h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
-        float2 v = make_float2(0.f, 0.f);
+    auto turned = [&](float2 v, int d, int rot) { return d < rot ? turn(v.x, v.y, s_sin[d >> 1], s_cos[d >> 1]) : v; };
+    auto pair_at = [&](const float* x, int d, int dim, int rot) { return turned(pair_of(x, d, dim), d, rot); };
+    constexpr int kBatch = 6;                             // loads in flight per thread
+    for (int e0 = tid; e0 < kHeads * (kd / 2); e0 += kBatch * kThreads) {
+      float2 in[kBatch];
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
+        in[x] = make_float2(0.f, 0.f);
         if (h < nh)
-            v = d < a.dim_pad ? pair_at(p.s.q + (size_t)(h0 + h) * p.s.q_stride, d, a.dim, p.s.rot_own)
-                              : pair_at(p.s.q_shared + (size_t)(h0 + h) * p.s.qs_stride, d - a.dim_pad, a.shared_dim, p.s.rot_shared);
+            in[x] = d < a.dim_pad ? pair_of(p.s.q + (size_t)(h0 + h) * p.s.q_stride, d, a.dim)
+                                  : pair_of(p.s.q_shared + (size_t)(h0 + h) * p.s.qs_stride, d - a.dim_pad, a.shared_dim);
+      }
+#pragma unroll
+      for (int x = 0; x < kBatch; ++x) {
+        const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
+        if (h >= kHeads) break;
+        const float2 v = d < a.dim_pad ? turned(in[x], d, p.s.rot_own) : turned(in[x], d - a.dim_pad, p.s.rot_shared);
         if constexpr (HALF) {
             uint32_t hi, low;
             split_bf16(v.x, v.y, hi, low);
@@ -155,8 +172,9 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
         } else {
             *reinterpret_cast<float2*>(sm + pl.q + h * pl.q_row + d * 4) = v;
         }
+      }
     }
-    const bool newest = j1 == tiles;                      // this CTA's range ends with the new position
+    const bool newest = j0 < j1 && j1 == tiles;                      // this CTA's range ends with the new position
     T* fresh = reinterpret_cast<T*>(sm + pl.fresh);
     if (newest) {
         float f = 1.f;
@@ -164,7 +182,7 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
         if (p.s.k_gain != nullptr) {
             float ss = 0.f;
             for (int d = tid; d < a.dim; d += kThreads) {
-                const float v = ld_cg_f32(kn + d);
+                const float v = __ldcg(kn + d);
                 ss = fmaf(v, v, ss);
             }
             f = 1.f / sqrtf(cta_sum(ss, s_tmp) / (float)a.dim + p.s.eps);
@@ -177,8 +195,8 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
             const bool own = d < a.dim_pad;
             float2 v;
             if (own && p.s.k_gain != nullptr)
-                v = make_float2(d < a.dim ? ld_cg_f32(kn + d) * f * __ldg(p.s.k_gain + d) : 0.f,
-                                d + 1 < a.dim ? ld_cg_f32(kn + d + 1) * f * __ldg(p.s.k_gain + d + 1) : 0.f);
+                v = make_float2(d < a.dim ? __ldcg(kn + d) * f * __ldg(p.s.k_gain + d) : 0.f,
+                                d + 1 < a.dim ? __ldcg(kn + d + 1) * f * __ldg(p.s.k_gain + d + 1) : 0.f);
             else
                 v = own ? pair_at(kn, d, a.dim, p.s.rot_own) : pair_at(p.s.shared_new, d - a.dim_pad, a.shared_dim, p.s.rot_shared);
             fresh[d] = from_f32<T>(v.x);
@@ -193,7 +211,7 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
             T* fv = reinterpret_cast<T*>(sm + pl.fresh + pl.k_row);
             T* v_out = static_cast<T*>(a.v) + (slot * a.kv_heads + g) * a.vdim_pad;
             for (int d = tid; d < a.vdim_pad; d += kThreads) {
-                const T v = from_f32<T>(d < a.vdim ? ld_cg_f32(p.s.v_new + (size_t)g * a.vdim + d) : 0.f);
+                const T v = from_f32<T>(d < a.vdim ? __ldcg(p.s.v_new + (size_t)g * a.vdim + d) : 0.f);
                 fv[d] = v;
                 if (hb == 0) v_out[d] = v;
             }
@@ -224,13 +242,17 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
 #pragma unroll
             for (int h = 0; h < kHeads; ++h) of[x][h] = 0.f;
     }
-    bool ok = true;
     for (int j = j0; j < j1; ++j) {
-        const int st = (j - j0) % pl.stages, round = (j - j0) / pl.stages, first = lo + j * KT, cnt = min(KT, i + 1 - first);
+        const int st = (j - j0) % pl.stages, first = lo + j * KT, cnt = min(KT, i + 1 - first);
         unsigned char* kt = sm + pl.stage + st * pl.stage_bytes;
         unsigned char* vt = V != nullptr ? kt + KT * pl.k_row : kt;
         const int v_row = V != nullptr ? pl.v_row : pl.k_row;
-        ok = ok && umma::bar_wait(bar(st), round & 1);
+        switch (pl.stages) {                              // all but the newer groups have landed
+            case 1: asm volatile("cp.async.wait_group 0;" ::: "memory"); break;
+            case 2: asm volatile("cp.async.wait_group 1;" ::: "memory"); break;
+            case 3: asm volatile("cp.async.wait_group 2;" ::: "memory"); break;
+            default: asm volatile("cp.async.wait_group 3;" ::: "memory"); break;
+        }
         if (j == tiles - 1) {                             // the new row, and zeros behind it
             const int words = (KT - cnt + 1) * (pl.k_row / 4), words_v = V != nullptr ? (KT - cnt + 1) * (pl.v_row / 4) : 0;
             for (int e = tid; e < words; e += kThreads)
@@ -241,13 +263,13 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
                     e < pl.v_row / 4 && e * 4 < a.vdim_pad * (int)sizeof(T)
                         ? reinterpret_cast<const uint32_t*>(sm + pl.fresh + pl.k_row)[e]
                         : 0u;
-            __syncthreads();
         }
+        __syncthreads();
         // scores
         if constexpr (HALF) {
             float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint32_t qa = umma::smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
-            const uint32_t ka = umma::smem_addr(kt) + (warp * 8 + (lane & 7)) * pl.k_row + (lane >> 3) * 16;
+            const uint32_t qa = smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
+            const uint32_t ka = smem_addr(kt) + (warp * 8 + (lane & 7)) * pl.k_row + (lane >> 3) * 16;
             for (int d = 0; d < kd; d += 32) {
                 uint32_t b[4], qh[4], ql[4];
                 const bool two = d + 16 < kd;             // the last block may hold 16 dimensions
@@ -321,7 +343,7 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
         if constexpr (HALF) {
             constexpr int PROW = StepPlan::row(KT * 2);
             const float f0 = stat[2 * kHeads + (lane >> 2)], f1 = stat[2 * kHeads + (lane >> 2) + 8];
-            const uint32_t pa = umma::smem_addr(sm + pl.p) + (lane & 15) * PROW + (lane >> 4) * 16;
+            const uint32_t pa = smem_addr(sm + pl.p) + (lane & 15) * PROW + (lane >> 4) * 16;
             uint32_t wh[KT / 16][4], wl[KT / 16][4];
 #pragma unroll
             for (int k = 0; k < KT / 16; ++k) {
@@ -337,7 +359,7 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
                     o[x][y][0] *= f0; o[x][y][1] *= f0;
                     o[x][y][2] *= f1; o[x][y][3] *= f1;
                 }
-                const uint32_t va = umma::smem_addr(vt) + (lane & 15) * v_row + col * 2 + (lane >> 4) * 16;
+                const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + col * 2 + (lane >> 4) * 16;
 #pragma unroll
                 for (int k = 0; k < KT / 16; ++k) {
                     uint32_t b[4];                        // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
@@ -365,29 +387,13 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
             }
         }
         __syncthreads();
-        if (issued < j1) {                                // this stage is free again
-            if (warp == 0) {
-                umma::fence_operands();
-                fetch(issued);
-            }
-            ++issued;
-        }
+        fetch(j + pl.stages);                             // this stage is free again
     }
-    if (!ok && p.s.status != nullptr && tid == 0) *p.s.status = 1;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
 
-    // ---- partial results, merged by the last CTA of the head block ----
-    const int gb = blockIdx.y;
-    auto finish = [&](int h, int d, float v) {            // v: normalised
-        const int at = (h0 + h) * a.vdim + d;
-        if (p.s.gate != nullptr) v *= sigmoid_f32(ld_cg_f32(p.s.gate + at));
-        p.s.out[at] = v;
-    };
-    float* part = p.part + ((size_t)gb * p.splits + split) * kHeads * a.vdim_pad;
-    auto put = [&](int h, int d, float v) {
-        if (h >= nh || d >= a.vdim) return;
-        if (active == 1) finish(h, d, v / stat[kHeads + h]);
-        else part[h * a.vdim_pad + d] = v;
-    };
+    // ---- merge: this CTA's outputs into shared memory, then a slice of the columns of all CTAs of the cluster ----
+    float* s_o = reinterpret_cast<float*>(sm + pl.stage);             // [kHeads][vdim_pad]
+    auto put = [&](int h, int d, float v) { s_o[h * a.vdim_pad + d] = v; };
     if constexpr (HALF) {
 #pragma unroll
         for (int x = 0; x < NP; ++x) {
@@ -396,7 +402,9 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
 #pragma unroll
             for (int y = 0; y < 2; ++y)
 #pragma unroll
-                for (int z = 0; z < 4; ++z) put((lane >> 2) + (z < 2 ? 0 : 8), col + y * 8 + (lane & 3) * 2 + (z & 1), o[x][y][z]);
+                for (int z = 0; z < 2; ++z)
+                    *reinterpret_cast<float2*>(s_o + ((lane >> 2) + z * 8) * a.vdim_pad + col + y * 8 + (lane & 3) * 2) =
+                        make_float2(o[x][y][2 * z], o[x][y][2 * z + 1]);
         }
     } else {
 #pragma unroll
@@ -407,56 +415,84 @@ __global__ void __launch_bounds__(kThreads, NP <= 1 ? 2 : 1) causal_step_kernel(
             for (int h = 0; h < kHeads; ++h) put(h, d, of[x][h]);
         }
     }
-    if (active == 1) return;
-    float* ml = p.ml + (size_t)gb * p.splits * kHeads * 2;
-    if (tid < nh) {
-        ml[(split * kHeads + tid) * 2] = stat[tid];
-        ml[(split * kHeads + tid) * 2 + 1] = stat[kHeads + tid];
-    }
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) s_last = atomicAdd(p.tickets + gb, 1u) == (unsigned)active - 1;
-    __syncthreads();
-    if (!s_last) return;
-    __threadfence();
-    if (tid == 0) p.tickets[gb] = 0;
-    float* factor = reinterpret_cast<float*>(sm + pl.q);            // [nh][active], room checked on the host
-    for (int h = warp; h < nh; h += kWarps) {
-        float best = -1e30f, l = 0.f;
-        for (int s = lane; s < active; s += 32) best = fmaxf(best, __ldcg(ml + (s * kHeads + h) * 2));
-        best = warp_max(best);
-        for (int s = lane; s < active; s += 32) {
-            const float f = exp2f(__ldcg(ml + (s * kHeads + h) * 2) - best);
-            factor[h * active + s] = f;
-            l += f * __ldcg(ml + (s * kHeads + h) * 2 + 1);
+    auto cl = cg::this_cluster();
+    cl.sync();
+    float* factor = reinterpret_cast<float*>(sm + pl.factor);         // [kHeads][C]: to the cluster's maximum
+    float* top = factor + kHeads * kMaxCluster;                       // [kHeads] maximum, sum of the cluster
+    if (tid < kHeads * C) {                                           // the C lanes of a head are neighbours, C 8 or 16
+        const int h = tid / C, r = tid - h * C;
+        const float* from = cl.map_shared_rank(stat, r);
+        const float m = h < nh ? from[h] : -1e30f, l = h < nh ? from[kHeads + h] : 0.f;
+        float best = m;
+        for (int x = C / 2; x > 0; x /= 2) best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, x));
+        const float f = exp2f(m - best);
+        float sum = f * l;
+        for (int x = C / 2; x > 0; x /= 2) sum += __shfl_xor_sync(0xffffffffu, sum, x);
+        factor[h * C + r] = active == 1 ? f / sum : f;
+        if (r == 0) {
+            top[h] = best;
+            top[kHeads + h] = sum;
         }
-        l = warp_sum(l);
-        __syncwarp();
-        for (int s = lane; s < active; s += 32) factor[h * active + s] /= l;
     }
     __syncthreads();
-    const float* all = p.part + (size_t)gb * p.splits * kHeads * a.vdim_pad;
-    const int v4 = a.vdim_pad / 4;
-    for (int e = tid; e < nh * v4; e += kThreads) {
-        const int h = e / v4, d = (e - h * v4) * 4;
-        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-        const float* src = all + (size_t)h * a.vdim_pad + d;
-#pragma unroll 8
-        for (int s = 0; s < active; ++s) {
-            const float4 v = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * kHeads * a.vdim_pad));
-            const float f = factor[h * active + s];
-            t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
+    const int v4 = a.vdim_pad / 4, e_lo = nh * v4 * rank / C, e_hi = nh * v4 * (rank + 1) / C;
+    auto finish = [&](int e, float4 t) {
+        const int h = e / v4, d = (e - h * v4) * 4, at = (h0 + h) * a.vdim + d;
+        const float v[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+            if (d + x < a.vdim) p.s.out[at + x] = p.s.gate != nullptr ? v[x] * sigmoid_f32(__ldcg(p.s.gate + at + x)) : v[x];
+    };
+    float* part = p.part + (size_t)gb * p.clusters * kHeads * a.vdim_pad;
+    for (int e = e_lo + tid; e < e_hi; e += kThreads) {
+        const int h = e / v4;
+        float4 v[kMaxCluster], t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int r = 0; r < kMaxCluster; ++r) v[r] = reinterpret_cast<const float4*>(cl.map_shared_rank(s_o, r < C ? r : 0))[e];
+#pragma unroll
+        for (int r = 0; r < kMaxCluster; ++r) {
+            const float f = r < C ? factor[h * C + r] : 0.f;
+            t.x = fmaf(f, v[r].x, t.x); t.y = fmaf(f, v[r].y, t.y); t.z = fmaf(f, v[r].z, t.z); t.w = fmaf(f, v[r].w, t.w);
         }
-        if (d < a.vdim) finish(h, d, t.x);
-        if (d + 1 < a.vdim) finish(h, d + 1, t.y);
-        if (d + 2 < a.vdim) finish(h, d + 2, t.z);
-        if (d + 3 < a.vdim) finish(h, d + 3, t.w);
+        if (active == 1) finish(e, t);
+        else reinterpret_cast<float4*>(part + (size_t)cluster * kHeads * a.vdim_pad)[e] = t;
     }
+    if (active > 1) {
+        float* ml = p.ml + ((size_t)gb * p.clusters * C + rank) * kHeads * 2;
+        const size_t ml_step = (size_t)C * kHeads * 2;
+        if (tid < 2 * kHeads) ml[cluster * ml_step + tid] = top[tid];
+        __threadfence();
+        __syncthreads();
+        unsigned* ticket = p.tickets + gb * C + rank;
+        if (tid == 0) s_last = atomicAdd(ticket, 1u) == (unsigned)active - 1;
+        __syncthreads();
+        if (s_last) {
+            __threadfence();
+            if (tid == 0) *ticket = 0;
+            for (int e = e_lo + tid; e < e_hi; e += kThreads) {
+                const int h = e / v4;
+                float best = -1e30f, l = 0.f;
+                float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+                for (int x = 0; x < active; ++x) best = fmaxf(best, __ldcg(ml + x * ml_step + h));
+#pragma unroll 4
+                for (int x = 0; x < active; ++x) {
+                    const float f = exp2f(__ldcg(ml + x * ml_step + h) - best);
+                    const float4 v = __ldcg(reinterpret_cast<const float4*>(part + (size_t)x * kHeads * a.vdim_pad) + e);
+                    l = fmaf(f, __ldcg(ml + x * ml_step + kHeads + h), l);
+                    t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
+                }
+                finish(e, make_float4(t.x / l, t.y / l, t.z / l, t.w / l));
+            }
+        }
+    }
+    cl.sync();                                            // the other CTAs still read this one's shared memory
 }
 
-struct Grid { int blocks, splits, limit; size_t part, ml, tickets, bytes; };
+struct Grid { int blocks, clusters, limit; size_t part, ml, tickets, bytes; };
 
-// Splits: enough CTAs to fill the device once (twice where two fit an SM), at most one per tile.
+// Clusters of a head block: enough CTAs to fill the device (twice where two fit an SM), at most one per kTilesPerCta
+// tiles of each CTA. Sized for clusters of 8; with 16 half as many are launched.
 template <typename T>
 int plan_grid(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
     constexpr int KT = kTileOf<T>;
@@ -469,16 +505,13 @@ int plan_grid(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
         per_sm = 1;
         if (StepPlan(a, KT, gr.limit).stages < 1) return LEANKV_ELIMIT;
     }
-    const int tiles = (std::min(a.size, max_pos) + KT - 1) / KT;
-    const StepPlan pl(a, KT, gr.limit);
-    const int fit = (pl.stage + pl.stages * pl.stage_bytes) / (kHeads * 4);           // merge factors
-    gr.splits = std::max(1, std::min({tiles, sm_count() * per_sm / (a.kv_heads * gr.blocks), fit}));
-    const size_t groups = (size_t)a.kv_heads * gr.blocks;
+    const int tiles = (std::min(a.size, max_pos) + KT - 1) / KT, groups = a.kv_heads * gr.blocks;
+    gr.clusters = std::max(1, std::min((tiles + 8 * kTilesPerCta - 1) / (8 * kTilesPerCta), sm_count() * per_sm / (8 * groups)));
     const auto take = [&](size_t n) { const size_t at = gr.bytes; gr.bytes += round_up(n, 256); return at; };
     gr.bytes = 0;
-    gr.tickets = take(groups * 4);
-    gr.ml = take(groups * gr.splits * kHeads * 2 * 4);
-    gr.part = take(groups * gr.splits * kHeads * a.vdim_pad * 4);
+    gr.tickets = take((size_t)groups * kMaxCluster * 4);
+    gr.ml = take((size_t)groups * gr.clusters * kMaxCluster * kHeads * 2 * 4);
+    gr.part = take((size_t)groups * gr.clusters * kHeads * a.vdim_pad * 4);
     return LEANKV_OK;
 }
 
@@ -488,11 +521,36 @@ int plan(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
 }
 
 template <typename T, int NP>
-int launch_step(const StepArgs& p, cudaStream_t st) {
+int launch_step(StepArgs p, cudaStream_t st) {
     const size_t smem = StepPlan(p.a, kTileOf<T>, p.limit).total;
-    LEANKV_CUDA_TRY(cudaFuncSetAttribute(causal_step_kernel<T, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    LEANKV_CUDA_TRY(launch_kernel_ex(true, causal_step_kernel<T, NP>, dim3(p.splits, p.a.kv_heads * p.blocks), dim3(kThreads), smem, st, p));
-    return LEANKV_OK;
+    const auto kernel = causal_step_kernel<T, NP>;
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LEANKV_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+    const int groups = p.a.kv_heads * p.blocks;
+    for (const int clusters8 = p.clusters;;) {
+        p.cluster = p.cluster == kMaxCluster ? 8 : kMaxCluster;
+        p.clusters = p.cluster == 8 ? clusters8 : (clusters8 + 1) / 2;
+        const dim3 grid(p.cluster * p.clusters, groups);
+        if (p.cluster > 8) {                             // does a cluster of this size fit this device, often enough?
+            cudaLaunchConfig_t cfg = {};
+            cfg.gridDim = grid;
+            cfg.blockDim = dim3(kThreads);
+            cfg.dynamicSmemBytes = smem;
+            cudaLaunchAttribute attr[1];
+            attr[0].id = cudaLaunchAttributeClusterDimension;
+            attr[0].val.clusterDim.x = p.cluster;
+            attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+            cfg.attrs = attr;
+            cfg.numAttrs = 1;
+            int fits = 0;
+            if (cudaOccupancyMaxActiveClusters(&fits, kernel, &cfg) != cudaSuccess || fits < p.clusters * groups) {
+                (void)cudaGetLastError();
+                continue;
+            }
+        }
+        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(true, dim3(p.cluster), kernel, grid, dim3(kThreads), smem, st, p));
+        return LEANKV_OK;
+    }
 }
 
 }  // namespace
@@ -524,7 +582,7 @@ extern "C" int leankv_causal_step(const leankv_causal_attn_t* a, const leankv_ca
     p.a = *a;
     p.s = *s;
     p.blocks = gr.blocks;
-    p.splits = gr.splits;
+    p.clusters = gr.clusters;
     p.limit = gr.limit;
     char* ws = static_cast<char*>(s->ws);
     p.tickets = reinterpret_cast<unsigned*>(ws + gr.tickets);

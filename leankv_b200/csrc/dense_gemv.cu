@@ -83,12 +83,12 @@ __device__ __forceinline__ float warp_reduce_rows(float (&acc)[R], int lane) {
 template <int R>
 __device__ __forceinline__ int row_of_lane(int lane) { return (lane * R) >> 5; }
 
-// kStaged: the input is prepared once in shared memory (a branch joins it, or a gain per column). kGrouped: row
-// groups with an input slice each.
-enum class Input { kPlain, kStaged, kGrouped };
+// kJoined: a branch joins the stream first, or there is a gain per column; every thread prepares its columns in registers
+// (one slab). kStaged: the same in shared memory, any number of slabs. kGrouped: row groups with an input slice each.
+enum class Input { kPlain, kJoined, kStaged, kGrouped };
 template <typename T, int CH, Input IN>
 __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel(const GemvParams p) {
-    constexpr bool STAGED = IN == Input::kStaged, GROUPED = IN == Input::kGrouped;
+    constexpr bool STAGED = IN == Input::kStaged, JOINED = IN == Input::kJoined, GROUPED = IN == Input::kGrouped;
     constexpr int R = 8 / CH;                        // rows in flight: R * CH 16-byte loads per lane (bf16)
     extern __shared__ __align__(16) float s_dyn[];
     float* s_part = STAGED ? s_dyn + p.x_smem : s_dyn;      // [rows of this CTA (x2 if gated)][warps]
@@ -115,7 +115,58 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
     pdl_begin();
 
     float rs = 1.f;
-    if constexpr (STAGED) {         // the normed input x', after a branch joined x, into shared memory
+    float xj[CH][8];                // kJoined: this thread's columns of x'
+    if constexpr (JOINED) {
+        float d[CH][8];
+        const int k0 = warp * 256 + lane * 8;
+        float sd = 0.f, ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            load_x8(a.x, c * warps * 256 + k0, cols, vec, xj[c]);
+            if (a.delta != nullptr) load_x8(a.delta, c * warps * 256 + k0, cols, vec, d[c]);
+        }
+        if (a.delta != nullptr) {
+#pragma unroll
+            for (int c = 0; c < CH; ++c)
+#pragma unroll
+                for (int i = 0; i < 8; ++i) sd = fmaf(d[c][i], d[c][i], sd);
+            const float f = a.post_mult / sqrtf(cta_sum(sd, s_tmp) / (float)cols + a.eps);
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+                const int k = c * warps * 256 + k0;
+                float g[8];
+                load_x8(a.post_gain, k, cols, vec, g);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) xj[c][i] = fmaf(d[c][i] * f, g[i], xj[c][i]);
+                if (blockIdx.x == 0)
+#pragma unroll
+                    for (int i = 0; i < 8; ++i)
+                        if (k + i < cols) a.x_out[k + i] = xj[c][i];
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ss = fmaf(xj[c][i], xj[c][i], ss);
+        if (a.gain != nullptr) {
+            rs = (a.gain_per_col ? 1.f : __ldg(a.gain)) / sqrtf(cta_sum(ss, s_tmp) / (float)cols + a.eps);
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+                float g[8];
+                if (a.gain_per_col) load_x8(a.gain, c * warps * 256 + k0, cols, vec, g);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) xj[c][i] *= a.gain_per_col ? rs * g[i] : rs;
+            }
+        }
+        if (a.prev != nullptr && blockIdx.x == 0) {
+            float* next = a.prev + (size_t)((a.state[kParity] & 1) ^ 1) * cols;
+#pragma unroll
+            for (int c = 0; c < CH; ++c)
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    if (c * warps * 256 + k0 + i < cols) next[c * warps * 256 + k0 + i] = xj[c][i];
+        }
+    } else if constexpr (STAGED) {         // the normed input x', after a branch joined x, into shared memory
         float f = 0.f, ss = 0.f;
         if (a.delta != nullptr) {
             float sd = 0.f;
@@ -155,7 +206,7 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
         const int par = a.state[kParity] & 1;
         prev = a.prev + (size_t)par * cols;
         float* next = a.prev + (size_t)(par ^ 1) * cols;
-        if (blockIdx.x == 0)
+        if (!JOINED && blockIdx.x == 0)
             for (int k = threadIdx.x; k < cols; k += blockDim.x)
                 next[k] = STAGED ? s_dyn[k] : ld_cg_f32(a.x + k) * rs;
     }
@@ -173,7 +224,10 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
 #pragma unroll
             for (int c = 0; c < CH; ++c) {
                 const int k = s * slab_cols + (c * warps + warp) * 256 + lane * 8;
-                if constexpr (STAGED) {
+                if constexpr (JOINED) {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) xs[c][i] = xj[c][i];
+                } else if constexpr (STAGED) {
                     const bool on = vec && k < cols;
                     const float4 lo4 = on ? *reinterpret_cast<const float4*>(s_dyn + k) : make_float4(0.f, 0.f, 0.f, 0.f);
                     const float4 hi4 = on ? *reinterpret_cast<const float4*>(s_dyn + k + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -288,12 +342,12 @@ extern "C" int leankv_dense_gemv(const leankv_dense_gemv_t* a, void* stream) {
     if (a->group_rows < 0 || (a->group_rows > 0 && (a->rows % a->group_rows || a->group_stride < 0 || a->gain || a->delta ||
                                                     a->n_mix > 0 || a->gated)))
         return LEANKV_EINVAL;
-    if (!aligned16(a->w) || !aligned16(a->x) || (a->gain_per_col && !aligned16(a->gain))) return LEANKV_EALIGN;
+    if (!aligned16(a->w) || !aligned16(a->x) || (a->gain_per_col && !aligned16(a->gain)) ||
+        (a->delta && (!aligned16(a->delta) || !aligned16(a->post_gain)))) return LEANKV_EALIGN;
     GemvParams p{};
     p.a = *a;
     p.vec = a->cols % 8 == 0 && (a->group_rows == 0 || a->group_stride % 4 == 0);
     const bool staged = a->delta || (a->gain && a->gain_per_col);
-    p.x_smem = staged ? (a->cols + 3) / 4 * 4 : 0;
     // warps x slabs x CH column chunks of 256: the widest CTA that pads least
     const int chunks = (a->cols + 255) / 256;
     int warps = 1, per = 1;
@@ -305,6 +359,7 @@ extern "C" int leankv_dense_gemv(const leankv_dense_gemv_t* a, void* stream) {
             if (best < 0 || score < best) { best = score; warps = w; per = ch; }
         }
     p.slabs = (chunks + warps * per - 1) / (warps * per);
+    p.x_smem = staged && p.slabs > 1 ? (a->cols + 3) / 4 * 4 : 0;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     const auto go = [&](auto tag) -> int {
         using T = decltype(tag);
@@ -312,6 +367,7 @@ extern "C" int leankv_dense_gemv(const leankv_dense_gemv_t* a, void* stream) {
             constexpr Input IN = decltype(in)::value;
             return per == 1 ? launch_gemv<T, 1, IN>(p, warps, st) : launch_gemv<T, 2, IN>(p, warps, st);
         };
+        if (staged && p.slabs == 1) return with(std::integral_constant<Input, Input::kJoined>{});
         if (staged) return with(std::integral_constant<Input, Input::kStaged>{});
         if (a->group_rows > 0) return with(std::integral_constant<Input, Input::kGrouped>{});
         return with(std::integral_constant<Input, Input::kPlain>{});

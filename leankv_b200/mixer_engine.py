@@ -354,9 +354,6 @@ class MixerDecodeEngine(DecodeLoop):
 
     # ── kernel status ────────────────────────────────────────────────────
 
-    def _queue_status(self) -> None:
-        self._pinned_status[:1].copy_(self.seq.status, non_blocking=True)
-
     def check_status(self) -> None:
         """Raise if a wait inside an attention kernel ran out (its results are not to be used)."""
         if int(self.seq.status.item()):
@@ -389,7 +386,6 @@ class MixerDecodeEngine(DecodeLoop):
                 self.step()
                 if len(want):
                     out[:] = self.logits
-                    self.check_status()
                 return out
             ids = torch.as_tensor(list(tokens), dtype=torch.int64, device=self.dev)
             for s0 in range(0, n, self.max_chunk):

@@ -418,7 +418,7 @@ class _CausalMixer:
             raise ValueError(f"the decode step does not take these sizes: {self.spec}")
         self._step_ws = torch.zeros(need, dtype=torch.uint8, device=state.device)
         return _native.CausalStep(eps=self.eps, rate=self.rate.data_ptr(), state=state.data_ptr(), max_pos=max_pos,
-                                  ws=self._step_ws.data_ptr(), ws_bytes=need, status=self.seq.status.data_ptr(), **kw)
+                                  ws=self._step_ws.data_ptr(), ws_bytes=need, **kw)
 
     def step(self, st: int) -> int:
         """Launch the step; returns the number of kernels."""
@@ -451,11 +451,11 @@ class RotaryAttention(_CausalMixer):
                                     dim_pad=pad16(s.dim), vdim_pad=pad16(s.vdim), size=self.size, scale=s.scale,
                                     k=st.k.data_ptr(), v=st.v.data_ptr(), k_ring=st.ring, k_rows=st.ring)
 
-    def portion(self, h: torch.Tensor, mixed, start: int, scratch) -> torch.Tensor:
-        s, c, T = self.spec, self.c, h.shape[0]
-        y = matmul(h, self.w_in)
-        q = torch.empty(T, s.heads, c.dim_pad, dtype=h.dtype, device=h.device)
-        src, n = y.data_ptr(), self.in_width
+    def place(self, y: torch.Tensor, start: int) -> torch.Tensor:
+        """Projections [T][q | k | v | ..]: keys and values into the rings; returns the queries."""
+        s, c, T = self.spec, self.c, y.shape[0]
+        q = torch.empty(T, s.heads, c.dim_pad, dtype=self.seq.dtype, device=y.device)
+        src, n = y.data_ptr(), y.stride(0)
         self._place(start, T, [
             dict(src=src, ld=n, heads=s.heads, head_stride=s.dim, n=s.dim, dst=q.data_ptr(), dst_ld=s.heads * c.dim_pad,
                  dst_head_stride=c.dim_pad, n_pad=c.dim_pad, rot=s.rot.dims),
@@ -463,7 +463,11 @@ class RotaryAttention(_CausalMixer):
                  dst_ld=s.kv_heads * c.dim_pad, dst_head_stride=c.dim_pad, n_pad=c.dim_pad, ring=c.k_ring, rot=s.rot.dims),
             dict(src=src + 4 * self.at_v, ld=n, heads=s.kv_heads, head_stride=s.vdim, n=s.vdim, dst=c.v,
                  dst_ld=s.kv_heads * c.vdim_pad, dst_head_stride=c.vdim_pad, n_pad=c.vdim_pad, ring=c.k_ring)])
-        return matmul(self._attend(c, q, y[:, self.at_g:], start), self.w_out)
+        return q
+
+    def portion(self, h: torch.Tensor, mixed, start: int, scratch) -> torch.Tensor:
+        y = matmul(h, self.w_in)
+        return matmul(self._attend(self.c, self.place(y, start), y[:, self.at_g:], start), self.w_out)
 
     def prepare_step(self, entry: dict, exit: dict, bufs: dict, state: torch.Tensor, max_pos: int) -> None:
         """Stream -> y (q | k | v | gate) -> out (gated heads) -> branch output."""
@@ -513,10 +517,36 @@ class LatentAttention(_CausalMixer):
                                     vdim_pad=pad16(s.kv_rank), size=self.size, scale=s.scale, k=st.k.data_ptr(), k_ring=st.ring,
                                     k_rows=st.ring, shared=_native.ptr(st.shared), s_ring=st.ring)
 
+    def place_latents(self, y: torch.Tensor, start: int) -> torch.Tensor:
+        """Projections [T][query latent | latent | key part]: the last two into the rings; returns the normed query latents."""
+        s, c, T = self.spec, self.c, y.shape[0]
+        cq = torch.empty(T, s.q_rank, dtype=self.seq.dtype, device=y.device)
+        src, ld, n, r = y.data_ptr(), y.stride(0), s.kv_rank, s.rot_dim
+        segments = [dict(src=src, ld=ld, heads=1, n=s.q_rank, dst=cq.data_ptr(), dst_ld=s.q_rank, n_pad=s.q_rank,
+                         gain=self.q_norm.data_ptr()),
+                    dict(src=src + 4 * s.q_rank, ld=ld, heads=1, n=n, dst=c.k, dst_ld=c.dim_pad, n_pad=c.dim_pad,
+                         ring=c.k_ring, gain=self.kv_norm.data_ptr())]
+        if r:
+            segments.append(dict(src=src + 4 * (s.q_rank + n), ld=ld, heads=1, n=r, dst=c.shared, dst_ld=c.shared_pad,
+                                 n_pad=c.shared_pad, ring=c.s_ring, rot=s.rot.dims))
+        self._place(start, T, segments)
+        return cq
+
+    def place_q(self, z: torch.Tensor, start: int) -> torch.Tensor:
+        """Queries [T][heads][own | rotated part] as operands, both parts padded."""
+        s, T = self.spec, z.shape[0]
+        H, d, r, dp, rp = s.heads, s.dim, s.rot_dim, pad16(s.dim), pad16(s.rot_dim)
+        q = torch.empty(T, H, dp + rp, dtype=self.seq.dtype, device=z.device)
+        part = lambda off, at, m, pad, rot: dict(src=z.data_ptr() + 4 * off, ld=z.stride(0), heads=H, head_stride=d + r, n=m,
+                                                 dst=q.data_ptr() + q.element_size() * at, dst_ld=H * (dp + rp),
+                                                 dst_head_stride=dp + rp, n_pad=pad, rot=rot)
+        self._place(start, T, [part(0, 0, d, dp, 0)] + ([part(d, dp, r, rp, s.rot.dims)] if r else []))
+        return q
+
     def _expanded(self, start: int, T: int) -> tuple:
-        """Keys and values of the positions that a portion sees, from a multiple of the ring step on: their first
-        position, [n][heads][pad16(dim)], [n][heads][pad16(vdim)]."""
-        s, ring = self.spec, self.state.ring
+        """Per-head keys and values of the positions that a portion sees, from a multiple of the ring step on: the
+        attention over them, and the buffers it reads."""
+        s, c, ring = self.spec, self.c, self.state.ring
         base = max(0, start - self.size + 1) // RING_STEP * RING_STEP
         n = start + T - base
         k = torch.empty(n, s.heads * pad16(s.dim), dtype=self.seq.dtype, device=self.seq.dev)
@@ -525,38 +555,20 @@ class LatentAttention(_CausalMixer):
         while at < n:
             slot = (base + at) % ring
             m = min(n - at, ring - slot)
-            c = self.state.k[slot:slot + m, 0, :s.kv_rank]
-            torch.mm(c, self.w_k.t(), out=k[at:at + m])
-            torch.mm(c, self.w_v.t(), out=v[at:at + m])
+            latents = self.state.k[slot:slot + m, 0, :s.kv_rank]
+            torch.mm(latents, self.w_k.t(), out=k[at:at + m])
+            torch.mm(latents, self.w_v.t(), out=v[at:at + m])
             at += m
-        return base, k, v
+        e = _native.CausalAttn(dtype=c.dtype, heads=s.heads, kv_heads=s.heads, dim=s.dim, shared_dim=s.rot_dim, vdim=s.vdim,
+                               dim_pad=pad16(s.dim), shared_pad=c.shared_pad, vdim_pad=pad16(s.vdim), size=self.size,
+                               scale=s.scale, k=k.data_ptr(), v=v.data_ptr(), k_base=base,
+                               k_ring=(n + RING_STEP - 1) // RING_STEP * RING_STEP, k_rows=n, shared=c.shared, s_ring=c.s_ring)
+        return e, (k, v)
 
     def portion(self, h: torch.Tensor, mixed, start: int, scratch) -> torch.Tensor:
-        s, c, T = self.spec, self.c, h.shape[0]
-        H, d, r, n, dp, rp = s.heads, s.dim, s.rot_dim, s.kv_rank, pad16(s.dim), pad16(s.rot_dim)
-        y = matmul(h, self.w_down)
-        cq = torch.empty(T, s.q_rank, dtype=h.dtype, device=h.device)
-        src, ld = y.data_ptr(), self.in_width
-        segments = [dict(src=src, ld=ld, heads=1, n=s.q_rank, dst=cq.data_ptr(), dst_ld=s.q_rank, n_pad=s.q_rank,
-                         gain=self.q_norm.data_ptr()),
-                    dict(src=src + 4 * s.q_rank, ld=ld, heads=1, n=n, dst=c.k, dst_ld=c.dim_pad, n_pad=c.dim_pad,
-                         ring=c.k_ring, gain=self.kv_norm.data_ptr())]
-        if r:
-            segments.append(dict(src=src + 4 * (s.q_rank + n), ld=ld, heads=1, n=r, dst=c.shared, dst_ld=rp, n_pad=rp,
-                                 ring=c.s_ring, rot=s.rot.dims))
-        self._place(start, T, segments)
-        z = matmul(cq, self.w_q)
-        q = torch.empty(T, H, dp + rp, dtype=h.dtype, device=h.device)
-        part = lambda off, m, pad, rot: dict(src=z.data_ptr() + 4 * off, ld=H * (d + r), heads=H, head_stride=d + r, n=m,
-                                             dst=q.data_ptr() + q.element_size() * (dp if off else 0), dst_ld=H * (dp + rp),
-                                             dst_head_stride=dp + rp, n_pad=pad, rot=rot)
-        self._place(start, T, [part(0, d, dp, 0)] + ([part(d, r, rp, s.rot.dims)] if r else []))
-        base, k, v = self._expanded(start, T)
-        rows = k.shape[0]
-        e = _native.CausalAttn(dtype=c.dtype, heads=H, kv_heads=H, dim=d, shared_dim=r, vdim=s.vdim, dim_pad=dp, shared_pad=rp,
-                               vdim_pad=pad16(s.vdim), size=self.size, scale=s.scale, k=k.data_ptr(), v=v.data_ptr(),
-                               k_base=base, k_ring=(rows + RING_STEP - 1) // RING_STEP * RING_STEP, k_rows=rows,
-                               shared=c.shared, s_ring=c.s_ring)
+        cq = self.place_latents(matmul(h, self.w_down), start)
+        q = self.place_q(matmul(cq, self.w_q), start)
+        e, buffers = self._expanded(start, h.shape[0])
         return matmul(self._attend(e, q, None, start), self.w_out)
 
     def prepare_step(self, entry: dict, exit: dict, bufs: dict, state: torch.Tensor, max_pos: int) -> None:
