@@ -1,11 +1,13 @@
 // One decode step of causal attention over a ring of keys, split over the keys. A CTA takes up to 16 query heads of one
-// kv head and a range of 64-key tiles, which come by asynchronous copies through a few stages; the first are on their
+// kv head and a range of key tiles, which come by asynchronous copies through a few stages; the first are on their
 // way before the launch ahead has finished. The CTAs of a cluster merge their outputs through distributed
 // shared memory, each a slice of the columns. A long sequence takes several clusters per head block: there the
 // last cluster to finish a slice merges the clusters' results, in cluster order.
 //
-// bf16: scores and outputs on tensor cores (16 heads x 8 keys, 16 heads x 8 columns). Queries and softmax weights enter
-// as two bf16 numbers each, so a 32-bit query meets the stored keys exactly. fp32: the same walk on FMA units.
+// Three ways to walk the tiles (Walk): up to 128 value columns, every warp for itself, 16 keys at a time, with scores
+// and weights in registers; more columns, the CTA together on 64 keys, a warp a share of the columns; fp32, the same
+// on FMA units. The first two use tensor cores (16 heads x 8 keys, 16 heads x 8 columns): queries and softmax weights
+// enter as two bf16 numbers each, so a 32-bit query meets the stored keys exactly.
 
 #include <algorithm>
 
@@ -19,16 +21,20 @@ namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr int kWarps = 8;
-constexpr int kThreads = 32 * kWarps;
 constexpr int kHeads = 16;                // query heads of a CTA
 constexpr int kMaxStages = 4;
 constexpr int kMaxCols = 1024;            // value columns
 constexpr int kMaxPairs = 512;            // rotated pairs
 constexpr int kMaxCluster = 16;           // non-portable; 8 where the device does not place 16
-constexpr int kTilesPerCta = 4;           // a further cluster joins when every CTA would have more tiles
+constexpr int kTilesPerUnit = 4;          // a further cluster joins when a warp / CTA would have more tiles
 
-template <typename T> constexpr int kTileOf = sizeof(T) == 2 ? 64 : 32;      // keys of a tile
+enum class Walk { kWarps, kColumns, kFma };
+constexpr int kWarpCols = 128;            // value columns of Walk::kWarps
+__host__ __device__ constexpr int tile_of(Walk w) { return w == Walk::kWarps ? 16 : w == Walk::kColumns ? 64 : 32; }
+__host__ __device__ constexpr int warps_of(Walk w) { return w == Walk::kWarps ? 4 : 8; }           // of a CTA
+__host__ __device__ constexpr int units_of(Walk w) { return w == Walk::kWarps ? 4 : 1; }           // that take tiles, per CTA
+template <Walk W> struct TypeOf { using T = bf16; };
+template <> struct TypeOf<Walk::kFma> { using T = float; };
 
 // Shared-memory plan in bytes. Row lengths are 16 bytes past a multiple of 128, so that the eight rows of a matrix
 // fragment fall into different banks.
@@ -36,34 +42,35 @@ struct StepPlan {
     int k_row, v_row, stages, stage_bytes;             // bytes of a key row (own part, then shared), of a value row
     int q, q_row, s, p, stat, factor, trig, fresh, stage, total;
     __host__ __device__ static constexpr int row(int bytes) { return (bytes + 127) / 128 * 128 + 16; }
-    __host__ __device__ StepPlan(const leankv_causal_attn_t& a, int tile, int limit) {
-        const int es = a.dtype == LEANKV_DT_BF16 ? 2 : 4, kd = a.dim_pad + a.shared_pad;
+    StepPlan() = default;
+    StepPlan(const leankv_causal_attn_t& a, Walk w, int limit) {
+        const int es = a.dtype == LEANKV_DT_BF16 ? 2 : 4, kd = a.dim_pad + a.shared_pad, tile = tile_of(w);
         k_row = row(kd * es);
         v_row = a.v != nullptr ? row(a.vdim_pad * es) : 0;
         int o = 0;
         const auto take = [&](int n) { const int at = o; o += (n + 127) / 128 * 128; return at; };
         q_row = es == 2 ? k_row : kd * 4;
         q = take(kHeads * q_row * (es == 2 ? 2 : 1));   // high parts, then low parts
-        s = take(kHeads * (tile + 4) * 4);
-        p = take(kHeads * row(tile * 2) * 2);
+        s = take(w == Walk::kWarps ? warps_of(w) * kHeads * 8 : kHeads * (tile + 4) * 4);      // scores; maxima and sums of the warps
+        p = take(w == Walk::kColumns ? kHeads * row(tile * 2) * 2 : 0);
         stat = take(kHeads * 4 * 4);                    // maximum, sum, rescale factor
         factor = take(kHeads * kMaxCluster * 4 + kHeads * 8);
         trig = take(kMaxPairs * 8);
         fresh = take(k_row + v_row);
         stage = o;
-        stage_bytes = (tile * (k_row + v_row) + 127) / 128 * 128;
-        stages = (limit - o) / stage_bytes;
-        if (stages > kMaxStages) stages = kMaxStages;
-        const int out = kHeads * a.vdim_pad * 4;        // the outputs take the stages' place
+        stage_bytes = (tile * (k_row + v_row) + 127) / 128 * 128;                          // of a unit
+        stages = std::min((limit - o) / (stage_bytes * units_of(w)), kMaxStages);
+        const int out = kHeads * a.vdim_pad * 4;        // the outputs of a unit take its stages' place
         if (stages * stage_bytes < out) stages = 0;
-        total = o + stages * stage_bytes;
+        total = o + stages * stage_bytes * units_of(w);
     }
 };
 
 struct StepArgs {
     leankv_causal_attn_t a;
     leankv_causal_step_t s;
-    int blocks, cluster, clusters, limit; // head blocks per kv head, CTAs of a cluster, clusters of a head block
+    StepPlan plan;
+    int blocks, cluster, clusters;        // head blocks per kv head, CTAs of a cluster, clusters of a head block
     float* part;                          // [head block][cluster][kHeads][vdim_pad]
     float* ml;                            // [head block][cluster][rank][kHeads][2]
     unsigned* tickets;                    // [head block][rank]
@@ -84,50 +91,76 @@ __device__ __forceinline__ void ldmatrix4_t(uint32_t (&r)[4], uint32_t addr) {
                  : "r"(addr));
 }
 
-// NP: 16-column pieces of the values that a warp accumulates at most (bf16).
-template <typename T, int NP>
-__global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) causal_step_kernel(const __grid_constant__ StepArgs p) {
+// All but the `newer` youngest copy groups of this thread have landed.
+__device__ __forceinline__ void wait_copies(int newer) {
+    switch (newer) {
+        case 0: asm volatile("cp.async.wait_group 0;" ::: "memory"); break;
+        case 1: asm volatile("cp.async.wait_group 1;" ::: "memory"); break;
+        case 2: asm volatile("cp.async.wait_group 2;" ::: "memory"); break;
+        default: asm volatile("cp.async.wait_group 3;" ::: "memory"); break;
+    }
+}
+
+// NP: 16-column pieces of the values that a warp accumulates at most (tensor cores).
+template <Walk W, int NP>
+__global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) causal_step_kernel(const __grid_constant__ StepArgs p) {
+    using T = typename TypeOf<W>::T;
     extern __shared__ __align__(128) unsigned char sm[];
     __shared__ float s_tmp[32];
     __shared__ int s_last;
-    constexpr bool HALF = sizeof(T) == 2;
-    constexpr int KT = kTileOf<T>;
+    constexpr bool HALF = sizeof(T) == 2, WARPS = W == Walk::kWarps;
+    constexpr int KT = tile_of(W), UNITS = units_of(W), kWarps = warps_of(W), kThreads = 32 * kWarps;
     const leankv_causal_attn_t& a = p.a;
-    const StepPlan pl(a, KT, p.limit);
+    const StepPlan& pl = p.plan;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int gb = blockIdx.y, g = gb / p.blocks, hb = gb % p.blocks, rep = a.heads / a.kv_heads;
     const int h0 = g * rep + hb * kHeads, nh = min(kHeads, rep - hb * kHeads);
     const int C = p.cluster, rank = blockIdx.x % C, cluster = blockIdx.x / C;
-    const int i = p.s.state[kPos], lo = first_visible(i, a.size), n = i + 1 - lo, tiles = (n + KT - 1) / KT;
-    const int active = max(1, min(p.clusters, (tiles + C * kTilesPerCta - 1) / (C * kTilesPerCta)));
+    const int i = p.s.state[kPos], lo = first_visible(i, a.size), tiles = (i - lo) / KT + 1;
+    const int active = max(1, min(p.clusters, (tiles + C * UNITS * kTilesPerUnit - 1) / (C * UNITS * kTilesPerUnit)));
     if (cluster >= active) {
         pdl_begin();
         return;
     }
-    const int split = cluster * C + rank, splits = active * C;
-    const int j0 = (int)((long long)tiles * split / splits), j1 = (int)((long long)tiles * (split + 1) / splits);
+    // tiles j0 .. j1 - 1 of this unit; the last unit has the last tile
+    const unsigned unit = (cluster * C + rank) * UNITS + (WARPS ? warp : 0), n_units = active * C * UNITS;
+    const int j0 = (int)((unsigned)tiles * unit / n_units), j1 = (int)((unsigned)tiles * (unit + 1) / n_units);
     const int kd = a.dim_pad + a.shared_pad;
     const T* K = static_cast<const T*>(a.k);
     const T* V = static_cast<const T*>(a.v);
     const T* S = static_cast<const T*>(a.shared);
 
-    // tile j into its stage, a warp a row; the position of this step is not in the ring yet
+    // tile j into its stage (a lane a 16-byte column, the rows in turn); the position of this step is not in the ring yet
     constexpr int E16 = 16 / (int)sizeof(T);
     const int c_own = a.dim_pad / E16, c_key = kd / E16, c_all = c_key + (V != nullptr ? a.vdim_pad / E16 : 0);
+    unsigned char* stage0 = sm + pl.stage + (WARPS ? warp * pl.stages * pl.stage_bytes : 0);
     auto fetch = [&](int j) {
         if (j < j1) {
-            const int st = (j - j0) % pl.stages, first = lo + j * KT, cnt = min(KT, i - first);
-            const uint32_t kb = smem_addr(sm + pl.stage + st * pl.stage_bytes), vb = kb + KT * pl.k_row;
-            const int slot0 = ring_slot(first, a.k_base, a.k_ring), sslot0 = a.shared_dim > 0 ? ring_slot(first, 0, a.s_ring) : 0;
-            for (int r = warp; r < cnt; r += kWarps) {
-                int slot = slot0 + r, sslot = sslot0 + r;           // a window fits into the ring once
-                if (slot >= a.k_ring) slot -= a.k_ring;
-                if (sslot >= a.s_ring) sslot -= a.s_ring;
-                const T* k_src = K + ((size_t)slot * a.kv_heads + g) * a.dim_pad;
-                for (int c = lane; c < c_all; c += 32) {
-                    if (c < c_own) copy16(kb + r * pl.k_row + c * 16, k_src + c * E16);
-                    else if (c < c_key) copy16(kb + r * pl.k_row + c * 16, S + (size_t)sslot * a.shared_pad + (c - c_own) * E16);
-                    else copy16(vb + r * pl.v_row + (c - c_key) * 16, V + ((size_t)slot * a.kv_heads + g) * a.vdim_pad + (c - c_key) * E16);
+            const int first = lo + j * KT, cnt = min(KT, i - first), r0 = WARPS ? 0 : warp;
+            const uint32_t kb = smem_addr(stage0 + (j - j0) % pl.stages * pl.stage_bytes);
+            const int k_slot = ring_slot(first, a.k_base, a.k_ring), s_slot = a.shared_dim > 0 ? ring_slot(first, 0, a.s_ring) : 0;
+            for (int c = lane; c < c_all; c += 32) {
+                const T* src;
+                int step, slot, ring, row;
+                uint32_t dst = kb;
+                if (c < c_own) {
+                    src = K + (size_t)g * a.dim_pad + c * E16;
+                    step = a.kv_heads * a.dim_pad, slot = k_slot, ring = a.k_ring, row = pl.k_row, dst += c * 16;
+                } else if (c < c_key) {
+                    src = S + (c - c_own) * E16;
+                    step = a.shared_pad, slot = s_slot, ring = a.s_ring, row = pl.k_row, dst += c * 16;
+                } else {
+                    src = V + (size_t)g * a.vdim_pad + (c - c_key) * E16;
+                    step = a.kv_heads * a.vdim_pad, slot = k_slot, ring = a.k_ring, row = pl.v_row;
+                    dst += KT * pl.k_row + (c - c_key) * 16;
+                }
+                slot += r0;
+                dst += r0 * row;
+                for (int r = r0; r < cnt; r += WARPS ? 1 : kWarps) {
+                    if (slot >= ring) slot -= ring;       // a window fits into the ring once
+                    copy16(dst, src + (size_t)slot * step);
+                    slot += WARPS ? 1 : kWarps;
+                    dst += (WARPS ? 1 : kWarps) * row;
                 }
             }
         }
@@ -150,31 +183,31 @@ __global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) c
     auto pair_at = [&](const float* x, int d, int dim, int rot) { return turned(pair_of(x, d, dim), d, rot); };
     constexpr int kBatch = 6;                             // loads in flight per thread
     for (int e0 = tid; e0 < kHeads * (kd / 2); e0 += kBatch * kThreads) {
-      float2 in[kBatch];
+        float2 in[kBatch];
 #pragma unroll
-      for (int x = 0; x < kBatch; ++x) {
-        const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
-        in[x] = make_float2(0.f, 0.f);
-        if (h < nh)
-            in[x] = d < a.dim_pad ? pair_of(p.s.q + (size_t)(h0 + h) * p.s.q_stride, d, a.dim)
-                                  : pair_of(p.s.q_shared + (size_t)(h0 + h) * p.s.qs_stride, d - a.dim_pad, a.shared_dim);
-      }
-#pragma unroll
-      for (int x = 0; x < kBatch; ++x) {
-        const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
-        if (h >= kHeads) break;
-        const float2 v = d < a.dim_pad ? turned(in[x], d, p.s.rot_own) : turned(in[x], d - a.dim_pad, p.s.rot_shared);
-        if constexpr (HALF) {
-            uint32_t hi, low;
-            split_bf16(v.x, v.y, hi, low);
-            *reinterpret_cast<uint32_t*>(sm + pl.q + h * pl.q_row + d * 2) = hi;
-            *reinterpret_cast<uint32_t*>(sm + pl.q + (kHeads + h) * pl.q_row + d * 2) = low;
-        } else {
-            *reinterpret_cast<float2*>(sm + pl.q + h * pl.q_row + d * 4) = v;
+        for (int x = 0; x < kBatch; ++x) {
+            const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
+            in[x] = make_float2(0.f, 0.f);
+            if (h < nh)
+                in[x] = d < a.dim_pad ? pair_of(p.s.q + (size_t)(h0 + h) * p.s.q_stride, d, a.dim)
+                                      : pair_of(p.s.q_shared + (size_t)(h0 + h) * p.s.qs_stride, d - a.dim_pad, a.shared_dim);
         }
-      }
+#pragma unroll
+        for (int x = 0; x < kBatch; ++x) {
+            const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
+            if (h >= kHeads) break;
+            const float2 v = d < a.dim_pad ? turned(in[x], d, p.s.rot_own) : turned(in[x], d - a.dim_pad, p.s.rot_shared);
+            if constexpr (HALF) {
+                uint32_t hi, low;
+                split_bf16(v.x, v.y, hi, low);
+                *reinterpret_cast<uint32_t*>(sm + pl.q + h * pl.q_row + d * 2) = hi;
+                *reinterpret_cast<uint32_t*>(sm + pl.q + (kHeads + h) * pl.q_row + d * 2) = low;
+            } else {
+                *reinterpret_cast<float2*>(sm + pl.q + h * pl.q_row + d * 4) = v;
+            }
+        }
     }
-    const bool newest = j0 < j1 && j1 == tiles;                      // this CTA's range ends with the new position
+    const bool newest = rank == C - 1 && cluster == active - 1;      // this CTA's range ends with the new position
     T* fresh = reinterpret_cast<T*>(sm + pl.fresh);
     if (newest) {
         float f = 1.f;
@@ -225,6 +258,17 @@ __global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) c
     __syncthreads();
 
     // ---- the tiles ----
+    // the new row into row cnt - 1 of the last tile, and zeros behind it
+    auto put_new_row = [&](unsigned char* kt, unsigned char* vt, int cnt, int id, int ids) {
+        const int words = (KT - cnt + 1) * (pl.k_row / 4), words_v = V != nullptr ? (KT - cnt + 1) * (pl.v_row / 4) : 0;
+        for (int e = id; e < words; e += ids)
+            reinterpret_cast<uint32_t*>(kt + (cnt - 1) * pl.k_row)[e] =
+                e * 4 < kd * (int)sizeof(T) ? reinterpret_cast<const uint32_t*>(fresh)[e] : 0u;
+        for (int e = id; e < words_v; e += ids)
+            reinterpret_cast<uint32_t*>(vt + (cnt - 1) * pl.v_row)[e] =
+                e * 4 < a.vdim_pad * (int)sizeof(T) ? reinterpret_cast<const uint32_t*>(sm + pl.fresh + pl.k_row)[e] : 0u;
+    };
+    const int v_row = V != nullptr ? pl.v_row : pl.k_row;
     float* s_s = reinterpret_cast<float*>(sm + pl.s);
     constexpr int SLD = KT + 4;
     constexpr int kColsOfThread = kMaxCols / kThreads;              // columns of a thread (fp32)
@@ -242,133 +286,271 @@ __global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) c
 #pragma unroll
             for (int h = 0; h < kHeads; ++h) of[x][h] = 0.f;
     }
-    for (int j = j0; j < j1; ++j) {
-        const int st = (j - j0) % pl.stages, first = lo + j * KT, cnt = min(KT, i + 1 - first);
-        unsigned char* kt = sm + pl.stage + st * pl.stage_bytes;
-        unsigned char* vt = V != nullptr ? kt + KT * pl.k_row : kt;
-        const int v_row = V != nullptr ? pl.v_row : pl.k_row;
-        switch (pl.stages) {                              // all but the newer groups have landed
-            case 1: asm volatile("cp.async.wait_group 0;" ::: "memory"); break;
-            case 2: asm volatile("cp.async.wait_group 1;" ::: "memory"); break;
-            case 3: asm volatile("cp.async.wait_group 2;" ::: "memory"); break;
-            default: asm volatile("cp.async.wait_group 3;" ::: "memory"); break;
-        }
-        if (j == tiles - 1) {                             // the new row, and zeros behind it
-            const int words = (KT - cnt + 1) * (pl.k_row / 4), words_v = V != nullptr ? (KT - cnt + 1) * (pl.v_row / 4) : 0;
-            for (int e = tid; e < words; e += kThreads)
-                reinterpret_cast<uint32_t*>(kt + (cnt - 1) * pl.k_row)[e] =
-                    e < pl.k_row / 4 && e * 4 < kd * (int)sizeof(T) ? reinterpret_cast<const uint32_t*>(fresh)[e] : 0u;
-            for (int e = tid; e < words_v; e += kThreads)
-                reinterpret_cast<uint32_t*>(vt + (cnt - 1) * pl.v_row)[e] =
-                    e < pl.v_row / 4 && e * 4 < a.vdim_pad * (int)sizeof(T)
-                        ? reinterpret_cast<const uint32_t*>(sm + pl.fresh + pl.k_row)[e]
-                        : 0u;
-        }
-        __syncthreads();
-        // scores
-        if constexpr (HALF) {
-            float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
+    if constexpr (WARPS) {
+        float m[2] = {-1e30f, -1e30f}, l[2] = {0.f, 0.f};           // of heads lane / 4 and lane / 4 + 8
+        for (int j = j0; j < j1; ++j) {
+            const int cnt = min(KT, i + 1 - lo - j * KT);
+            unsigned char* kt = stage0 + (j - j0) % pl.stages * pl.stage_bytes;
+            unsigned char* vt = V != nullptr ? kt + KT * pl.k_row : kt;
+            wait_copies(pl.stages - 1);
+            if (j == tiles - 1) put_new_row(kt, vt, cnt, lane, 32);
+            __syncwarp();
+            float hi[2][4] = {}, low[2][4] = {};                    // keys 0-7, 8-15
             const uint32_t qa = smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
-            const uint32_t ka = smem_addr(kt) + (warp * 8 + (lane & 7)) * pl.k_row + (lane >> 3) * 16;
-            for (int d = 0; d < kd; d += 32) {
+            const uint32_t ka = smem_addr(kt) + ((lane & 7) + (lane >> 4) * 8) * pl.k_row + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+            for (int d = 0; d < kd; d += 16) {
                 uint32_t b[4], qh[4], ql[4];
-                const bool two = d + 16 < kd;             // the last block may hold 16 dimensions
-                ldmatrix4(b, ka + (two || lane < 16 ? d * 2 : d * 2 - 32));
+                ldmatrix4(b, ka + d * 2);
                 ldmatrix4(qh, qa + d * 2);
                 ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2);
-                mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[0], b[1]);
-                mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[0], b[1]);
-                if (two) {
-                    ldmatrix4(qh, qa + d * 2 + 32);
-                    ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2 + 32);
-                    mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[2], b[3]);
-                    mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[2], b[3]);
+                mma_bf16(hi[0], qh[0], qh[1], qh[2], qh[3], b[0], b[1]);
+                mma_bf16(hi[1], qh[0], qh[1], qh[2], qh[3], b[2], b[3]);
+                mma_bf16(low[0], ql[0], ql[1], ql[2], ql[3], b[0], b[1]);
+                mma_bf16(low[1], ql[0], ql[1], ql[2], ql[3], b[2], b[3]);
+            }
+            float best[2] = {m[0], m[1]}, f[2];
+#pragma unroll
+            for (int y = 0; y < 2; ++y)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    const int k = y * 8 + (lane & 3) * 2 + (x & 1);
+                    hi[y][x] = k < cnt ? (hi[y][x] + low[y][x]) * c : -INFINITY;
+                    best[x >> 1] = fmaxf(best[x >> 1], hi[y][x]);
                 }
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                best[x] = fmaxf(best[x], __shfl_xor_sync(0xffffffffu, best[x], 1));
+                best[x] = fmaxf(best[x], __shfl_xor_sync(0xffffffffu, best[x], 2));
+                f[x] = exp2f(m[x] - best[x]);
+                m[x] = best[x];
+                l[x] *= f[x];
             }
 #pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                const int h = (lane >> 2) + (x < 2 ? 0 : 8), k = warp * 8 + (lane & 3) * 2 + (x & 1);
-                s_s[h * SLD + k] = k < cnt ? (acc[x] + acc2[x]) * c : -INFINITY;
-            }
-        } else {
-            for (int k = warp; k < KT; k += kWarps) {
-                const float* row = reinterpret_cast<const float*>(kt + k * pl.k_row);
-                for (int h = 0; h < nh; ++h) {
-                    const float* q = reinterpret_cast<const float*>(sm + pl.q + h * pl.q_row);
-                    float t = 0.f;
-                    if (k < cnt)
-                        for (int d = lane; d < kd; d += 32) t = fmaf(q[d], row[d], t);
-                    t = warp_sum(t);
-                    if (lane == 0) s_s[h * SLD + k] = k < cnt ? t * c : -INFINITY;
+            for (int y = 0; y < 2; ++y)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    hi[y][x] = exp2f(hi[y][x] - m[x >> 1]);
+                    l[x >> 1] += hi[y][x];
                 }
-            }
-        }
-        __syncthreads();
-        // softmax: a warp two heads
+            uint32_t wh[4], wl[4];                                  // the weights as an operand: 16 heads x 16 keys
 #pragma unroll
-        for (int x = 0; x < kHeads / kWarps; ++x) {
-            const int h = warp * (kHeads / kWarps) + x;
-            if (h >= nh) continue;
-            float v[KT / 32], best = stat[h], l = 0.f;
+            for (int y = 0; y < 2; ++y)
 #pragma unroll
-            for (int y = 0; y < KT / 32; ++y) {
-                v[y] = s_s[h * SLD + lane * (KT / 32) + y];
-                best = fmaxf(best, v[y]);
-            }
-            best = warp_max(best);
-            const float f = exp2f(stat[h] - best);
+                for (int x = 0; x < 2; ++x) split_bf16(hi[y][2 * x], hi[y][2 * x + 1], wh[2 * y + x], wl[2 * y + x]);
+            const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + (lane >> 4) * 16;
 #pragma unroll
-            for (int y = 0; y < KT / 32; ++y) {
-                v[y] = exp2f(v[y] - best);
-                l += v[y];
-            }
-            l = warp_sum(l);
-            if constexpr (HALF) {
-                uint32_t hi, low;
-                split_bf16(v[0], v[KT / 32 - 1], hi, low);
-                *reinterpret_cast<uint32_t*>(sm + pl.p + h * StepPlan::row(KT * 2) + lane * 4) = hi;
-                *reinterpret_cast<uint32_t*>(sm + pl.p + (kHeads + h) * StepPlan::row(KT * 2) + lane * 4) = low;
-            } else {
-                s_s[h * SLD + lane] = v[0];
+            for (int x = 0; x < NP; ++x) {
+                if (x * 16 >= a.vdim_pad) break;
+                uint32_t b[4];                            // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
+                ldmatrix4_t(b, va + x * 32);
+#pragma unroll
+                for (int y = 0; y < 2; ++y) {
+#pragma unroll
+                    for (int z = 0; z < 4; ++z) o[x][y][z] *= f[z >> 1];
+                    mma_bf16(o[x][y], wh[0], wh[1], wh[2], wh[3], b[2 * y], b[2 * y + 1]);
+                    mma_bf16(o[x][y], wl[0], wl[1], wl[2], wl[3], b[2 * y], b[2 * y + 1]);
+                }
             }
             __syncwarp();
-            if (lane == 0) {
-                stat[h] = best;
-                stat[kHeads + h] = stat[kHeads + h] * f + l;
-                stat[2 * kHeads + h] = f;
+            fetch(j + pl.stages);                         // this stage is free again
+        }
+        wait_copies(0);
+        // the warps' outputs, to the CTA's maximum, summed in the first warp's place
+        float* s_m = s_s;                                 // [warp][maximum, sum][kHeads]
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            l[x] += __shfl_xor_sync(0xffffffffu, l[x], 1);
+            l[x] += __shfl_xor_sync(0xffffffffu, l[x], 2);
+            if ((lane & 3) == 0) {
+                s_m[warp * 2 * kHeads + (lane >> 2) + 8 * x] = m[x];
+                s_m[(warp * 2 + 1) * kHeads + (lane >> 2) + 8 * x] = l[x];
             }
         }
         __syncthreads();
-        // outputs
-        if constexpr (HALF) {
-            constexpr int PROW = StepPlan::row(KT * 2);
-            const float f0 = stat[2 * kHeads + (lane >> 2)], f1 = stat[2 * kHeads + (lane >> 2) + 8];
-            const uint32_t pa = smem_addr(sm + pl.p) + (lane & 15) * PROW + (lane >> 4) * 16;
-            uint32_t wh[KT / 16][4], wl[KT / 16][4];
+        float f[2], best[2] = {-1e30f, -1e30f}, sum[2] = {0.f, 0.f};
 #pragma unroll
-            for (int k = 0; k < KT / 16; ++k) {
-                ldmatrix4(wh[k], pa + k * 32);
-                ldmatrix4(wl[k], pa + kHeads * PROW + k * 32);
+        for (int x = 0; x < 2; ++x) {
+            const float* at = s_m + (lane >> 2) + 8 * x;
+#pragma unroll
+            for (int w = 0; w < kWarps; ++w) best[x] = fmaxf(best[x], at[w * 2 * kHeads]);
+#pragma unroll
+            for (int w = 0; w < kWarps; ++w) sum[x] = fmaf(exp2f(at[w * 2 * kHeads] - best[x]), at[(w * 2 + 1) * kHeads], sum[x]);
+            f[x] = exp2f(m[x] - best[x]);
+            if (warp == 0 && (lane & 3) == 0) {
+                stat[(lane >> 2) + 8 * x] = best[x];
+                stat[kHeads + (lane >> 2) + 8 * x] = sum[x];
             }
+        }
+        float* mine = reinterpret_cast<float*>(stage0);
+#pragma unroll
+        for (int x = 0; x < NP; ++x) {
+            if (x * 16 >= a.vdim_pad) break;
+#pragma unroll
+            for (int y = 0; y < 2; ++y)
+#pragma unroll
+                for (int z = 0; z < 2; ++z)
+                    *reinterpret_cast<float2*>(mine + ((lane >> 2) + z * 8) * a.vdim_pad + x * 16 + y * 8 + (lane & 3) * 2) =
+                        make_float2(o[x][y][2 * z] * f[z], o[x][y][2 * z + 1] * f[z]);
+        }
+        __syncthreads();
+        const int next = pl.stages * pl.stage_bytes / 16;
+        float4* sum4 = reinterpret_cast<float4*>(sm + pl.stage);
+        for (int e = tid; e < nh * a.vdim_pad / 4; e += kThreads) {
+            float4 t = sum4[e];
+#pragma unroll
+            for (int w = 1; w < kWarps; ++w) {
+                const float4 v = sum4[e + w * next];
+                t.x += v.x; t.y += v.y; t.z += v.z; t.w += v.w;
+            }
+            sum4[e] = t;
+        }
+    } else {
+        for (int j = j0; j < j1; ++j) {
+            const int cnt = min(KT, i + 1 - lo - j * KT);
+            unsigned char* kt = stage0 + (j - j0) % pl.stages * pl.stage_bytes;
+            unsigned char* vt = V != nullptr ? kt + KT * pl.k_row : kt;
+            wait_copies(pl.stages - 1);
+            if (j == tiles - 1) put_new_row(kt, vt, cnt, tid, kThreads);
+            __syncthreads();
+            // scores
+            if constexpr (HALF) {
+                float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
+                const uint32_t qa = smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
+                const uint32_t ka = smem_addr(kt) + (warp * 8 + (lane & 7)) * pl.k_row + (lane >> 3) * 16;
+                for (int d = 0; d < kd; d += 32) {
+                    uint32_t b[4], qh[4], ql[4];
+                    const bool two = d + 16 < kd;             // the last block may hold 16 dimensions
+                    ldmatrix4(b, ka + (two || lane < 16 ? d * 2 : d * 2 - 32));
+                    ldmatrix4(qh, qa + d * 2);
+                    ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2);
+                    mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[0], b[1]);
+                    mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[0], b[1]);
+                    if (two) {
+                        ldmatrix4(qh, qa + d * 2 + 32);
+                        ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2 + 32);
+                        mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[2], b[3]);
+                        mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[2], b[3]);
+                    }
+                }
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    const int h = (lane >> 2) + (x < 2 ? 0 : 8), k = warp * 8 + (lane & 3) * 2 + (x & 1);
+                    s_s[h * SLD + k] = k < cnt ? (acc[x] + acc2[x]) * c : -INFINITY;
+                }
+            } else {
+                for (int k = warp; k < KT; k += kWarps) {
+                    const float* row = reinterpret_cast<const float*>(kt + k * pl.k_row);
+                    for (int h = 0; h < nh; ++h) {
+                        const float* q = reinterpret_cast<const float*>(sm + pl.q + h * pl.q_row);
+                        float t = 0.f;
+                        if (k < cnt)
+                            for (int d = lane; d < kd; d += 32) t = fmaf(q[d], row[d], t);
+                        t = warp_sum(t);
+                        if (lane == 0) s_s[h * SLD + k] = k < cnt ? t * c : -INFINITY;
+                    }
+                }
+            }
+            __syncthreads();
+            // softmax: a warp two heads
+#pragma unroll
+            for (int x = 0; x < kHeads / kWarps; ++x) {
+                const int h = warp * (kHeads / kWarps) + x;
+                if (h >= nh) continue;
+                float v[KT / 32], best = stat[h], l = 0.f;
+#pragma unroll
+                for (int y = 0; y < KT / 32; ++y) {
+                    v[y] = s_s[h * SLD + lane * (KT / 32) + y];
+                    best = fmaxf(best, v[y]);
+                }
+                best = warp_max(best);
+                const float f = exp2f(stat[h] - best);
+#pragma unroll
+                for (int y = 0; y < KT / 32; ++y) {
+                    v[y] = exp2f(v[y] - best);
+                    l += v[y];
+                }
+                l = warp_sum(l);
+                if constexpr (HALF) {
+                    uint32_t hi, low;
+                    split_bf16(v[0], v[KT / 32 - 1], hi, low);
+                    *reinterpret_cast<uint32_t*>(sm + pl.p + h * StepPlan::row(KT * 2) + lane * 4) = hi;
+                    *reinterpret_cast<uint32_t*>(sm + pl.p + (kHeads + h) * StepPlan::row(KT * 2) + lane * 4) = low;
+                } else {
+                    s_s[h * SLD + lane] = v[0];
+                }
+                __syncwarp();
+                if (lane == 0) {
+                    stat[h] = best;
+                    stat[kHeads + h] = stat[kHeads + h] * f + l;
+                    stat[2 * kHeads + h] = f;
+                }
+            }
+            __syncthreads();
+            // outputs
+            if constexpr (HALF) {
+                constexpr int PROW = StepPlan::row(KT * 2);
+                const float f0 = stat[2 * kHeads + (lane >> 2)], f1 = stat[2 * kHeads + (lane >> 2) + 8];
+                const uint32_t pa = smem_addr(sm + pl.p) + (lane & 15) * PROW + (lane >> 4) * 16;
+                uint32_t wh[KT / 16][4], wl[KT / 16][4];
+#pragma unroll
+                for (int k = 0; k < KT / 16; ++k) {
+                    ldmatrix4(wh[k], pa + k * 32);
+                    ldmatrix4(wl[k], pa + kHeads * PROW + k * 32);
+                }
+#pragma unroll
+                for (int x = 0; x < NP; ++x) {
+                    const int col = (warp + x * kWarps) * 16;
+                    if (col >= a.vdim_pad) break;
+#pragma unroll
+                    for (int y = 0; y < 2; ++y) {
+                        o[x][y][0] *= f0; o[x][y][1] *= f0;
+                        o[x][y][2] *= f1; o[x][y][3] *= f1;
+                    }
+                    const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + col * 2 + (lane >> 4) * 16;
+#pragma unroll
+                    for (int k = 0; k < KT / 16; ++k) {
+                        uint32_t b[4];                        // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
+                        ldmatrix4_t(b, va + k * 16 * v_row);
+                        mma_bf16(o[x][0], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[0], b[1]);
+                        mma_bf16(o[x][1], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[2], b[3]);
+                        mma_bf16(o[x][0], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[0], b[1]);
+                        mma_bf16(o[x][1], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[2], b[3]);
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int x = 0; x < kColsOfThread; ++x) {
+                    const int d = tid + x * kThreads;
+                    if (d >= a.vdim_pad) break;
+#pragma unroll
+                    for (int h = 0; h < kHeads; ++h)
+                        if (h < nh) of[x][h] *= stat[2 * kHeads + h];
+                    for (int k = 0; k < cnt; ++k) {
+                        const float v = reinterpret_cast<const float*>(vt + k * v_row)[d];
+#pragma unroll
+                        for (int h = 0; h < kHeads; ++h)
+                            if (h < nh) of[x][h] = fmaf(s_s[h * SLD + k], v, of[x][h]);
+                    }
+                }
+            }
+            __syncthreads();
+            fetch(j + pl.stages);                             // this stage is free again
+        }
+        wait_copies(0);
+        float* s_o = reinterpret_cast<float*>(sm + pl.stage);
+        auto put = [&](int h, int d, float v) { s_o[h * a.vdim_pad + d] = v; };
+        if constexpr (HALF) {
 #pragma unroll
             for (int x = 0; x < NP; ++x) {
                 const int col = (warp + x * kWarps) * 16;
                 if (col >= a.vdim_pad) break;
 #pragma unroll
-                for (int y = 0; y < 2; ++y) {
-                    o[x][y][0] *= f0; o[x][y][1] *= f0;
-                    o[x][y][2] *= f1; o[x][y][3] *= f1;
-                }
-                const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + col * 2 + (lane >> 4) * 16;
+                for (int y = 0; y < 2; ++y)
 #pragma unroll
-                for (int k = 0; k < KT / 16; ++k) {
-                    uint32_t b[4];                        // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
-                    ldmatrix4_t(b, va + k * 16 * v_row);
-                    mma_bf16(o[x][0], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[0], b[1]);
-                    mma_bf16(o[x][1], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[2], b[3]);
-                    mma_bf16(o[x][0], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[0], b[1]);
-                    mma_bf16(o[x][1], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[2], b[3]);
-                }
+                    for (int z = 0; z < 2; ++z)
+                        *reinterpret_cast<float2*>(s_o + ((lane >> 2) + z * 8) * a.vdim_pad + col + y * 8 + (lane & 3) * 2) =
+                            make_float2(o[x][y][2 * z], o[x][y][2 * z + 1]);
             }
         } else {
 #pragma unroll
@@ -376,51 +558,19 @@ __global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) c
                 const int d = tid + x * kThreads;
                 if (d >= a.vdim_pad) break;
 #pragma unroll
-                for (int h = 0; h < kHeads; ++h)
-                    if (h < nh) of[x][h] *= stat[2 * kHeads + h];
-                for (int k = 0; k < cnt; ++k) {
-                    const float v = reinterpret_cast<const float*>(vt + k * v_row)[d];
-#pragma unroll
-                    for (int h = 0; h < kHeads; ++h)
-                        if (h < nh) of[x][h] = fmaf(s_s[h * SLD + k], v, of[x][h]);
-                }
+                for (int h = 0; h < kHeads; ++h) put(h, d, of[x][h]);
             }
         }
-        __syncthreads();
-        fetch(j + pl.stages);                             // this stage is free again
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
 
-    // ---- merge: this CTA's outputs into shared memory, then a slice of the columns of all CTAs of the cluster ----
+    // ---- merge: every CTA of the cluster has its outputs in shared memory and takes a slice of the columns ----
     float* s_o = reinterpret_cast<float*>(sm + pl.stage);             // [kHeads][vdim_pad]
-    auto put = [&](int h, int d, float v) { s_o[h * a.vdim_pad + d] = v; };
-    if constexpr (HALF) {
-#pragma unroll
-        for (int x = 0; x < NP; ++x) {
-            const int col = (warp + x * kWarps) * 16;
-            if (col >= a.vdim_pad) break;
-#pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int z = 0; z < 2; ++z)
-                    *reinterpret_cast<float2*>(s_o + ((lane >> 2) + z * 8) * a.vdim_pad + col + y * 8 + (lane & 3) * 2) =
-                        make_float2(o[x][y][2 * z], o[x][y][2 * z + 1]);
-        }
-    } else {
-#pragma unroll
-        for (int x = 0; x < kColsOfThread; ++x) {
-            const int d = tid + x * kThreads;
-            if (d >= a.vdim_pad) break;
-#pragma unroll
-            for (int h = 0; h < kHeads; ++h) put(h, d, of[x][h]);
-        }
-    }
     auto cl = cg::this_cluster();
     cl.sync();
     float* factor = reinterpret_cast<float*>(sm + pl.factor);         // [kHeads][C]: to the cluster's maximum
     float* top = factor + kHeads * kMaxCluster;                       // [kHeads] maximum, sum of the cluster
-    if (tid < kHeads * C) {                                           // the C lanes of a head are neighbours, C 8 or 16
-        const int h = tid / C, r = tid - h * C;
+    for (int e = tid; e < kHeads * C; e += kThreads) {                // the C lanes of a head are neighbours, C 8 or 16
+        const int h = e / C, r = e - h * C;
         const float* from = cl.map_shared_rank(stat, r);
         const float m = h < nh ? from[h] : -1e30f, l = h < nh ? from[kHeads + h] : 0.f;
         float best = m;
@@ -489,24 +639,31 @@ __global__ void __launch_bounds__(kThreads, sizeof(T) == 2 && NP <= 1 ? 2 : 1) c
     cl.sync();                                            // the other CTAs still read this one's shared memory
 }
 
-struct Grid { int blocks, clusters, limit; size_t part, ml, tickets, bytes; };
+struct Grid {
+    Walk walk;
+    StepPlan plan;
+    int blocks, clusters;
+    size_t part, ml, tickets, bytes;
+};
 
-// Clusters of a head block: enough CTAs to fill the device (twice where two fit an SM), at most one per kTilesPerCta
-// tiles of each CTA. Sized for clusters of 8; with 16 half as many are launched.
-template <typename T>
+// Clusters of a head block: enough CTAs to fill the device, at most one per kTilesPerUnit tiles of each unit. Sized for
+// clusters of 8; with 16 half as many are launched.
 int plan_grid(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
-    constexpr int KT = kTileOf<T>;
-    const int rep = a.heads / a.kv_heads;
-    gr.blocks = (rep + kHeads - 1) / kHeads;
-    gr.limit = 112 * 1024;                               // two CTAs per SM
-    int per_sm = 2;
-    if (StepPlan(a, KT, gr.limit).stages < 2) {
-        gr.limit = 226 * 1024;
+    if (a.vdim_pad > kMaxCols) return LEANKV_ELIMIT;
+    int limit = 112 * 1024, per_sm = 2;                  // two CTAs per SM for warps on their own
+    gr.walk = a.dtype != LEANKV_DT_BF16 ? Walk::kFma : a.vdim_pad <= kWarpCols ? Walk::kWarps : Walk::kColumns;
+    gr.plan = StepPlan(a, gr.walk, limit);
+    if (gr.walk == Walk::kWarps && gr.plan.stages < 1) gr.walk = Walk::kColumns;
+    if (gr.walk != Walk::kWarps) {
         per_sm = 1;
-        if (StepPlan(a, KT, gr.limit).stages < 1) return LEANKV_ELIMIT;
+        limit = 226 * 1024;
+        gr.plan = StepPlan(a, gr.walk, limit);
     }
-    const int tiles = (std::min(a.size, max_pos) + KT - 1) / KT, groups = a.kv_heads * gr.blocks;
-    gr.clusters = std::max(1, std::min((tiles + 8 * kTilesPerCta - 1) / (8 * kTilesPerCta), sm_count() * per_sm / (8 * groups)));
+    if (gr.plan.stages < 1) return LEANKV_ELIMIT;
+    gr.blocks = (a.heads / a.kv_heads + kHeads - 1) / kHeads;
+    const int keys = std::min(a.size, max_pos), per = 8 * units_of(gr.walk) * kTilesPerUnit * tile_of(gr.walk);
+    const int groups = a.kv_heads * gr.blocks;
+    gr.clusters = std::max(1, std::min((keys + per - 1) / per, sm_count() * per_sm / (8 * groups)));
     const auto take = [&](size_t n) { const size_t at = gr.bytes; gr.bytes += round_up(n, 256); return at; };
     gr.bytes = 0;
     gr.tickets = take((size_t)groups * kMaxCluster * 4);
@@ -515,15 +672,11 @@ int plan_grid(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
     return LEANKV_OK;
 }
 
-int plan(const leankv_causal_attn_t& a, int max_pos, Grid& gr) {
-    if (a.vdim_pad > kMaxCols) return LEANKV_ELIMIT;
-    return a.dtype == LEANKV_DT_BF16 ? plan_grid<bf16>(a, max_pos, gr) : plan_grid<float>(a, max_pos, gr);
-}
-
-template <typename T, int NP>
+template <Walk W, int NP>
 int launch_step(StepArgs p, cudaStream_t st) {
-    const size_t smem = StepPlan(p.a, kTileOf<T>, p.limit).total;
-    const auto kernel = causal_step_kernel<T, NP>;
+    const size_t smem = p.plan.total;
+    const dim3 block(32 * warps_of(W));
+    const auto kernel = causal_step_kernel<W, NP>;
     LEANKV_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     LEANKV_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
     const int groups = p.a.kv_heads * p.blocks;
@@ -534,7 +687,7 @@ int launch_step(StepArgs p, cudaStream_t st) {
         if (p.cluster > 8) {                             // does a cluster of this size fit this device, often enough?
             cudaLaunchConfig_t cfg = {};
             cfg.gridDim = grid;
-            cfg.blockDim = dim3(kThreads);
+            cfg.blockDim = block;
             cfg.dynamicSmemBytes = smem;
             cudaLaunchAttribute attr[1];
             attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -548,7 +701,7 @@ int launch_step(StepArgs p, cudaStream_t st) {
                 continue;
             }
         }
-        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(true, dim3(p.cluster), kernel, grid, dim3(kThreads), smem, st, p));
+        LEANKV_CUDA_TRY(launch_cluster_kernel_ex(true, dim3(p.cluster), kernel, grid, block, smem, st, p));
         return LEANKV_OK;
     }
 }
@@ -560,7 +713,7 @@ using namespace leankv;
 
 extern "C" size_t leankv_causal_step_workspace_bytes(const leankv_causal_attn_t* a, int max_pos) {
     Grid gr;
-    return check_causal(a) || max_pos <= 0 || plan(*a, max_pos, gr) ? 0 : gr.bytes;
+    return check_causal(a) || max_pos <= 0 || plan_grid(*a, max_pos, gr) ? 0 : gr.bytes;
 }
 
 extern "C" int leankv_causal_step(const leankv_causal_attn_t* a, const leankv_causal_step_t* s, void* stream) {
@@ -575,7 +728,7 @@ extern "C" int leankv_causal_step(const leankv_causal_attn_t* a, const leankv_ca
     const int keys = std::min(a->size, s->max_pos);
     if (keys > a->k_ring || (a->shared_dim > 0 && keys > a->s_ring) || a->k_rows < a->k_ring) return LEANKV_ELIMIT;
     Grid gr;
-    rc = plan(*a, s->max_pos, gr);
+    rc = plan_grid(*a, s->max_pos, gr);
     if (rc) return rc;
     if (!s->ws || s->ws_bytes < gr.bytes) return LEANKV_EWORKSPACE;
     StepArgs p{};
@@ -583,13 +736,18 @@ extern "C" int leankv_causal_step(const leankv_causal_attn_t* a, const leankv_ca
     p.s = *s;
     p.blocks = gr.blocks;
     p.clusters = gr.clusters;
-    p.limit = gr.limit;
+    p.plan = gr.plan;
     char* ws = static_cast<char*>(s->ws);
     p.tickets = reinterpret_cast<unsigned*>(ws + gr.tickets);
     p.ml = reinterpret_cast<float*>(ws + gr.ml);
     p.part = reinterpret_cast<float*>(ws + gr.part);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    if (a->dtype == LEANKV_DT_F32) return launch_step<float, 1>(p, st);
-    if (a->vdim_pad <= 16 * kWarps) return launch_step<bf16, 1>(p, st);
-    return a->vdim_pad <= 4 * 16 * kWarps ? launch_step<bf16, 4>(p, st) : launch_step<bf16, kMaxCols / 16 / kWarps>(p, st);
+    switch (gr.walk) {
+        case Walk::kFma: return launch_step<Walk::kFma, 1>(p, st);
+        case Walk::kWarps: return a->vdim_pad <= 64 ? launch_step<Walk::kWarps, 4>(p, st) : launch_step<Walk::kWarps, 8>(p, st);
+        default: break;
+    }
+    if (a->vdim_pad <= 128) return launch_step<Walk::kColumns, 1>(p, st);
+    return a->vdim_pad <= 512 ? launch_step<Walk::kColumns, 4>(p, st)
+                                          : launch_step<Walk::kColumns, kMaxCols / 128>(p, st);
 }
