@@ -1,12 +1,13 @@
-// One decode step of causal attention over a ring of keys, split over the keys. A CTA takes up to 16 query heads of one
+// One decode step of causal attention over a ring of keys, split over the keys. A CTA takes up to 8 query heads of one
 // kv head and a range of key tiles, which come by asynchronous copies through a few stages; the first are on their
-// way before the launch ahead has finished. The CTAs of a cluster merge their outputs through distributed
-// shared memory, each a slice of the columns. A long sequence takes several clusters per head block: there the
-// last cluster to finish a slice merges the clusters' results, in cluster order.
+// way before the launch ahead has finished. Every CTA of a cluster owns a slice of the outputs and merges it: the
+// others write their share of it into its shared memory, one cluster barrier later everything is there. A long
+// sequence takes several clusters per head block: there the last cluster to finish a slice merges the clusters'
+// results, in cluster order.
 //
 // Three ways to walk the tiles (Walk): up to 128 value columns, every warp for itself, 16 keys at a time, with scores
 // and weights in registers; more columns, the CTA together on 64 keys, a warp a share of the columns; fp32, the same
-// on FMA units. The first two use tensor cores (16 heads x 8 keys, 16 heads x 8 columns): queries and softmax weights
+// on FMA units. The first two use tensor cores (16 keys x 8 heads, 16 columns x 8 heads): queries and softmax weights
 // enter as two bf16 numbers each, so a 32-bit query meets the stored keys exactly.
 
 #include <algorithm>
@@ -21,7 +22,7 @@ namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr int kHeads = 16;                // query heads of a CTA
+constexpr int kHeads = 8;                 // query heads of a CTA
 constexpr int kMaxStages = 4;
 constexpr int kMaxCols = 1024;            // value columns
 constexpr int kMaxPairs = 512;            // rotated pairs
@@ -40,7 +41,7 @@ template <> struct TypeOf<Walk::kFma> { using T = float; };
 // fragment fall into different banks.
 struct StepPlan {
     int k_row, v_row, stages, stage_bytes;             // bytes of a key row (own part, then shared), of a value row
-    int q, q_row, s, p, stat, factor, trig, fresh, stage, total;
+    int q, q_row, s, p, stat, trig, fresh, inbox, stage, total;
     __host__ __device__ static constexpr int row(int bytes) { return (bytes + 127) / 128 * 128 + 16; }
     StepPlan() = default;
     StepPlan(const leankv_causal_attn_t& a, Walk w, int limit) {
@@ -51,10 +52,12 @@ struct StepPlan {
         const auto take = [&](int n) { const int at = o; o += (n + 127) / 128 * 128; return at; };
         q_row = es == 2 ? k_row : kd * 4;
         q = take(kHeads * q_row * (es == 2 ? 2 : 1));   // high parts, then low parts
-        s = take(w == Walk::kWarps ? warps_of(w) * kHeads * 8 : kHeads * (tile + 4) * 4);      // scores; maxima and sums of the warps
+        s = take(w == Walk::kWarps ? warps_of(w) * kHeads * 8 : 2 * kHeads * (tile + 4) * 4);      // scores; maxima and sums of the warps
         p = take(w == Walk::kColumns ? kHeads * row(tile * 2) * 2 : 0);
         stat = take(kHeads * 4 * 4);                    // maximum, sum, rescale factor
-        factor = take(kHeads * kMaxCluster * 4 + kHeads * 8);
+        // from every CTA of the cluster: maxima and sums, its share of this CTA's slice of the outputs; merge factors
+        inbox = take((kMaxCluster * 3 + 2) * kHeads * 4 +
+                     (std::min(kHeads, a.heads / a.kv_heads) * (a.vdim_pad / 4) + kMaxCluster) * 16);
         trig = take(kMaxPairs * 8);
         fresh = take(k_row + v_row);
         stage = o;
@@ -99,6 +102,32 @@ __device__ __forceinline__ void wait_copies(int newer) {
         case 2: asm volatile("cp.async.wait_group 2;" ::: "memory"); break;
         default: asm volatile("cp.async.wait_group 3;" ::: "memory"); break;
     }
+}
+
+// Scores of 16 keys (rows at k, k_row bytes apart) with 8 heads (rows at q: high parts, then low parts), dimensions d0 ..
+// d1: s[0], s[1] key lane / 4 with heads 2 (lane % 4) and the next one, s[2], s[3] key lane / 4 + 8.
+__device__ __forceinline__ void tile_scores(float (&s)[4], uint32_t k, uint32_t q, int k_row, int d0, int d1) {
+    const int lane = threadIdx.x & 31;
+    float low[4] = {0.f, 0.f, 0.f, 0.f};
+    s[0] = s[1] = s[2] = s[3] = 0.f;
+    const uint32_t ka = k + (lane & 15) * k_row + (lane >> 4) * 16;
+    const uint32_t qa = q + ((lane & 7) + (lane >> 4) * kHeads) * k_row + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+    for (int d = d0; d < d1; d += 16) {
+        uint32_t x[4], y[4];
+        ldmatrix4(x, ka + d * 2);
+        ldmatrix4(y, qa + d * 2);
+        mma_bf16(s, x[0], x[1], x[2], x[3], y[0], y[1]);
+        mma_bf16(low, x[0], x[1], x[2], x[3], y[2], y[3]);
+    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x) s[x] += low[x];
+}
+// An 8 x 8 matrix of 16-bit numbers, two per lane, transposed.
+__device__ __forceinline__ uint32_t transpose8(uint32_t x) {
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
 }
 
 // NP: 16-column pieces of the values that a warp accumulates at most (tensor cores).
@@ -167,6 +196,7 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (int x = 0; x < pl.stages; ++x) fetch(j0 + x);
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // this CTA runs: its inbox may be written
     float* s_sin = reinterpret_cast<float*>(sm + pl.trig);
     float* s_cos = s_sin + kMaxPairs;
     for (int x = tid; x < max(p.s.rot_own, p.s.rot_shared) / 2; x += kThreads)
@@ -181,9 +211,9 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
     };
     auto turned = [&](float2 v, int d, int rot) { return d < rot ? turn(v.x, v.y, s_sin[d >> 1], s_cos[d >> 1]) : v; };
     auto pair_at = [&](const float* x, int d, int dim, int rot) { return turned(pair_of(x, d, dim), d, rot); };
-    constexpr int kBatch = 6;                             // loads in flight per thread
-    for (int e0 = tid; e0 < kHeads * (kd / 2); e0 += kBatch * kThreads) {
-        float2 in[kBatch];
+    constexpr int kBatch = 5;                             // loads in flight per thread
+    float2 in[kBatch];
+    auto load_queries = [&](int e0) {
 #pragma unroll
         for (int x = 0; x < kBatch; ++x) {
             const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
@@ -192,6 +222,8 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
                 in[x] = d < a.dim_pad ? pair_of(p.s.q + (size_t)(h0 + h) * p.s.q_stride, d, a.dim)
                                       : pair_of(p.s.q_shared + (size_t)(h0 + h) * p.s.qs_stride, d - a.dim_pad, a.shared_dim);
         }
+    };
+    auto put_queries = [&](int e0) {
 #pragma unroll
         for (int x = 0; x < kBatch; ++x) {
             const int e = e0 + x * kThreads, h = e / (kd / 2), d = (e - h * (kd / 2)) * 2;
@@ -206,6 +238,23 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
                 *reinterpret_cast<float2*>(sm + pl.q + h * pl.q_row + d * 4) = v;
             }
         }
+    };
+    load_queries(tid);
+    // this CTA's slice of the outputs, and its gate
+    const int v4 = a.vdim_pad / 4, slice = (nh * v4 + C - 1) / C, mine = rank * slice + tid;      // float4s
+    const int n_mine = min(slice, nh * v4 - rank * slice);
+    auto place_of = [&](int e, int& at) {                 // of float4 e: first element, elements that exist
+        const int h = e / v4, d = (e - h * v4) * 4;
+        at = (h0 + h) * a.vdim + d;
+        return min(4, a.vdim - d);
+    };
+    float gate[4] = {1.f, 1.f, 1.f, 1.f};
+    if (p.s.gate != nullptr && tid < n_mine) {
+        int at;
+        const int cnt = place_of(mine, at);
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+            if (x < cnt) gate[x] = __ldcg(p.s.gate + at + x);
     }
     const bool newest = rank == C - 1 && cluster == active - 1;      // this CTA's range ends with the new position
     T* fresh = reinterpret_cast<T*>(sm + pl.fresh);
@@ -250,6 +299,11 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             }
         }
     }
+    put_queries(tid);
+    for (int e0 = tid + kBatch * kThreads; e0 < kHeads * (kd / 2); e0 += kBatch * kThreads) {
+        load_queries(e0);
+        put_queries(e0);
+    }
     float* stat = reinterpret_cast<float*>(sm + pl.stat);
     if (tid < kHeads) {
         stat[tid] = -1e30f;
@@ -272,14 +326,12 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
     float* s_s = reinterpret_cast<float*>(sm + pl.s);
     constexpr int SLD = KT + 4;
     constexpr int kColsOfThread = kMaxCols / kThreads;              // columns of a thread (fp32)
-    float o[HALF ? NP : 1][2][4], of[HALF ? 1 : kColsOfThread][kHeads];
+    float o[HALF ? NP : 1][4], of[HALF ? 1 : kColsOfThread][kHeads];
     if constexpr (HALF) {
 #pragma unroll
         for (int x = 0; x < NP; ++x)
 #pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int z = 0; z < 4; ++z) o[x][y][z] = 0.f;
+            for (int z = 0; z < 4; ++z) o[x][z] = 0.f;
     } else {
 #pragma unroll
         for (int x = 0; x < kColsOfThread; ++x)
@@ -287,7 +339,8 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             for (int h = 0; h < kHeads; ++h) of[x][h] = 0.f;
     }
     if constexpr (WARPS) {
-        float m[2] = {-1e30f, -1e30f}, l[2] = {0.f, 0.f};           // of heads lane / 4 and lane / 4 + 8
+        // a lane: keys lane / 4 and lane / 4 + 8, heads 2 (lane % 4) and the next one
+        float m[2] = {-1e30f, -1e30f}, l[2] = {0.f, 0.f};
         for (int j = j0; j < j1; ++j) {
             const int cnt = min(KT, i + 1 - lo - j * KT);
             unsigned char* kt = stage0 + (j - j0) % pl.stages * pl.stage_bytes;
@@ -295,115 +348,78 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             wait_copies(pl.stages - 1);
             if (j == tiles - 1) put_new_row(kt, vt, cnt, lane, 32);
             __syncwarp();
-            float hi[2][4] = {}, low[2][4] = {};                    // keys 0-7, 8-15
-            const uint32_t qa = smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
-            const uint32_t ka = smem_addr(kt) + ((lane & 7) + (lane >> 4) * 8) * pl.k_row + ((lane >> 3) & 1) * 16;
-#pragma unroll 4
-            for (int d = 0; d < kd; d += 16) {
-                uint32_t b[4], qh[4], ql[4];
-                ldmatrix4(b, ka + d * 2);
-                ldmatrix4(qh, qa + d * 2);
-                ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2);
-                mma_bf16(hi[0], qh[0], qh[1], qh[2], qh[3], b[0], b[1]);
-                mma_bf16(hi[1], qh[0], qh[1], qh[2], qh[3], b[2], b[3]);
-                mma_bf16(low[0], ql[0], ql[1], ql[2], ql[3], b[0], b[1]);
-                mma_bf16(low[1], ql[0], ql[1], ql[2], ql[3], b[2], b[3]);
-            }
-            float best[2] = {m[0], m[1]}, f[2];
+            float sc[4];
+            tile_scores(sc, smem_addr(kt), smem_addr(sm + pl.q), pl.k_row, 0, kd);
+            float f[2];
 #pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    const int k = y * 8 + (lane & 3) * 2 + (x & 1);
-                    hi[y][x] = k < cnt ? (hi[y][x] + low[y][x]) * c : -INFINITY;
-                    best[x >> 1] = fmaxf(best[x >> 1], hi[y][x]);
-                }
+            for (int x = 0; x < 4; ++x) sc[x] = (lane >> 2) + (x < 2 ? 0 : 8) < cnt ? sc[x] * c : -INFINITY;
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
-                best[x] = fmaxf(best[x], __shfl_xor_sync(0xffffffffu, best[x], 1));
-                best[x] = fmaxf(best[x], __shfl_xor_sync(0xffffffffu, best[x], 2));
-                f[x] = exp2f(m[x] - best[x]);
-                m[x] = best[x];
-                l[x] *= f[x];
+                float best = fmaxf(m[x], fmaxf(sc[x], sc[x + 2]));
+#pragma unroll
+                for (int y = 4; y < 32; y *= 2) best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, y));
+                f[x] = exp2f(m[x] - best);
+                m[x] = best;
+                sc[x] = exp2f(sc[x] - best);
+                sc[x + 2] = exp2f(sc[x + 2] - best);
+                l[x] = l[x] * f[x] + sc[x] + sc[x + 2];
             }
+            uint32_t wh[2], wl[2];                                  // the weights as an operand: 16 keys x 8 heads
 #pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    hi[y][x] = exp2f(hi[y][x] - m[x >> 1]);
-                    l[x >> 1] += hi[y][x];
-                }
-            uint32_t wh[4], wl[4];                                  // the weights as an operand: 16 heads x 16 keys
-#pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int x = 0; x < 2; ++x) split_bf16(hi[y][2 * x], hi[y][2 * x + 1], wh[2 * y + x], wl[2 * y + x]);
-            const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + (lane >> 4) * 16;
+            for (int y = 0; y < 2; ++y) {
+                split_bf16(sc[2 * y], sc[2 * y + 1], wh[y], wl[y]);
+                wh[y] = transpose8(wh[y]);
+                wl[y] = transpose8(wl[y]);
+            }
+            const uint32_t va = smem_addr(vt) + ((lane & 7) + (lane >> 4) * 8) * v_row + ((lane >> 3) & 1) * 16;
 #pragma unroll
             for (int x = 0; x < NP; ++x) {
                 if (x * 16 >= a.vdim_pad) break;
-                uint32_t b[4];                            // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
+                uint32_t b[4];                            // columns 0-7, 8-15 of keys 0-7, then of keys 8-15
                 ldmatrix4_t(b, va + x * 32);
 #pragma unroll
-                for (int y = 0; y < 2; ++y) {
-#pragma unroll
-                    for (int z = 0; z < 4; ++z) o[x][y][z] *= f[z >> 1];
-                    mma_bf16(o[x][y], wh[0], wh[1], wh[2], wh[3], b[2 * y], b[2 * y + 1]);
-                    mma_bf16(o[x][y], wl[0], wl[1], wl[2], wl[3], b[2 * y], b[2 * y + 1]);
-                }
+                for (int z = 0; z < 4; ++z) o[x][z] *= f[z & 1];
+                mma_bf16(o[x], b[0], b[1], b[2], b[3], wh[0], wh[1]);
+                mma_bf16(o[x], b[0], b[1], b[2], b[3], wl[0], wl[1]);
             }
             __syncwarp();
             fetch(j + pl.stages);                         // this stage is free again
         }
         wait_copies(0);
-        // the warps' outputs, to the CTA's maximum, summed in the first warp's place
+        // the warps' outputs, to the CTA's maximum
         float* s_m = s_s;                                 // [warp][maximum, sum][kHeads]
+        const int hl = (lane & 3) * 2;
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
-            l[x] += __shfl_xor_sync(0xffffffffu, l[x], 1);
-            l[x] += __shfl_xor_sync(0xffffffffu, l[x], 2);
-            if ((lane & 3) == 0) {
-                s_m[warp * 2 * kHeads + (lane >> 2) + 8 * x] = m[x];
-                s_m[(warp * 2 + 1) * kHeads + (lane >> 2) + 8 * x] = l[x];
+#pragma unroll
+            for (int y = 4; y < 32; y *= 2) l[x] += __shfl_xor_sync(0xffffffffu, l[x], y);
+            if (lane < 4) {
+                s_m[warp * 2 * kHeads + hl + x] = m[x];
+                s_m[(warp * 2 + 1) * kHeads + hl + x] = l[x];
             }
         }
         __syncthreads();
-        float f[2], best[2] = {-1e30f, -1e30f}, sum[2] = {0.f, 0.f};
+        float* own = reinterpret_cast<float*>(stage0);
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
-            const float* at = s_m + (lane >> 2) + 8 * x;
+            const float* at = s_m + hl + x;
+            float best = -1e30f, sum = 0.f;
 #pragma unroll
-            for (int w = 0; w < kWarps; ++w) best[x] = fmaxf(best[x], at[w * 2 * kHeads]);
+            for (int w = 0; w < kWarps; ++w) best = fmaxf(best, at[w * 2 * kHeads]);
 #pragma unroll
-            for (int w = 0; w < kWarps; ++w) sum[x] = fmaf(exp2f(at[w * 2 * kHeads] - best[x]), at[(w * 2 + 1) * kHeads], sum[x]);
-            f[x] = exp2f(m[x] - best[x]);
-            if (warp == 0 && (lane & 3) == 0) {
-                stat[(lane >> 2) + 8 * x] = best[x];
-                stat[kHeads + (lane >> 2) + 8 * x] = sum[x];
+            for (int w = 0; w < kWarps; ++w) sum = fmaf(exp2f(at[w * 2 * kHeads] - best), at[(w * 2 + 1) * kHeads], sum);
+            const float f = exp2f(m[x] - best);
+            if (warp == 0 && lane < 4) {
+                stat[hl + x] = best;
+                stat[kHeads + hl + x] = sum;
             }
-        }
-        float* mine = reinterpret_cast<float*>(stage0);
 #pragma unroll
-        for (int x = 0; x < NP; ++x) {
-            if (x * 16 >= a.vdim_pad) break;
-#pragma unroll
-            for (int y = 0; y < 2; ++y)
-#pragma unroll
-                for (int z = 0; z < 2; ++z)
-                    *reinterpret_cast<float2*>(mine + ((lane >> 2) + z * 8) * a.vdim_pad + x * 16 + y * 8 + (lane & 3) * 2) =
-                        make_float2(o[x][y][2 * z] * f[z], o[x][y][2 * z + 1] * f[z]);
-        }
-        __syncthreads();
-        const int next = pl.stages * pl.stage_bytes / 16;
-        float4* sum4 = reinterpret_cast<float4*>(sm + pl.stage);
-        for (int e = tid; e < nh * a.vdim_pad / 4; e += kThreads) {
-            float4 t = sum4[e];
-#pragma unroll
-            for (int w = 1; w < kWarps; ++w) {
-                const float4 v = sum4[e + w * next];
-                t.x += v.x; t.y += v.y; t.z += v.z; t.w += v.w;
+            for (int y = 0; y < NP; ++y) {
+                if (y * 16 >= a.vdim_pad) break;
+                float* to = own + (hl + x) * a.vdim_pad + y * 16 + (lane >> 2);
+                to[0] = o[y][x] * f;
+                to[8] = o[y][x + 2] * f;
             }
-            sum4[e] = t;
         }
     } else {
         for (int j = j0; j < j1; ++j) {
@@ -414,29 +430,14 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             if (j == tiles - 1) put_new_row(kt, vt, cnt, tid, kThreads);
             __syncthreads();
             // scores
-            if constexpr (HALF) {
-                float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
-                const uint32_t qa = smem_addr(sm + pl.q) + (lane & 15) * pl.q_row + (lane >> 4) * 16;
-                const uint32_t ka = smem_addr(kt) + (warp * 8 + (lane & 7)) * pl.k_row + (lane >> 3) * 16;
-                for (int d = 0; d < kd; d += 32) {
-                    uint32_t b[4], qh[4], ql[4];
-                    const bool two = d + 16 < kd;             // the last block may hold 16 dimensions
-                    ldmatrix4(b, ka + (two || lane < 16 ? d * 2 : d * 2 - 32));
-                    ldmatrix4(qh, qa + d * 2);
-                    ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2);
-                    mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[0], b[1]);
-                    mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[0], b[1]);
-                    if (two) {
-                        ldmatrix4(qh, qa + d * 2 + 32);
-                        ldmatrix4(ql, qa + kHeads * pl.q_row + d * 2 + 32);
-                        mma_bf16(acc, qh[0], qh[1], qh[2], qh[3], b[2], b[3]);
-                        mma_bf16(acc2, ql[0], ql[1], ql[2], ql[3], b[2], b[3]);
-                    }
-                }
+            if constexpr (HALF) {                         // a warp 16 keys and half of the dimensions
+                const int half = (kd / 16 + 1) / 2 * 16, part = warp / (KT / 16), k0 = warp % (KT / 16) * 16;
+                float sc[4];
+                tile_scores(sc, smem_addr(kt) + k0 * pl.k_row, smem_addr(sm + pl.q), pl.k_row, part * half, part ? kd : half);
 #pragma unroll
                 for (int x = 0; x < 4; ++x) {
-                    const int h = (lane >> 2) + (x < 2 ? 0 : 8), k = warp * 8 + (lane & 3) * 2 + (x & 1);
-                    s_s[h * SLD + k] = k < cnt ? (acc[x] + acc2[x]) * c : -INFINITY;
+                    const int h = (lane & 3) * 2 + (x & 1), k = k0 + (lane >> 2) + (x < 2 ? 0 : 8);
+                    s_s[(part * kHeads + h) * SLD + k] = k < cnt ? sc[x] * c : -INFINITY;
                 }
             } else {
                 for (int k = warp; k < KT; k += kWarps) {
@@ -460,7 +461,7 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
                 float v[KT / 32], best = stat[h], l = 0.f;
 #pragma unroll
                 for (int y = 0; y < KT / 32; ++y) {
-                    v[y] = s_s[h * SLD + lane * (KT / 32) + y];
+                    v[y] = s_s[h * SLD + lane * (KT / 32) + y] + (HALF ? s_s[(kHeads + h) * SLD + lane * (KT / 32) + y] : 0.f);
                     best = fmaxf(best, v[y]);
                 }
                 best = warp_max(best);
@@ -490,32 +491,24 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             // outputs
             if constexpr (HALF) {
                 constexpr int PROW = StepPlan::row(KT * 2);
-                const float f0 = stat[2 * kHeads + (lane >> 2)], f1 = stat[2 * kHeads + (lane >> 2) + 8];
-                const uint32_t pa = smem_addr(sm + pl.p) + (lane & 15) * PROW + (lane >> 4) * 16;
-                uint32_t wh[KT / 16][4], wl[KT / 16][4];
+                const float f0 = stat[2 * kHeads + (lane & 3) * 2], f1 = stat[2 * kHeads + (lane & 3) * 2 + 1];
+                uint32_t w[KT / 16][4];                   // 16 keys x 8 heads: high parts, low parts
+                const uint32_t pa = smem_addr(sm + pl.p) + ((lane & 7) + (lane >> 4) * kHeads) * PROW + ((lane >> 3) & 1) * 16;
 #pragma unroll
-                for (int k = 0; k < KT / 16; ++k) {
-                    ldmatrix4(wh[k], pa + k * 32);
-                    ldmatrix4(wl[k], pa + kHeads * PROW + k * 32);
-                }
+                for (int k = 0; k < KT / 16; ++k) ldmatrix4(w[k], pa + k * 32);
+                const uint32_t va = smem_addr(vt) + ((lane & 7) + (lane >> 4) * 8) * v_row + ((lane >> 3) & 1) * 16;
 #pragma unroll
                 for (int x = 0; x < NP; ++x) {
                     const int col = (warp + x * kWarps) * 16;
                     if (col >= a.vdim_pad) break;
-#pragma unroll
-                    for (int y = 0; y < 2; ++y) {
-                        o[x][y][0] *= f0; o[x][y][1] *= f0;
-                        o[x][y][2] *= f1; o[x][y][3] *= f1;
-                    }
-                    const uint32_t va = smem_addr(vt) + (lane & 15) * v_row + col * 2 + (lane >> 4) * 16;
+                    o[x][0] *= f0; o[x][1] *= f1;
+                    o[x][2] *= f0; o[x][3] *= f1;
 #pragma unroll
                     for (int k = 0; k < KT / 16; ++k) {
-                        uint32_t b[4];                        // keys 0-7, 8-15 of columns 0-7, then of columns 8-15
-                        ldmatrix4_t(b, va + k * 16 * v_row);
-                        mma_bf16(o[x][0], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[0], b[1]);
-                        mma_bf16(o[x][1], wh[k][0], wh[k][1], wh[k][2], wh[k][3], b[2], b[3]);
-                        mma_bf16(o[x][0], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[0], b[1]);
-                        mma_bf16(o[x][1], wl[k][0], wl[k][1], wl[k][2], wl[k][3], b[2], b[3]);
+                        uint32_t b[4];                    // columns 0-7, 8-15 of keys 0-7, then of keys 8-15
+                        ldmatrix4_t(b, va + k * 16 * v_row + col * 2);
+                        mma_bf16(o[x], b[0], b[1], b[2], b[3], w[k][0], w[k][1]);
+                        mma_bf16(o[x], b[0], b[1], b[2], b[3], w[k][2], w[k][3]);
                     }
                 }
             } else {
@@ -538,7 +531,7 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
             fetch(j + pl.stages);                             // this stage is free again
         }
         wait_copies(0);
-        float* s_o = reinterpret_cast<float*>(sm + pl.stage);
+        float* s_o = reinterpret_cast<float*>(sm + pl.stage);                  // [kHeads][vdim_pad]
         auto put = [&](int h, int d, float v) { s_o[h * a.vdim_pad + d] = v; };
         if constexpr (HALF) {
 #pragma unroll
@@ -546,11 +539,7 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
                 const int col = (warp + x * kWarps) * 16;
                 if (col >= a.vdim_pad) break;
 #pragma unroll
-                for (int y = 0; y < 2; ++y)
-#pragma unroll
-                    for (int z = 0; z < 2; ++z)
-                        *reinterpret_cast<float2*>(s_o + ((lane >> 2) + z * 8) * a.vdim_pad + col + y * 8 + (lane & 3) * 2) =
-                            make_float2(o[x][y][2 * z], o[x][y][2 * z + 1]);
+                for (int z = 0; z < 4; ++z) put((lane & 3) * 2 + (z & 1), col + (lane >> 2) + (z < 2 ? 0 : 8), o[x][z]);
             }
         } else {
 #pragma unroll
@@ -563,16 +552,37 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
         }
     }
 
-    // ---- merge: every CTA of the cluster has its outputs in shared memory and takes a slice of the columns ----
-    float* s_o = reinterpret_cast<float*>(sm + pl.stage);             // [kHeads][vdim_pad]
+    // ---- merge: every CTA's outputs to the owners of their slices ----
+    float* box_ml = reinterpret_cast<float*>(sm + pl.inbox);          // [rank][maximum, sum][kHeads]
+    float* factor = box_ml + kMaxCluster * 2 * kHeads;                // [kHeads][C]
+    float* top = factor + kMaxCluster * kHeads;                       // [maximum, sum][kHeads] of the cluster
+    float4* box = reinterpret_cast<float4*>(top + 2 * kHeads);        // [rank][slice]
     auto cl = cg::this_cluster();
-    cl.sync();
-    float* factor = reinterpret_cast<float*>(sm + pl.factor);         // [kHeads][C]: to the cluster's maximum
-    float* top = factor + kHeads * kMaxCluster;                       // [kHeads] maximum, sum of the cluster
+    __syncthreads();
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    for (int e = tid; e < C * 2 * kHeads; e += kThreads) {
+        const int r = e / (2 * kHeads), x = e - r * 2 * kHeads;
+        cl.map_shared_rank(box_ml, r)[rank * 2 * kHeads + x] = stat[x];
+    }
+    {
+        const float4* from = reinterpret_cast<const float4*>(sm + pl.stage);
+        const int next = pl.stages * pl.stage_bytes / 16;
+        for (int e = tid; e < nh * v4; e += kThreads) {
+            float4 t = from[e];
+#pragma unroll
+            for (int w = 1; w < UNITS; ++w) {                         // the warps' sums
+                const float4 v = from[e + w * next];
+                t.x += v.x; t.y += v.y; t.z += v.z; t.w += v.w;
+            }
+            const int r = e / slice;
+            cl.map_shared_rank(box, r)[rank * slice + e - r * slice] = t;
+        }
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
     for (int e = tid; e < kHeads * C; e += kThreads) {                // the C lanes of a head are neighbours, C 8 or 16
         const int h = e / C, r = e - h * C;
-        const float* from = cl.map_shared_rank(stat, r);
-        const float m = h < nh ? from[h] : -1e30f, l = h < nh ? from[kHeads + h] : 0.f;
+        const float m = h < nh ? box_ml[r * 2 * kHeads + h] : -1e30f, l = h < nh ? box_ml[(r * 2 + 1) * kHeads + h] : 0.f;
         float best = m;
         for (int x = C / 2; x > 0; x /= 2) best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, x));
         const float f = exp2f(m - best);
@@ -585,58 +595,58 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
         }
     }
     __syncthreads();
-    const int v4 = a.vdim_pad / 4, e_lo = nh * v4 * rank / C, e_hi = nh * v4 * (rank + 1) / C;
-    auto finish = [&](int e, float4 t) {
-        const int h = e / v4, d = (e - h * v4) * 4, at = (h0 + h) * a.vdim + d;
+    auto finish = [&](int k, float4 t) {                              // float4 k of the slice
+        int at;
+        const int cnt = place_of(rank * slice + k, at);
         const float v[4] = {t.x, t.y, t.z, t.w};
 #pragma unroll
         for (int x = 0; x < 4; ++x)
-            if (d + x < a.vdim) p.s.out[at + x] = p.s.gate != nullptr ? v[x] * sigmoid_f32(__ldcg(p.s.gate + at + x)) : v[x];
-    };
-    float* part = p.part + (size_t)gb * p.clusters * kHeads * a.vdim_pad;
-    for (int e = e_lo + tid; e < e_hi; e += kThreads) {
-        const int h = e / v4;
-        float4 v[kMaxCluster], t = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int r = 0; r < kMaxCluster; ++r) v[r] = reinterpret_cast<const float4*>(cl.map_shared_rank(s_o, r < C ? r : 0))[e];
-#pragma unroll
-        for (int r = 0; r < kMaxCluster; ++r) {
-            const float f = r < C ? factor[h * C + r] : 0.f;
-            t.x = fmaf(f, v[r].x, t.x); t.y = fmaf(f, v[r].y, t.y); t.z = fmaf(f, v[r].z, t.z); t.w = fmaf(f, v[r].w, t.w);
-        }
-        if (active == 1) finish(e, t);
-        else reinterpret_cast<float4*>(part + (size_t)cluster * kHeads * a.vdim_pad)[e] = t;
-    }
-    if (active > 1) {
-        float* ml = p.ml + ((size_t)gb * p.clusters * C + rank) * kHeads * 2;
-        const size_t ml_step = (size_t)C * kHeads * 2;
-        if (tid < 2 * kHeads) ml[cluster * ml_step + tid] = top[tid];
-        __threadfence();
-        __syncthreads();
-        unsigned* ticket = p.tickets + gb * C + rank;
-        if (tid == 0) s_last = atomicAdd(ticket, 1u) == (unsigned)active - 1;
-        __syncthreads();
-        if (s_last) {
-            __threadfence();
-            if (tid == 0) *ticket = 0;
-            for (int e = e_lo + tid; e < e_hi; e += kThreads) {
-                const int h = e / v4;
-                float best = -1e30f, l = 0.f;
-                float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-                for (int x = 0; x < active; ++x) best = fmaxf(best, __ldcg(ml + x * ml_step + h));
-#pragma unroll 4
-                for (int x = 0; x < active; ++x) {
-                    const float f = exp2f(__ldcg(ml + x * ml_step + h) - best);
-                    const float4 v = __ldcg(reinterpret_cast<const float4*>(part + (size_t)x * kHeads * a.vdim_pad) + e);
-                    l = fmaf(f, __ldcg(ml + x * ml_step + kHeads + h), l);
-                    t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
-                }
-                finish(e, make_float4(t.x / l, t.y / l, t.z / l, t.w / l));
+            if (x < cnt) {
+                float g = 1.f;
+                if (p.s.gate != nullptr) g = sigmoid_f32(k == tid ? gate[x] : __ldcg(p.s.gate + at + x));
+                p.s.out[at + x] = v[x] * g;
             }
+    };
+    float4* part = reinterpret_cast<float4*>(p.part) + (size_t)gb * p.clusters * kHeads * v4 + rank * slice;
+    for (int k = tid; k < n_mine; k += kThreads) {
+        const int h = (rank * slice + k) / v4;
+        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int r = 0; r < C; ++r) {
+            const float f = factor[h * C + r];
+            const float4 v = box[r * slice + k];
+            t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
         }
+        if (active == 1) finish(k, t);
+        else part[(size_t)cluster * kHeads * v4 + k] = t;
     }
-    cl.sync();                                            // the other CTAs still read this one's shared memory
+    if (active == 1) return;
+    float* ml = p.ml + ((size_t)gb * p.clusters * C + rank) * kHeads * 2;
+    const size_t ml_step = (size_t)C * kHeads * 2;
+    if (tid < 2 * kHeads) ml[cluster * ml_step + tid] = top[tid];
+    __threadfence();
+    __syncthreads();
+    unsigned* ticket = p.tickets + gb * C + rank;
+    if (tid == 0) s_last = atomicAdd(ticket, 1u) == (unsigned)active - 1;
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    if (tid == 0) *ticket = 0;
+    for (int k = tid; k < n_mine; k += kThreads) {
+        const int h = (rank * slice + k) / v4;
+        float best = -1e30f, l = 0.f;
+        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int x = 0; x < active; ++x) best = fmaxf(best, __ldcg(ml + x * ml_step + h));
+#pragma unroll 4
+        for (int x = 0; x < active; ++x) {
+            const float f = exp2f(__ldcg(ml + x * ml_step + h) - best);
+            const float4 v = __ldcg(part + (size_t)x * kHeads * v4 + k);
+            l = fmaf(f, __ldcg(ml + x * ml_step + kHeads + h), l);
+            t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
+        }
+        finish(k, make_float4(t.x / l, t.y / l, t.z / l, t.w / l));
+    }
 }
 
 struct Grid {
