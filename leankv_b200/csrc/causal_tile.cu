@@ -44,6 +44,27 @@ __device__ __forceinline__ float ex2(float x) {
     return y;
 }
 
+// Two floats at a time.
+struct Two { float x, y; };
+__device__ __forceinline__ Two fma2(Two a, Two b, Two c) {
+    Two d;
+    asm("{\n\t.reg .b64 a, b, c, d;\n\t"
+        "mov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\t"
+        "fma.rn.f32x2 d, a, b, c;\n\tmov.b64 {%0, %1}, d;\n\t}"
+        : "=f"(d.x), "=f"(d.y)
+        : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+    return d;
+}
+__device__ __forceinline__ Two add2(Two a, Two b) {
+    Two d;
+    asm("{\n\t.reg .b64 a, b, d;\n\t"
+        "mov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\t"
+        "add.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
+        : "=f"(d.x), "=f"(d.y)
+        : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+    return d;
+}
+
 enum { kQ, kKFull, kVFull, kS, kP, kKFree, kVFree, kO, kBars };
 
 __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_constant__ TileArgs p) {
@@ -99,19 +120,23 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
     } else if (tid == 160) {                             // ---- products ----
         constexpr uint32_t idesc_s = tma::idesc_bf16(kTile, false);
         const uint32_t idesc_o = tma::idesc_bf16(p.vdim_pad, true);
+        const uint64_t desc_q = tma::swizzled(sq, 16), desc_k = tma::swizzled(sk, 16), desc_v = tma::swizzled(sv, kBlock);
         ok = umma::bar_wait(bar(kQ), 0);
         for (int j = 0; j < n_tiles && ok; ++j) {
             ok = umma::bar_wait(bar(kKFull), j & 1);
             if (!ok) break;
             umma::fence_after_sync();
+            // a K = 16 step is 32 bytes further in the rows of a block; descriptors count in 16 bytes
             uint32_t first = 0;
-            for (int part = 0; part < 2; ++part) {
-                const int steps = (part == 0 ? p.dim_pad : p.shared_pad) / 16;
-                const uint32_t off = part == 0 ? 0 : p.nb1 * kBlock;
-                for (int s = 0; s < steps; ++s, first = 1) {
-                    const uint32_t o = off + (s >> 2) * kBlock + (s & 3) * 32;
-                    umma::mma_f16_n(tm_s, tma::swizzled(sq + o, 16), tma::swizzled(sk + o, 16), idesc_s, first);
-                }
+            uint64_t dq = desc_q, dk = desc_k;
+            for (int b = 0; b < p.nb1 + p.nb2; ++b, dq += kBlock >> 4, dk += kBlock >> 4) {
+                const int steps = min(4, b < p.nb1 ? p.dim_pad / 16 - b * 4 : p.shared_pad / 16 - (b - p.nb1) * 4);
+#pragma unroll
+                for (int s = 0; s < 4; ++s)
+                    if (s < steps) {
+                        umma::mma_f16_n(tm_s, dq + 2 * s, dk + 2 * s, idesc_s, first);
+                        first = 1;
+                    }
             }
             umma::commit(bar(kS));
             umma::commit(bar(kKFree));
@@ -119,11 +144,11 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
             ok = ok && umma::bar_wait(bar(kP), j & 1);
             if (!ok) break;
             umma::fence_after_sync();
+#pragma unroll
             for (int s = 0; s < kTile / 16; ++s) {       // 16 keys: high parts, then low parts
-                const uint64_t v = tma::swizzled(sv + s * 2048, kBlock);
                 const uint32_t pa = tm_s + (s >> 1) * 32 + (s & 1) * 8;
-                umma::mma_f16_ts(tm_o, pa, v, idesc_o, j > 0 || s > 0);
-                umma::mma_f16_ts(tm_o, pa + 16, v, idesc_o, 1);
+                umma::mma_f16_ts(tm_o, pa, desc_v + s * (2048 >> 4), idesc_o, j > 0 || s > 0);
+                umma::mma_f16_ts(tm_o, pa + 16, desc_v + s * (2048 >> 4), idesc_o, 1);
             }
             umma::commit(bar(kVFree));
             // the next scores go over these weights
@@ -143,23 +168,25 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
             const int at = (t0 + j) * kTile;
             // this row's keys of the tile: from k0 to k1
             const int k0 = max(see0 - at, 0), k1 = min(i - at, kTile - 1);
-            const bool all = k0 == 0 && k1 == kTile - 1;
-            float best = -INFINITY;
-#pragma unroll 1
-            for (int c = 0; c < 4; ++c) {
-                uint32_t s[32];
-                umma::ld32(s, tm_s, row0, c * 32);
-                if (all) {
+            uint32_t s[4][32];
 #pragma unroll
-                    for (int x = 0; x < 32; ++x) best = fmaxf(best, __uint_as_float(s[x]));
-                } else {
+            for (int c = 0; c < 4; ++c) umma::ld32_async(s[c], tm_s, row0, c * 32);
+            umma::settle(s[0]);
 #pragma unroll
-                    for (int x = 0; x < 32; ++x) {
-                        const int k = c * 32 + x;
-                        best = fmaxf(best, k >= k0 && k <= k1 ? __uint_as_float(s[x]) : -INFINITY);
-                    }
-                }
+            for (int c = 1; c < 4; ++c) umma::settled(s[c]);
+            if (__any_sync(0xffffffffu, k0 > 0 || k1 < kTile - 1)) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int x = 0; x < 32; ++x)
+                        if (c * 32 + x < k0 || c * 32 + x > k1) s[c][x] = 0xff800000u;      // -inf
             }
+            float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+#pragma unroll
+                for (int x = 0; x < 32; ++x) top[x & 3] = fmaxf(top[x & 3], __uint_as_float(s[c][x]));
+            const float best = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3]));
             const bool raise = best * p.c > m + kSlack;
             if (__any_sync(0xffffffffu, raise)) {
                 const float mn = raise ? best * p.c : m, f = ex2(m - mn);
@@ -175,25 +202,26 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
                         umma::st32(o, tm_o, row0, c);
                     }
             }
-#pragma unroll 1
+            Two sum[2] = {{0.f, 0.f}, {0.f, 0.f}};
+#pragma unroll
             for (int c = 0; c < 4; ++c) {
-                uint32_t s[32], ph[16], pl[16];
-                umma::ld32(s, tm_s, row0, c * 32);
+                uint32_t ph[16], pl[16];
 #pragma unroll
                 for (int x = 0; x < 32; x += 2) {
-                    float w[2];
-#pragma unroll
-                    for (int y = 0; y < 2; ++y) {
-                        const int k = c * 32 + x + y;
-                        const float e = ex2(fmaf(__uint_as_float(s[x + y]), p.c, -m));
-                        w[y] = all || (k >= k0 && k <= k1) ? e : 0.f;
-                        l += w[y];
-                    }
-                    split_bf16(w[0], w[1], ph[x / 2], pl[x / 2]);
+                    Two w = fma2({__uint_as_float(s[c][x]), __uint_as_float(s[c][x + 1])}, {p.c, p.c}, {-m, -m});
+                    w.x = ex2(w.x);
+                    w.y = ex2(w.y);
+                    sum[(x >> 1) & 1] = add2(sum[(x >> 1) & 1], w);
+                    const uint32_t hi = pack_bf16(w.x, w.y);
+                    const Two left = add2(w, {-__uint_as_float(hi << 16), -__uint_as_float(hi & 0xffff0000u)});
+                    ph[x / 2] = hi;
+                    pl[x / 2] = pack_bf16(left.x, left.y);
                 }
-                umma::st16(ph, tm_s, row0, c * 32);
-                umma::st16(pl, tm_s, row0, c * 32 + 16);
+                umma::st16_async(ph, tm_s, row0, c * 32);
+                umma::st16_async(pl, tm_s, row0, c * 32 + 16);
             }
+            l += (sum[0].x + sum[0].y) + (sum[1].x + sum[1].y);
+            umma::stored();
             umma::fence_before_sync();
             umma::bar_arrive(bar(kP));
         }
@@ -249,7 +277,7 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
 int causal_tile_attend(const leankv_causal_attn_t& a, const void* q, const float* gate, int gate_ld, void* out, int out_ld,
                        int rows, int start, int32_t* status, cudaStream_t st) {
     const int rep = a.heads / a.kv_heads;
-    if (a.dtype != LEANKV_DT_BF16 || rep > kTile || a.vdim_pad > 256 || a.kv_heads > 65535 || a.k_base % kTile ||
+    if (a.dtype != LEANKV_DT_BF16 || !(a.scale > 0.f) || rep > kTile || a.vdim_pad > 256 || a.kv_heads > 65535 || a.k_base % kTile ||
         a.k_ring % kTile || (a.shared_dim > 0 && a.s_ring % kTile))
         return LEANKV_EUNSUPPORTED;
     TileArgs p{};
