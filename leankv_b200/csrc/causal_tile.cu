@@ -74,7 +74,7 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
     __shared__ __align__(8) uint64_t s_bar[kBars];
     __shared__ uint32_t s_tmem;
     pdl_begin();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
     const uint32_t base = (umma::smem_addr(raw) + 1023u) & ~1023u;
     const int nbk = p.nb1 + p.nb2;
     const uint32_t k_bytes = nbk * kKeyBlock, v_bytes = p.v_from_k ? k_bytes : p.nbv * kKeyBlock;      // of a buffer
@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
     umma::fence_before_sync();
     __syncthreads();
     umma::fence_after_sync();
-    const uint32_t tmem = s_tmem, tm_s = tmem, tm_o = tmem + kTile;
+    const uint32_t tmem = __shfl_sync(0xffffffffu, s_tmem, 0), tm_s = tmem, tm_o = tmem + kTile;
 
     const int g = blockIdx.y, q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * p.tq;      // the longest rows first
     const int nt = min(p.tq, p.rows - q0);
@@ -124,50 +124,56 @@ __global__ void __launch_bounds__(kThreads, 2) causal_tile_kernel(const __grid_c
             for (int j = max(nk - 2, 0); j < nk; ++j) wait(kKFull, j);
             for (int j = max(nv - 2, 0); j < nv; ++j) wait(kVFull, j);
         }
-    } else if (tid == 160) {                             // ---- products ----
+    } else if (warp == 5) {                              // ---- products: the whole warp waits, one lane issues ----
         constexpr uint32_t idesc_s = tma::idesc_bf16(kKeys, false);
         const uint32_t idesc_o = tma::idesc_bf16(p.vdim_pad, true);
         const uint64_t desc_q = tma::swizzled(sq, 16), desc_k = tma::swizzled(sk, 16), desc_v = tma::swizzled(sv, kKeyBlock);
+        auto all = [&](bool done) { return __all_sync(0xffffffffu, done) != 0; };
         // a K = 16 step is 32 bytes further in the rows of a block; descriptors count in 16 bytes
         auto scores = [&](int j) {
-            ok = wait(kKFull, j);
+            ok = all(wait(kKFull, j));
             if (!ok) return;
             umma::fence_after_sync();
-            uint32_t first = 0;
+            const uint32_t to = tm_s + (j & 1) * kKeys;
             uint64_t dq = desc_q, dk = desc_k + (j & 1) * (k_bytes >> 4);
-            for (int b = 0; b < nbk; ++b, dq += kBlock >> 4, dk += kKeyBlock >> 4) {
-                const int steps = min(4, b < p.nb1 ? p.dim_pad / 16 - b * 4 : p.shared_pad / 16 - (b - p.nb1) * 4);
+            if (umma::elect()) {
+                for (int b = 0; b < nbk; ++b, dq += kBlock >> 4, dk += kKeyBlock >> 4) {
+                    const int steps = b < p.nb1 ? p.dim_pad / 16 - b * 4 : p.shared_pad / 16 - (b - p.nb1) * 4;
+                    umma::mma_f16_n(to, dq, dk, idesc_s, b > 0);
 #pragma unroll
-                for (int s = 0; s < 4; ++s)
-                    if (s < steps) {
-                        umma::mma_f16_n(tm_s + (j & 1) * kKeys, dq + 2 * s, dk + 2 * s, idesc_s, first);
-                        first = 1;
-                    }
+                    for (int s = 1; s < 4; ++s)
+                        if (s < steps) umma::mma_f16_n(to, dq + 2 * s, dk + 2 * s, idesc_s, 1);
+                }
+                umma::commit(bar(kS + (j & 1)));
+                umma::commit(bar(kKFree + (j & 1)));
             }
-            umma::commit(bar(kS + (j & 1)));
-            umma::commit(bar(kKFree + (j & 1)));
+            __syncwarp();
         };
-        ok = umma::bar_wait(bar(kQ), 0);
+        ok = all(umma::bar_wait(bar(kQ), 0));
         for (int j = 0; j < min(2, n_tiles) && ok; ++j) scores(j);
         for (int j = 0; j < n_tiles && ok; ++j) {
-            if (!p.v_from_k) ok = wait(kVFull, j);
-            ok = ok && wait(kP, j);
+            if (!p.v_from_k) ok = all(wait(kVFull, j));
+            ok = ok && all(wait(kP, j));
             if (!ok) break;
             umma::fence_after_sync();
             const uint64_t dv = desc_v + (j & 1) * (v_bytes >> 4);
+            const uint32_t pa = tm_s + (j & 1) * kKeys;
+            if (umma::elect()) {
 #pragma unroll
-            for (int s = 0; s < kKeys / 16; ++s) {       // 16 keys: high parts, then low parts
-                const uint32_t pa = tm_s + (j & 1) * kKeys + (s >> 1) * 32 + (s & 1) * 8;
-                umma::mma_f16_ts(tm_o, pa, dv + s * (2048 >> 4), idesc_o, j > 0 || s > 0);
-                umma::mma_f16_ts(tm_o, pa + 16, dv + s * (2048 >> 4), idesc_o, 1);
+                for (int s = 0; s < kKeys / 16; ++s) {   // 16 keys: high parts, then low parts
+                    umma::mma_f16_ts(tm_o, pa + (s >> 1) * 32 + (s & 1) * 8, dv + s * (2048 >> 4), idesc_o, j > 0 || s > 0);
+                    umma::mma_f16_ts(tm_o, pa + (s >> 1) * 32 + (s & 1) * 8 + 16, dv + s * (2048 >> 4), idesc_o, 1);
+                }
+                umma::commit(bar(kPV + (j & 1)));
             }
-            umma::commit(bar(kPV + (j & 1)));
+            __syncwarp();
             if (j + 2 < n_tiles) {                       // its scores go over these weights
-                ok = wait(kPV, j);
+                ok = all(wait(kPV, j));
                 if (ok) scores(j + 2);
             }
         }
-        umma::commit(bar(kO));
+        if (umma::elect()) umma::commit(bar(kO));
+        __syncwarp();
         if (!ok) umma::bar_wait(bar(kO), 0);
     } else if (tid < kTile) {                            // ---- rows ----
         const int row0 = warp * 32, used = p.rep * nt;

@@ -51,6 +51,17 @@ __device__ __forceinline__ void mma_f16(uint32_t tmem_d, uint64_t a_desc, uint64
 __device__ __forceinline__ void commit(uint32_t bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
 }
+// true in one lane of a converged warp. Loops that issue MMAs stay warp-uniform around it, so that descriptors are
+// computed in uniform registers.
+__device__ __forceinline__ bool elect() {
+    uint32_t one;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "elect.sync _|p, 0xffffffff;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(one));
+    return one != 0;
+}
 // one warp (all 32 lanes) allocates / frees kTmemCols columns; the base address lands in *slot (shared memory)
 __device__ __forceinline__ void tmem_alloc(uint32_t slot_addr) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(slot_addr), "r"(kTmemCols)
