@@ -147,10 +147,7 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
     const int C = p.cluster, rank = blockIdx.x % C, cluster = blockIdx.x / C;
     const int i = p.s.state[kPos], lo = first_visible(i, a.size), tiles = (i - lo) / KT + 1;
     const int active = max(1, min(p.clusters, (tiles + C * UNITS * kTilesPerUnit - 1) / (C * UNITS * kTilesPerUnit)));
-    if (cluster >= active) {
-        pdl_begin();
-        return;
-    }
+    if (cluster >= active) return;        // without waiting: the clusters that work do
     // tiles j0 .. j1 - 1 of this unit; the last unit has the last tile
     const unsigned unit = (cluster * C + rank) * UNITS + (WARPS ? warp : 0), n_units = active * C * UNITS;
     const int j0 = (int)((unsigned)tiles * unit / n_units), j1 = (int)((unsigned)tiles * (unit + 1) / n_units);
