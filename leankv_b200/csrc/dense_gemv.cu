@@ -92,7 +92,7 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
     constexpr int R = 8 / CH;                        // rows in flight: R * CH 16-byte loads per lane (bf16)
     extern __shared__ __align__(16) float s_dyn[];
     float* s_part = STAGED ? s_dyn + p.x_smem : s_dyn;      // [rows of this CTA (x2 if gated)][warps]
-    __shared__ float s_tmp[32];
+    __shared__ float s_tmp[64];
     const leankv_dense_gemv_t& a = p.a;
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int lo = (int)((long long)a.rows * blockIdx.x / gridDim.x);
@@ -110,6 +110,16 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
         if (off < bytes && part < mult) {
             const char* base = reinterpret_cast<const char*>(W + ((size_t)lo + (size_t)part * a.rows) * cols);
             asm volatile("prefetch.global.L2 [%0];" ::"l"(base + off));
+        }
+    }
+    // kJoined: the gains do not depend on the launch ahead
+    float gn[CH][8], pg[CH][8];
+    if constexpr (JOINED) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int k = (c * warps + warp) * 256 + lane * 8;
+            if (a.gain_per_col) load_x8(a.gain, k, cols, vec, gn[c]);
+            if (a.delta != nullptr) load_x8(a.post_gain, k, cols, vec, pg[c]);
         }
     }
     pdl_begin();
@@ -130,14 +140,12 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
             for (int c = 0; c < CH; ++c)
 #pragma unroll
                 for (int i = 0; i < 8; ++i) sd = fmaf(d[c][i], d[c][i], sd);
-            const float f = a.post_mult / sqrtf(cta_sum(sd, s_tmp) / (float)cols + a.eps);
+            const float f = a.post_mult / sqrtf(cta_sum_once(sd, s_tmp) / (float)cols + a.eps);
 #pragma unroll
             for (int c = 0; c < CH; ++c) {
                 const int k = c * warps * 256 + k0;
-                float g[8];
-                load_x8(a.post_gain, k, cols, vec, g);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) xj[c][i] = fmaf(d[c][i] * f, g[i], xj[c][i]);
+                for (int i = 0; i < 8; ++i) xj[c][i] = fmaf(d[c][i] * f, pg[c][i], xj[c][i]);
                 if (blockIdx.x == 0)
 #pragma unroll
                     for (int i = 0; i < 8; ++i)
@@ -149,14 +157,11 @@ __global__ void __launch_bounds__(512, sizeof(T) == 2 ? 2 : 1) dense_gemv_kernel
 #pragma unroll
             for (int i = 0; i < 8; ++i) ss = fmaf(xj[c][i], xj[c][i], ss);
         if (a.gain != nullptr) {
-            rs = (a.gain_per_col ? 1.f : __ldg(a.gain)) / sqrtf(cta_sum(ss, s_tmp) / (float)cols + a.eps);
+            rs = (a.gain_per_col ? 1.f : __ldg(a.gain)) / sqrtf(cta_sum_once(ss, s_tmp + 32) / (float)cols + a.eps);
 #pragma unroll
-            for (int c = 0; c < CH; ++c) {
-                float g[8];
-                if (a.gain_per_col) load_x8(a.gain, c * warps * 256 + k0, cols, vec, g);
+            for (int c = 0; c < CH; ++c)
 #pragma unroll
-                for (int i = 0; i < 8; ++i) xj[c][i] *= a.gain_per_col ? rs * g[i] : rs;
-            }
+                for (int i = 0; i < 8; ++i) xj[c][i] *= a.gain_per_col ? rs * gn[c][i] : rs;
         }
         if (a.prev != nullptr && blockIdx.x == 0) {
             float* next = a.prev + (size_t)((a.state[kParity] & 1) ^ 1) * cols;

@@ -68,8 +68,9 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
-// Sum over the CTA (whole warps), the same value in every thread; s_tmp holds 32 floats.
-__device__ __forceinline__ float cta_sum(float v, float* s_tmp) {
+// Sum over the CTA (whole warps), the same value in every thread; s_tmp holds 32 floats. The `once` form leaves
+// s_tmp in use until the next barrier.
+__device__ __forceinline__ float cta_sum_once(float v, float* s_tmp) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     v = warp_sum(v);
     if (lane == 0) s_tmp[warp] = v;
@@ -77,6 +78,10 @@ __device__ __forceinline__ float cta_sum(float v, float* s_tmp) {
     const int nw = (blockDim.x + 31) >> 5;
     float t = 0.f;
     for (int w = 0; w < nw; ++w) t += s_tmp[w];   // fixed order: bit-reproducible
+    return t;
+}
+__device__ __forceinline__ float cta_sum(float v, float* s_tmp) {
+    const float t = cta_sum_once(v, s_tmp);
     __syncthreads();
     return t;
 }
