@@ -142,9 +142,9 @@ __global__ void __launch_bounds__(32 * warps_of(W), W == Walk::kWarps ? 2 : 1) c
     const leankv_causal_attn_t& a = p.a;
     const StepPlan& pl = p.plan;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int gb = blockIdx.y, g = gb / p.blocks, hb = gb % p.blocks, rep = a.heads / a.kv_heads;
+    const int C = p.cluster, rank = blockIdx.x % C, gb = blockIdx.x / C, cluster = blockIdx.y;      // idle clusters come last
+    const int g = gb / p.blocks, hb = gb % p.blocks, rep = a.heads / a.kv_heads;
     const int h0 = g * rep + hb * kHeads, nh = min(kHeads, rep - hb * kHeads);
-    const int C = p.cluster, rank = blockIdx.x % C, cluster = blockIdx.x / C;
     const int i = p.s.state[kPos], lo = first_visible(i, a.size), tiles = (i - lo) / KT + 1;
     const int active = max(1, min(p.clusters, (tiles + C * UNITS * kTilesPerUnit - 1) / (C * UNITS * kTilesPerUnit)));
     if (cluster >= active) return;        // without waiting: the clusters that work do
@@ -690,7 +690,7 @@ int launch_step(StepArgs p, cudaStream_t st) {
     for (const int clusters8 = p.clusters;;) {
         p.cluster = p.cluster == kMaxCluster ? 8 : kMaxCluster;
         p.clusters = p.cluster == 8 ? clusters8 : (clusters8 + 1) / 2;
-        const dim3 grid(p.cluster * p.clusters, groups);
+        const dim3 grid(p.cluster * groups, p.clusters);
         if (p.cluster > 8) {                             // does a cluster of this size fit this device, often enough?
             cudaLaunchConfig_t cfg = {};
             cfg.gridDim = grid;
