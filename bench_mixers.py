@@ -170,7 +170,6 @@ def pefitar_leg(size, dev, steps, peaks):
 
     from leankv_b200 import _native
     from leankv_b200.mixer_engine import MixerDecodeEngine, MixerModelConfig
-    from leankv_b200.mixers import pad16
 
     width, heads, kv, _, ff, layers = SIZES[size]
     cfg = MixerModelConfig.from_dict(pefitar_config(*SIZES[size]))
